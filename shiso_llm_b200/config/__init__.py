@@ -16,10 +16,12 @@ from . import filulix  # registers Filulix
 from . import zetavik  # registers Zetavik
 from . import volalorn  # registers Volalorn
 from . import povilorn  # registers Povilorn
+from . import nodepel  # registers Nodepel
 from .filulix import FilulixConfig
 from .zetavik import ZetavikConfig
 from .volalorn import VolalornConfig
 from .povilorn import PovilornConfig
+from .nodepel import NodepelConfig
 from .lfm2 import Lfm2Config, feed_forward_width
 
 __all__ = [
@@ -29,6 +31,7 @@ __all__ = [
     "FilulixConfig",
     "InvalidValue",
     "Lfm2Config",
+    "NodepelConfig",
     "PovilornConfig",
     "UnknownArchitecture",
     "UnsupportedShape",

@@ -83,6 +83,7 @@ struct DecodeTmaArgs {
     __nv_bfloat16* v_cache;
     float eps;
     int store;
+    const float* sink;        // [heads] or null: exp(sink) joins a head's softmax sum, with no key and no value
 };
 
 __device__ __forceinline__ void ldsm_x4(uint32_t addr, uint32_t& r0, uint32_t& r1, uint32_t& r2, uint32_t& r3) {
@@ -105,6 +106,12 @@ __device__ __forceinline__ void mma16816(float* c, const uint32_t* a, uint32_t b
 __device__ __forceinline__ uint32_t pack2(float lo, float hi) {
     __nv_bfloat162 v = __floats2bfloat162_rn(lo, hi);
     return *reinterpret_cast<uint32_t*>(&v);
+}
+
+// What a head's sink adds to its softmax sum against the maximum `m` (log2 units); infinite where
+// the sink outweighs every key by 2^128 and more, and the head's output is then the zero it tends to.
+__device__ __forceinline__ float sink_share(const DecodeTmaArgs& a, size_t row_head, float m) {
+    return a.sink ? exp2f(a.sink[row_head % a.heads] * 1.4426950408889634f - m) : 0.0f;
 }
 
 // All threads of all CTAs of the cluster meet.
@@ -490,6 +497,7 @@ decode_tma_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_consta
         }
         if (alone) {
             const size_t head = (size_t)t * a.heads + g_head * group + h;
+            sum += sink_share(a, head, m);
             a.out[head * HEAD + col] = __float2bfloat16_rn(sum > 0.0f ? o / sum : 0.0f);
         } else {
             const uint32_t row = in_cta(inbox_local, (uint32_t)(h % parts)) + (uint32_t)(((h / parts) * parts + split) * MERGE_ROW) * 4u;
@@ -516,6 +524,7 @@ decode_tma_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_consta
                 acc += f * base[s * MERGE_ROW + col];
             }
             const size_t head = (size_t)t * a.heads + g_head * group + h;
+            sum += sink_share(a, head, m);
             a.out[head * HEAD + col] = __float2bfloat16_rn(sum > 0.0f ? acc / sum : 0.0f);
         }
     }
@@ -707,11 +716,12 @@ SHISO_API int shiso_decode_attention_from_qkv(const void* qkv, const float* q_w,
 
 // shiso_decode_attention_fused for a window that keeps the first `keep_first` positions of every
 // sequence visible at their true positions; q may be a column range of wider rows (q_ld elements apart).
+// `sink` ([heads] float, or null): exp(sink[h]) joins head h's softmax sum.
 SHISO_API int shiso_decode_attention_fused_kept(const void* q, long long q_ld, const void* k_cache, const void* v_cache,
                                                 const int* block_table, int table_width, const int* positions,
                                                 const int* seq_of_token, void* out, int tokens, int heads, int kv_heads,
                                                 int head_dim, int page_size, long long num_pages, float scale, int window,
-                                                int keep_first, int splits, cudaStream_t stream) {
+                                                int keep_first, int splits, const float* sink, cudaStream_t stream) {
     if (tokens <= 0) return SHISO_OK;
     if (((uintptr_t)q & 15) || (q_ld % 8) || keep_first < 0) return SHISO_ERR_ALIGN;
     DecodeTmaArgs a;
@@ -723,6 +733,7 @@ SHISO_API int shiso_decode_attention_fused_kept(const void* q, long long q_ld, c
     a.q = (const __nv_bfloat16*)q;
     a.q_ld = q_ld;
     a.keep_first = keep_first;
+    a.sink = sink;
     return launch_decode_tma<false>(mk, mv, a, tokens, stream);
 }
 

@@ -65,6 +65,7 @@ struct TcArgs {
     int cache_rows;          // pages * page size: a row coordinate from here on reads zeros
     float scale_log2;        // scale * log2(e)
     float out_scale;         // a constant the normalised result is multiplied by
+    const float* sink;       // [heads] or null: exp(sink) joins a head's softmax sum, with no key and no value
 };
 
 __device__ __forceinline__ float ex2(float x) {
@@ -368,6 +369,8 @@ flash_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant
         pdl_trigger();
         if (!mbar_wait(&pv_done[(num_tiles - 1) & 1], ((num_tiles - 1) >> 1) & 1)) failed = true;
         asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
+        // (a sink that outweighs every key by 2^128 makes its share infinite and the output the zero it tends to)
+        if (a.sink && row_sum > 0.0f) row_sum += exp2f(a.sink[head] * 1.4426950408889634f - row_max);
         const float inv = row_sum > 0.0f ? a.out_scale / row_sum : 0.0f;  // an empty span yields zeros
         if (a.log_sum && r < rows)  // for a caller that folds further keys into the same softmax
             a.log_sum[(size_t)(first_token + r) * a.heads + head] =
@@ -431,7 +434,8 @@ static bool strided_map(const void* ptr, int rows, int cols, long long ld, CUten
 static int launch_flash_tc(const void* q, long long q_ld, const void* k_cache, const void* v_cache, const int* block_table,
                            int table_width, const int* q_start, const int* start_pos, void* out, long long out_ld,
                            float* log_sum, float out_scale, int tokens, int num_seqs, int max_tiles, int heads, int kv_heads,
-                           int page_size, long long num_pages, float scale, int window, cudaStream_t stream, int keep_first = 0) {
+                           int page_size, long long num_pages, float scale, int window, cudaStream_t stream, int keep_first = 0,
+                           const float* sink = nullptr) {
     if (num_seqs <= 0 || max_tiles <= 0 || tokens <= 0) return SHISO_OK;
     if (keep_first < 0) return SHISO_ERR_SHAPE;
     if (kv_heads <= 0 || heads % kv_heads) return SHISO_ERR_SHAPE;
@@ -462,6 +466,7 @@ static int launch_flash_tc(const void* q, long long q_ld, const void* k_cache, c
     a.cache_rows = (int)cache_rows;
     a.scale_log2 = scale * 1.4426950408889634f;
     a.out_scale = out_scale;
+    a.sink = sink;
     static bool configured = false;
     if (!configured) {
         cudaError_t e = cudaFuncSetAttribute(flash_tc_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, SMEM_BYTES);
@@ -507,11 +512,12 @@ SHISO_API int shiso_prefill_attention_tc_open(const void* q, long long q_ld, con
 
 // The same for a window that keeps the first `keep_first` positions of every sequence visible (at
 // their true positions) to all later rows; queries and outputs may be column ranges of wider rows.
+// `sink` ([heads] float, or null): exp(sink[h]) joins head h's softmax sum.
 SHISO_API int shiso_prefill_attention_tc_kept(const void* q, long long q_ld, const void* k_cache, const void* v_cache,
                                               const int* block_table, int table_width, const int* q_start, const int* start_pos,
                                               void* out, long long out_ld, int tokens, int num_seqs, int max_tiles, int heads,
                                               int kv_heads, int page_size, long long num_pages, float scale, int window,
-                                              int keep_first, cudaStream_t stream) {
+                                              int keep_first, const float* sink, cudaStream_t stream) {
     return launch_flash_tc(q, q_ld, k_cache, v_cache, block_table, table_width, q_start, start_pos, out, out_ld, nullptr, 1.0f, tokens,
-                           num_seqs, max_tiles, heads, kv_heads, page_size, num_pages, scale, window, stream, keep_first);
+                           num_seqs, max_tiles, heads, kv_heads, page_size, num_pages, scale, window, stream, keep_first, sink);
 }

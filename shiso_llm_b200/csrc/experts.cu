@@ -6,7 +6,7 @@
 // gather[m] / gather_div).  CUDA cores, float accumulation, a tile of 32 rows x 64 outputs per CTA
 // and 32 columns of K per pass; an output's sum runs over K in order, whatever else is in its tile, so
 // a row's result does not depend on the batch.  Epilogues: none; times sigmoid(gate[m, b]); or, for
-// a matrix that stacks gate over up rows, the gated pair glu_pair(gate, up): silu(gate) * up, the
+// a plain matrix, the square of relu; for one that stacks gate over up rows, the gated pair glu_pair(gate, up): silu(gate) * up, the
 // tanh form of gelu(gate) * up, or the clamped pair min(g, L) sigmoid(1.702 min(g, L)) (clamp(u, -L, L) + 1).
 // bfloat16 inputs whose strides allow 16-byte copies take tile_gemm_mma_kernel instead: the same
 // tiles on the tensor cores.
@@ -25,7 +25,7 @@
 #define MOE_MAX_EXPERTS 256
 #define MOE_MAX_TOP 16
 
-enum { GLU_SILU = 0, GLU_GELU_TANH = 1, GLU_SWISH_CLAMPED = 2 };
+enum { GLU_SILU = 0, GLU_GELU_TANH = 1, GLU_SWISH_CLAMPED = 2, ACT_RELU2 = 3 };  // the last: an ungated max(z, 0)^2
 
 // The gated pair of a feed-forward, in float with the library's expf and tanhf.
 __device__ __forceinline__ float glu_pair(float g, float u, int act, float limit) {
@@ -51,7 +51,7 @@ struct TileGemmArgs {
     const void* gate;
     long long gate_ld;
     int M, N, K, batches;
-    int act;      // the gated pair of a stacked gate/up matrix (GLU_*)
+    int act;      // the gated pair of a stacked gate/up matrix (GLU_*), or ACT_RELU2 on a plain one
     float limit;  // its clamp
 };
 
@@ -145,6 +145,7 @@ __global__ void __launch_bounds__(256) tile_gemm_kernel(const TileGemmArgs a) {
             if (n >= a.N) continue;
             float v = acc[i][j];
             if (GLU) v = glu_pair(v, acc2[i][j], a.act, a.limit);
+            else if (a.act == ACT_RELU2) v = fmaxf(v, 0.0f), v *= v;
             out[(size_t)m * a.out_ld + n] = from_f32<OT>(v * scale);
         }
     }
@@ -307,6 +308,7 @@ __global__ void __launch_bounds__(256) tile_gemm_mma_kernel(const TileGemmArgs a
                     if (n >= a.N) continue;
                     float v = acc[mi][nj][hrow * 2 + e];
                     if (GLU) v = glu_pair(v, acc2[mi][nj][hrow * 2 + e], a.act, a.limit);
+                    else if (a.act == ACT_RELU2) v = fmaxf(v, 0.0f), v *= v;
                     out[(size_t)m * a.out_ld + n] = from_f32<OT>(v * scale);
                 }
             }
@@ -365,14 +367,17 @@ SHISO_API int shiso_head_linear(const void* x, long long x_ld, long long x_hs, i
 
 // --------------------------------------------------------------------------- routing
 
+enum { ROUTE_SOFTMAX = 0, ROUTE_SIGMOID = 1, ROUTE_CHOSEN_SOFTMAX = 2 };
+
 // A warp per row.  scores = softmax(logits) (or sigmoids); experts and groups are ranked by the
 // choice score = score + correction[e] (which may be negative); experts in `group_count` groups of
 // neighbours, a group's value its largest choice score; the `group_keep` best groups stay; among
 // their experts the `top` largest choice scores win (the lower index on a tie); weight = score
-// (/ (the chosen scores' sum + renorm_eps)) * scale.  Rows of logits are `ld` apart.
+// (/ (the chosen scores' sum + renorm_eps)) * scale.  ROUTE_CHOSEN_SOFTMAX: the scores are the logits
+// themselves, and the weights the softmax over the chosen ones, times scale.  Rows of logits are `ld` apart.
 __global__ void moe_route_kernel(const float* __restrict__ logits, long long ld, const float* __restrict__ correction,
                                  int* __restrict__ ids, float* __restrict__ weights, int tokens, int experts, int top,
-                                 int group_count, int group_keep, float scale, int sigmoid, int renormalize, float renorm_eps) {
+                                 int group_count, int group_keep, float scale, int scoring, int renormalize, float renorm_eps) {
     pdl_begin();
     __shared__ float s_scores[8][MOE_MAX_EXPERTS];
     __shared__ float s_choice[8][MOE_MAX_EXPERTS];  // NaN once taken: no comparison picks it again
@@ -386,17 +391,18 @@ __global__ void moe_route_kernel(const float* __restrict__ logits, long long ld,
     float* gs = s_group[warp];
     unsigned char* kept = s_kept[warp];
     const float* z = logits + (size_t)t * ld;
+    const bool sigmoid = scoring == ROUTE_SIGMOID, plain = scoring == ROUTE_CHOSEN_SOFTMAX;
     float mx = -INFINITY;
     for (int e = lane; e < experts; e += 32) mx = fmaxf(mx, z[e]);
     mx = warp_max(mx);
     float sum = 0.0f;
     for (int e = lane; e < experts; e += 32) {
-        const float v = sigmoid ? 1.0f / (1.0f + expf(-z[e])) : expf(z[e] - mx);
+        const float v = plain ? z[e] : sigmoid ? 1.0f / (1.0f + expf(-z[e])) : expf(z[e] - mx);
         sc[e] = v;
         sum += v;
     }
     sum = warp_sum(sum);
-    const float inv = sigmoid ? 1.0f : 1.0f / sum;
+    const float inv = sigmoid || plain ? 1.0f : 1.0f / sum;
     for (int e = lane; e < experts; e += 32) {
         const float v = sc[e] * inv;
         sc[e] = v;
@@ -449,22 +455,27 @@ __global__ void moe_route_kernel(const float* __restrict__ logits, long long ld,
         if (lane == 0) ch[at] = NAN;  // taken
         __syncwarp();
     }
+    if (plain) {
+        const float most = warp_max(lane < top ? my_w : -INFINITY);
+        my_w = lane < top ? expf(my_w - most) : 0.0f;
+        my_w /= warp_sum(my_w);
+    }
     if (lane < top) {
         ids[(size_t)t * top + lane] = my_id;
-        weights[(size_t)t * top + lane] = (renormalize ? my_w / (chosen_sum + renorm_eps) : my_w) * scale;
+        weights[(size_t)t * top + lane] = (renormalize && !plain ? my_w / (chosen_sum + renorm_eps) : my_w) * scale;
     }
 }
 
 SHISO_API int shiso_moe_route(const float* logits, long long ld, const float* correction, int* ids, float* weights, int tokens,
-                              int experts, int top, int group_count, int group_keep, float scale, int sigmoid, int renormalize,
+                              int experts, int top, int group_count, int group_keep, float scale, int scoring, int renormalize,
                               float renorm_eps, cudaStream_t stream) {
     if (tokens <= 0) return SHISO_OK;
     if (experts <= 0 || experts > MOE_MAX_EXPERTS || top <= 0 || top > MOE_MAX_TOP || top > experts || group_count <= 0 ||
         experts % group_count || group_keep <= 0 || group_keep > group_count || group_keep * (experts / group_count) < top ||
-        ld < experts)
+        ld < experts || scoring < ROUTE_SOFTMAX || scoring > ROUTE_CHOSEN_SOFTMAX)
         return SHISO_ERR_SHAPE;
     launch_kernel(moe_route_kernel, ceil_div_u(tokens, 8), 256, 0, stream, logits, ld, correction, ids, weights, tokens, experts, top,
-                  group_count, group_keep, scale, sigmoid, renormalize, renorm_eps);
+                  group_count, group_keep, scale, scoring, renormalize, renorm_eps);
     return launch_status();
 }
 
@@ -525,6 +536,7 @@ __global__ void moe_combine_kernel(const float* __restrict__ y, const int* __res
 }
 
 // The experts of one step.  ids / weights [T, top]; gate_up [E, 2 ff, hidden]; down [E, hidden, ff];
+// with act ACT_RELU2 the experts are ungated: gate_up is [E, ff, hidden] and `mid` max(z, 0)^2;
 // ids from E up to E + identity - 1 are identity experts (no matrices: their rows are grouped
 // behind the others' and never multiplied); `act` / `limit`: the experts' gated pair; extra: rows
 // added to every token (a shared expert's), times sigmoid(extra_gate[t * extra_gate_ld]) if given.
@@ -536,7 +548,7 @@ SHISO_API int shiso_routed_experts(const void* x, int act_dtype, const int* ids,
     if (tokens <= 0) return SHISO_OK;
     const int outputs = experts + identity;
     if (experts <= 0 || identity < 0 || outputs > MOE_MAX_EXPERTS || top <= 0 || hidden <= 0 || ff <= 0 || act < GLU_SILU ||
-        act > GLU_SWISH_CLAMPED)
+        act > ACT_RELU2)
         return SHISO_ERR_SHAPE;
     const int total = tokens * top;
     int* counts = ints;
@@ -549,8 +561,10 @@ SHISO_API int shiso_routed_experts(const void* x, int act_dtype, const int* ids,
                   total, outputs);
     int status = launch_status();
     if (status) return status;
-    TileGemmArgs up = {x, hidden, 0, source, top, gate_up, (long long)2 * ff * hidden, mid, ff, 0, counts, nullptr, 0, total, ff, hidden, experts, act, limit};
-    status = launch_tile_gemm<true>(up, act_dtype, w_dtype, act_dtype, total, experts, 1, stream);
+    const int halves = act == ACT_RELU2 ? 1 : 2;  // an ungated expert has one matrix before its activation
+    TileGemmArgs up = {x, hidden, 0, source, top, gate_up, (long long)halves * ff * hidden, mid, ff, 0, counts, nullptr, 0, total, ff, hidden, experts, act, limit};
+    status = halves == 2 ? launch_tile_gemm<true>(up, act_dtype, w_dtype, act_dtype, total, experts, 1, stream)
+                         : launch_tile_gemm<false>(up, act_dtype, w_dtype, act_dtype, total, experts, 1, stream);
     if (status) return status;
     TileGemmArgs dn = {mid, ff, 0, nullptr, 1, down, (long long)hidden * ff, y, hidden, 0, counts, nullptr, 0, total, hidden, ff, experts, 0, 0.0f};
     status = launch_tile_gemm<false>(dn, act_dtype, w_dtype, SHISO_F32, total, experts, 1, stream);

@@ -11,7 +11,8 @@
 //               chunk   j <= i with j / size == i / size, chunks counted from position 0.
 //             A score is (q . k) * scale, then softcap * tanh(score / softcap) when a cap is
 //             given.  Weights are a softmax over the visible keys, or sigmoid(score + bias[head])
-//             per key with no normalisation.  The head's output may be multiplied by
+//             per key with no normalisation; a softmax may have a sink per head, exp(sink[head]) in
+//             its denominator with no key and no value.  The head's output may be multiplied by
 //             sigmoid(gate[row, head]) - or, with a wide gate, every output entry by the sigmoid of its own column.
 //
 // The visible keys form two lists in position order - the kept first positions that lie before
@@ -271,6 +272,7 @@ struct MaskedArgs {
     const int* positions;
     const int* seq_of_token;
     const float* key_bias;  // [heads], sigmoid weighting only; may be null
+    const float* sink;      // [heads], softmax only; may be null: exp(sink) joins a head's sum, with no key and no value
     long long q_ld, out_ld, gate_ld;
     int table_width, heads, kv_heads, dim, vdim, page_size, mask_kind, size, keep_first;
     int gate_wide;   // the gate has a column per output entry (heads * vdim) instead of one per head
@@ -454,6 +456,7 @@ masked_attention_kernel(const AT* __restrict__ q, const AT* __restrict__ k_cache
         factor[w] = part_max[w] == -INFINITY ? 0.0f : expf(part_max[w] - top);
         total += part_sum[w] * factor[w];
     }
+    if (a.sink) total += expf(a.sink[head] - top);  // (infinite where it outweighs every key by e^88: the output tends to zero)
     for (int c = threadIdx.x; c < a.vdim; c += blockDim.x) {
         float sum = 0.0f;
 #pragma unroll
@@ -484,6 +487,7 @@ masked_attention_merge_kernel(AT* out, const AT* __restrict__ gate, MaskedArgs a
             const float m = parts[(size_t)s * (a.vdim + 2) + a.vdim];
             total += parts[(size_t)s * (a.vdim + 2) + a.vdim + 1] * (m == -INFINITY ? 0.0f : expf(m - top));
         }
+        if (a.sink) total += expf(a.sink[head] - top);
     }
     for (int c = threadIdx.x; c < a.vdim; c += blockDim.x) {
         float sum = 0.0f;
@@ -573,7 +577,7 @@ SHISO_API int shiso_masked_attention(const void* q, long long q_ld, int act_dtyp
                                      long long out_ld, const void* gate, long long gate_ld, const float* key_bias, int tokens,
                                      int heads, int kv_heads, int dim, int vdim, int page_size, float scale, float softcap,
                                      int mask_kind, int size, int keep_first, int sigmoid, int splits, float* scratch,
-                                     int gate_wide, cudaStream_t stream) {
+                                     int gate_wide, const float* sink, cudaStream_t stream) {
     if (tokens <= 0) return SHISO_OK;
     if (splits < 1 || (splits > 1 && !scratch)) return SHISO_ERR_SHAPE;
     if (dim <= 0 || dim > MA_MAX_DIM || vdim <= 0 || vdim > MA_MAX_DIM || kv_heads <= 0 || heads % kv_heads || size < 1 || keep_first < 0 ||
@@ -585,6 +589,7 @@ SHISO_API int shiso_masked_attention(const void* q, long long q_ld, int act_dtyp
     a.positions = positions;
     a.seq_of_token = seq_of_token;
     a.key_bias = key_bias;
+    a.sink = sink;
     a.q_ld = q_ld;
     a.out_ld = out_ld;
     a.gate_ld = gate_ld;

@@ -2,7 +2,7 @@
 //
 // The same function as the general kernel of masked_attention.cu - a window with kept first
 // positions or chunks counted from position 0, scores optionally capped through a tanh, weights a
-// softmax or one sigmoid per key, a gate per head on the output - computed 64 query rows at a
+// softmax (with or without a sink per head) or one sigmoid per key, a gate per head on the output - computed 64 query rows at a
 // time on the tensor cores.  One CTA owns 64 consecutive rows of one sequence and one query
 // head; four warps, 16 rows each.  It walks the key tiles (64 positions, aligned to multiples of
 // 64 of the sequence) that its rows can see: first the tiles that hold kept first positions and
@@ -36,6 +36,7 @@ struct TileArgs {
     const __nv_bfloat16* v_cache;  // [pages, page, kv_heads, vdim]
     const __nv_bfloat16* gate;     // [T, ...] rows gate_ld apart, head h at column h; or null
     const float* key_bias;         // [heads] or null
+    const float* sink;             // [heads] or null (softmax): exp(sink) joins a head's sum, with no key and no value
     const int* block_table;        // [S, width]
     const int* q_start;            // [S + 1]
     const int* start_pos;          // [S]
@@ -295,6 +296,8 @@ masked_tiles_kernel(TileArgs a) {
             float s = row_sum[r];
             s += __shfl_xor_sync(0xffffffffu, s, 1);
             s += __shfl_xor_sync(0xffffffffu, s, 2);
+            // (a sink that outweighs every key by 2^128 makes its share infinite and the output the zero it tends to)
+            if (a.sink && s > 0.0f) s += exp2f(a.sink[head] * LOG2E - row_max[r]);
             factor[r] = s > 0.0f ? 1.0f / s : 0.0f;
         }
     }
@@ -351,7 +354,8 @@ SHISO_API int shiso_masked_attention_tiles(const void* q, long long q_ld, const 
                                            int table_width, const int* q_start, const int* start_pos, void* out, long long out_ld,
                                            const void* gate, long long gate_ld, const float* key_bias, int num_seqs, int max_tiles,
                                            int heads, int kv_heads, int dim, int vdim, int page_size, float scale, float softcap,
-                                           int mask_kind, int size, int keep_first, int sigmoid, int gate_wide, cudaStream_t stream) {
+                                           int mask_kind, int size, int keep_first, int sigmoid, int gate_wide, const float* sink,
+                                           cudaStream_t stream) {
     if (num_seqs <= 0 || max_tiles <= 0) return SHISO_OK;
     if (kv_heads <= 0 || heads % kv_heads || size < 1 || keep_first < 0 || (mask_kind != MT_MASK_WINDOW && mask_kind != MT_MASK_CHUNK))
         return SHISO_ERR_SHAPE;
@@ -363,6 +367,7 @@ SHISO_API int shiso_masked_attention_tiles(const void* q, long long q_ld, const 
     a.v_cache = (const __nv_bfloat16*)v_cache;
     a.gate = (const __nv_bfloat16*)gate;
     a.key_bias = key_bias;
+    a.sink = sink;
     a.block_table = table;
     a.q_start = q_start;
     a.start_pos = start_pos;

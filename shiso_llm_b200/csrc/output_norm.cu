@@ -2,6 +2,8 @@
 //
 //   norm_into   residual[t] += y[t] * rsqrt(mean(y[t]^2) + eps) * w   (float, in place), and, when
 //               asked, the new residual row in the activation type: what the next sublayer reads.
+//   normed_pair residual[t] += scale * (norm(left[t]) + norm(right[t])), and the norm of the new row: what
+//               closes a mixer of two branches and opens the sublayer behind it.
 //   polynorm    out[t] = a * N(z[t]) + b * N(z[t]^2) + c * N(z[t]^3) + e, powers taken element by
 //               element, N(u) = u * rsqrt(mean(u^2) + eps) over the row.
 //
@@ -149,6 +151,110 @@ bool aligned16(const void* a, const void* b, const void* c, const void* d) {
     return !(((uintptr_t)a | (uintptr_t)b | (uintptr_t)c | (uintptr_t)d) & 15);
 }
 
+
+// --------------------------------------------------------------------------- two outputs, each normed, halved or otherwise scaled
+
+// d[t] = scale * (a[t] * rsqrt(mean(a[t]^2) + eps) * wa + b[t] * rsqrt(mean(b[t]^2) + eps) * wb), and then, as far as asked:
+//   residual given, rows null   residual[t] += d[t] (stored), out[t] = norm(residual[t]) with weight w
+//   residual given, rows given  out[r] = norm(residual[rows[r]] + d[rows[r]]), the residual left alone
+//   residual null               sum[t] = d[t] (float)
+// A thread takes N neighbouring columns at a time; the row of sums waits in shared memory for its own
+// statistic.
+struct NormedPairArgs {
+    float* residual;
+    const int* rows;
+    const float *wa, *wb, *w;
+    float* sum;
+    int hidden;
+    float scale, pair_eps, eps;
+};
+
+template <int N> __device__ __forceinline__ void pair_load(const float* p, float (&v)[N]) {
+    if constexpr (N == 8) {
+        const float4 a = reinterpret_cast<const float4*>(p)[0], b = reinterpret_cast<const float4*>(p)[1];
+        v[0] = a.x, v[1] = a.y, v[2] = a.z, v[3] = a.w, v[4] = b.x, v[5] = b.y, v[6] = b.z, v[7] = b.w;
+    } else {
+        v[0] = p[0];
+    }
+}
+template <int N> __device__ __forceinline__ void pair_load(const __nv_bfloat16* p, float (&v)[N]) {
+    if constexpr (N == 8) unpack8(*reinterpret_cast<const uint4*>(p), v);
+    else v[0] = __bfloat162float(p[0]);
+}
+template <int N> __device__ __forceinline__ void pair_store(float* p, const float (&v)[N]) {
+    if constexpr (N == 8) {
+        reinterpret_cast<float4*>(p)[0] = make_float4(v[0], v[1], v[2], v[3]);
+        reinterpret_cast<float4*>(p)[1] = make_float4(v[4], v[5], v[6], v[7]);
+    } else {
+        p[0] = v[0];
+    }
+}
+template <int N> __device__ __forceinline__ void pair_store(__nv_bfloat16* p, const float (&v)[N]) {
+    if constexpr (N == 8) *reinterpret_cast<uint4*>(p) = pack8(v);
+    else p[0] = __float2bfloat16_rn(v[0]);
+}
+
+template <typename AT, int N>
+__global__ void normed_pair_kernel(const NormedPairArgs a, const AT* __restrict__ left, const AT* __restrict__ right, AT* __restrict__ out) {
+    __shared__ float scratch[33];
+    extern __shared__ __align__(16) float row_cache[];
+    pdl_begin();
+    const int src = a.rows ? a.rows[blockIdx.x] : blockIdx.x;
+    const AT* l = left + (size_t)src * a.hidden;
+    const AT* r = right + (size_t)src * a.hidden;
+    const int first = threadIdx.x * N, stride = blockDim.x * N;
+    float sl = 0.0f, sr = 0.0f;
+    for (int i = first; i < a.hidden; i += stride) {
+        float x[N], y[N];
+        pair_load<N>(l + i, x);
+        pair_load<N>(r + i, y);
+#pragma unroll
+        for (int e = 0; e < N; ++e) sl += x[e] * x[e], sr += y[e] * y[e];
+    }
+    const float il = rsqrtf(block_sum(sl, scratch) / (float)a.hidden + a.pair_eps);
+    const float ir = rsqrtf(block_sum(sr, scratch) / (float)a.hidden + a.pair_eps);
+    float* res = a.residual ? a.residual + (size_t)src * a.hidden : nullptr;
+    float ss = 0.0f;
+    for (int i = first; i < a.hidden; i += stride) {
+        float x[N], y[N], wl[N], wr[N];
+        pair_load<N>(l + i, x);
+        pair_load<N>(r + i, y);
+        pair_load<N>(a.wa + i, wl);
+        pair_load<N>(a.wb + i, wr);
+#pragma unroll
+        for (int e = 0; e < N; ++e) x[e] = a.scale * (x[e] * il * wl[e] + y[e] * ir * wr[e]);
+        if (!res) {
+            pair_store<N>(a.sum + (size_t)blockIdx.x * a.hidden + i, x);
+            continue;
+        }
+        pair_load<N>(res + i, y);
+#pragma unroll
+        for (int e = 0; e < N; ++e) x[e] += y[e], ss += x[e] * x[e];
+        if (!a.rows) pair_store<N>(res + i, x);
+        pair_store<N>(row_cache + i, x);
+    }
+    if (!res) return;
+    const float inv = rsqrtf(block_sum(ss, scratch) / (float)a.hidden + a.eps);
+    for (int i = first; i < a.hidden; i += stride) {  // what this thread wrote itself
+        float x[N], w[N];
+        pair_load<N>(row_cache + i, x);
+        pair_load<N>(a.w + i, w);
+#pragma unroll
+        for (int e = 0; e < N; ++e) x[e] = x[e] * inv * w[e];
+        pair_store<N>(out + (size_t)blockIdx.x * a.hidden + i, x);
+    }
+}
+
+template <typename AT>
+int launch_normed_pair(const NormedPairArgs& a, const void* left, const void* right, void* out, int out_rows, bool wide, cudaStream_t stream) {
+    const size_t smem = a.residual ? (size_t)a.hidden * sizeof(float) : 0;
+    auto kernel = wide ? normed_pair_kernel<AT, 8> : normed_pair_kernel<AT, 1>;
+    if (smem > 48 * 1024) cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+    launch_kernel(kernel, out_rows, wide ? vec_block_for(a.hidden) : block_for(a.hidden), smem, stream, a, (const AT*)left, (const AT*)right,
+                  (AT*)out);
+    return launch_status();
+}
+
 }  // namespace
 
 SHISO_API int shiso_norm_into(float* residual, const void* y, int act_dtype, const float* w, void* out, int tokens, int hidden, float eps,
@@ -183,4 +289,18 @@ SHISO_API int shiso_polynorm(const void* z, long long z_ld, int act_dtype, const
     else
         return SHISO_ERR_DTYPE;
     return launch_status();
+}
+
+// left, right [T, hidden] in the activation type; weights float [hidden].  out_rows: T, or the length of `rows`.
+SHISO_API int shiso_normed_pair(const void* left, const void* right, int act_dtype, const float* wa, const float* wb, float scale,
+                                float pair_eps, float* residual, const int* rows, const float* w, float eps, void* out, float* sum,
+                                int out_rows, int hidden, cudaStream_t stream) {
+    if (out_rows <= 0) return SHISO_OK;
+    if (hidden <= 0 || hidden > 50 * 1024) return SHISO_ERR_SHAPE;
+    if (residual ? (!w || !out) : !sum) return SHISO_ERR_UNSUPPORTED;
+    const NormedPairArgs a = {residual, rows, wa, wb, w, sum, hidden, scale, pair_eps, eps};
+    const bool wide = hidden % 8 == 0 && aligned16(left, right, residual, out) && aligned16(wa, wb, w, sum);
+    if (act_dtype == SHISO_F32) return launch_normed_pair<float>(a, left, right, out, out_rows, wide, stream);
+    if (act_dtype == SHISO_BF16) return launch_normed_pair<__nv_bfloat16>(a, left, right, out, out_rows, wide, stream);
+    return SHISO_ERR_DTYPE;
 }

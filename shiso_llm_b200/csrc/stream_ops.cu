@@ -9,9 +9,13 @@
 //                      of gelu(g) u, or min(g, L) sigmoid(1.702 min(g, L)) (clamp(u, -L, L) + 1).
 // joined_norm_store:   rows [q | k | (v) | ..]: one RMS norm over all query columns together and one
 //                      over all key columns, each with a weight per column; the queries times a
-//                      temperature 1 + coef * ln(floor((p + 1) / every) + 1) of the row's position p,
-//                      written back in place; normed keys to the paged key cache; to the value cache
-//                      the value columns, or (values_from_keys) the key columns as they came.
+//                      temperature 1 + coef * ln(floor((p + 1) / every) + 1) of the row's position p;
+//                      both then rotated head by head (half-split pairs over the first rotary_dim
+//                      entries) where an encoding is given; queries written back in place, keys to
+//                      the paged key cache; to the value cache the value columns, or
+//                      (values_from_keys) the key columns as they came.
+// stream_concat:       out[t] = [residual[t] + up to two blocks of rows | first[t]], in the product's
+//                      input type: what a projection of the stream and the embedding's rows reads.
 //
 // Everything is evaluated in float with the library's tanhf, expf and logf, whatever the row type.
 #include "common.cuh"
@@ -176,6 +180,64 @@ SHISO_API int shiso_stream_add(const float* residual, float* out, const void* d0
     return launch_status();
 }
 
+// --------------------------------------------------------------------------- the stream beside the first rows
+
+struct StreamConcatArgs {
+    const float *residual, *first;
+    const void* d[2];
+    int dtype[2];
+    int tokens, hidden;
+};
+
+// A thread per N neighbouring columns of the output rows [2 * hidden].
+template <typename AT, int N>
+__global__ void __launch_bounds__(256) stream_concat_kernel(const StreamConcatArgs a, AT* __restrict__ out) {
+    pdl_begin();
+    const int per_row = 2 * a.hidden / N;
+    const long long i = (long long)blockIdx.x * blockDim.x + threadIdx.x;
+    if (i >= (long long)a.tokens * per_row) return;
+    const int t = (int)(i / per_row), c = (int)(i % per_row) * N;
+    float x[N];
+    if (c >= a.hidden) {
+        load_n<N>(a.first + (size_t)t * a.hidden + c - a.hidden, x);
+    } else {
+        const size_t at = (size_t)t * a.hidden + c;
+        load_n<N>(a.residual + at, x);
+#pragma unroll
+        for (int j = 0; j < 2; ++j) {
+            if (!a.d[j]) continue;
+            float d[N];
+            if (a.dtype[j] == SHISO_F32) load_n<N>((const float*)a.d[j] + at, d);
+            else load_n<N>((const __nv_bfloat16*)a.d[j] + at, d);
+#pragma unroll
+            for (int e = 0; e < N; ++e) x[e] += d[e];
+        }
+    }
+    store_n<N>(out + (size_t)t * 2 * a.hidden + c, x);
+}
+
+SHISO_API int shiso_stream_concat(const float* residual, const void* d0, int d0_dtype, const void* d1, int d1_dtype, const float* first,
+                                  void* out, int out_dtype, int tokens, int hidden, cudaStream_t stream) {
+    if (tokens <= 0 || hidden <= 0) return SHISO_OK;
+    StreamConcatArgs a = {residual, first, {d0, d1}, {d0_dtype, d1_dtype}, tokens, hidden};
+    for (int j = 0; j < 2; ++j)
+        if (a.d[j] && a.dtype[j] != SHISO_F32 && a.dtype[j] != SHISO_BF16) return SHISO_ERR_DTYPE;
+    const bool aligned = ((((uintptr_t)residual) | ((uintptr_t)first) | ((uintptr_t)d0) | ((uintptr_t)d1) | ((uintptr_t)out)) & 15) == 0;
+    const int n = !aligned ? 1 : hidden % 8 == 0 ? 8 : hidden % 4 == 0 ? 4 : 1;
+    const unsigned blocks = ceil_div_u((long long)tokens * (2 * hidden / n), 256);
+#define CONCAT_GO(AT)                                                                                  \
+    {                                                                                                  \
+        if (n == 8) launch_kernel(stream_concat_kernel<AT, 8>, blocks, 256, 0, stream, a, (AT*)out);   \
+        else if (n == 4) launch_kernel(stream_concat_kernel<AT, 4>, blocks, 256, 0, stream, a, (AT*)out); \
+        else launch_kernel(stream_concat_kernel<AT, 1>, blocks, 256, 0, stream, a, (AT*)out);          \
+    }
+    if (out_dtype == SHISO_F32) CONCAT_GO(float)
+    else if (out_dtype == SHISO_BF16) CONCAT_GO(__nv_bfloat16)
+    else return SHISO_ERR_DTYPE;
+#undef CONCAT_GO
+    return launch_status();
+}
+
 // --------------------------------------------------------------------------- gated pairs
 
 template <typename AT>
@@ -250,6 +312,48 @@ SHISO_API int shiso_gate_rows(void* x, long long x_ld, const void* gate, long lo
 
 // --------------------------------------------------------------------------- heads normalised together
 
+#define JOINED_MAX_PAIRS 128  // rotation pairs of a head
+
+struct Rotation {
+    const float* inv_freq;  // [dims / 2]
+    int head_dim, dims;     // dims = 0: nothing turns
+};
+
+// dst[h] = rotate(src[h] * inv * w[h]) for the heads of one row's columns; cosines and sines of the
+// row's position in shared memory.  A thread takes N columns and their partners half a rotation away,
+// or N columns behind the rotated ones.
+template <typename AT, int N>
+__device__ __forceinline__ void norm_rotate_columns(const AT* src, AT* dst, const float* __restrict__ w, float inv, int cols,
+                                                    const Rotation& rot, const float* cs, const float* sn) {
+    const int half = rot.dims / 2, turning = half / N, per_head = rot.head_dim / N - turning;
+    const int items = cols / rot.head_dim * per_head;
+    for (int i = threadIdx.x; i < items; i += blockDim.x) {
+        const int head = i / per_head, j = i % per_head;
+        const int at = head * rot.head_dim + (j < turning ? j * N : rot.dims + (j - turning) * N);
+        float u[N], wu[N];
+        load_n<N>(src + at, u);
+        load_n<N>(w + at, wu);
+#pragma unroll
+        for (int e = 0; e < N; ++e) u[e] = u[e] * inv * wu[e];
+        if (j < turning) {
+            float v[N], x[N];
+            load_n<N>(src + at + half, v);
+            load_n<N>(w + at + half, wu);
+#pragma unroll
+            for (int e = 0; e < N; ++e) {
+                const float c = cs[j * N + e], s = sn[j * N + e];
+                v[e] = v[e] * inv * wu[e];
+                x[e] = u[e] * c - v[e] * s;
+                v[e] = v[e] * c + u[e] * s;
+            }
+            store_n<N>(dst + at, x);
+            store_n<N>(dst + at + half, v);
+        } else {
+            store_n<N>(dst + at, u);
+        }
+    }
+}
+
 // One block per row.  Columns [0, q_cols) are the queries, [q_cols, q_cols + k_cols) the keys,
 // v_cols columns from v_col on the values (v_col = q_cols when the values are the keys as they came).
 // A thread takes N neighbouring columns at a time (N > 1: every extent and stride is a multiple of N
@@ -259,15 +363,17 @@ __global__ void __launch_bounds__(256)
 joined_norm_store_kernel(AT* __restrict__ proj, long long ld, int q_cols, int k_cols, int v_col, int v_cols, const float* __restrict__ q_w,
                          const float* __restrict__ k_w, const int* __restrict__ positions, const int* __restrict__ seq_of_token,
                          const int* __restrict__ table, int table_width, AT* __restrict__ k_cache, AT* __restrict__ v_cache,
-                         int page_size, float eps, float temp_coef, int temp_every) {
+                         int page_size, float eps, float temp_coef, int temp_every, const Rotation rot) {
     pdl_begin();
     __shared__ float scratch[33];
+    __shared__ float cs[JOINED_MAX_PAIRS], sn[JOINED_MAX_PAIRS];
     const int t = blockIdx.x;
     AT* row = proj + (size_t)t * ld;
     const int pos = positions[t];
     const int first = threadIdx.x * N, stride = blockDim.x * N;
     float v[N], w[N];
     float sq = 0.0f, sk = 0.0f;
+    for (int i = threadIdx.x; i < rot.dims / 2; i += blockDim.x) sincosf((float)pos * rot.inv_freq[i], &sn[i], &cs[i]);  // (a barrier follows, in block_sum)
     for (int i = first; i < q_cols; i += stride) {
         load_n<N>(row + i, v);
 #pragma unroll
@@ -286,17 +392,25 @@ joined_norm_store_kernel(AT* __restrict__ proj, long long ld, int q_cols, int k_
         const size_t at = (size_t)page * page_size + pos % page_size;
         AT* k_dst = k_cache + at * k_cols;
         AT* v_dst = v_cache + at * v_cols;
-        for (int i = first; i < k_cols; i += stride) {
-            load_n<N>(row + q_cols + i, v);
-            load_n<N>(k_w + i, w);
+        if (rot.dims > 0) {
+            norm_rotate_columns<AT, N>(row + q_cols, k_dst, k_w, k_inv, k_cols, rot, cs, sn);
+        } else {
+            for (int i = first; i < k_cols; i += stride) {
+                load_n<N>(row + q_cols + i, v);
+                load_n<N>(k_w + i, w);
 #pragma unroll
-            for (int e = 0; e < N; ++e) v[e] = v[e] * k_inv * w[e];
-            store_n<N>(k_dst + i, v);
+                for (int e = 0; e < N; ++e) v[e] = v[e] * k_inv * w[e];
+                store_n<N>(k_dst + i, v);
+            }
         }
         for (int i = first; i < v_cols; i += stride) {  // the values as they stand: a copy
             load_n<N>(row + v_col + i, v);
             store_n<N>(v_dst + i, v);
         }
+    }
+    if (rot.dims > 0) {
+        norm_rotate_columns<AT, N>(row, row, q_w, q_inv, q_cols, rot, cs, sn);
+        return;
     }
     for (int i = first; i < q_cols; i += stride) {
         load_n<N>(row + i, v);
@@ -310,16 +424,21 @@ joined_norm_store_kernel(AT* __restrict__ proj, long long ld, int q_cols, int k_
 SHISO_API int shiso_joined_norm_store(void* proj, long long ld, int act_dtype, int q_cols, int k_cols, int v_col, int v_cols,
                                       const float* q_w, const float* k_w, const int* positions, const int* seq_of_token,
                                       const int* table, int table_width, void* k_cache, void* v_cache, int tokens, int page_size,
-                                      float eps, float temp_coef, int temp_every, cudaStream_t stream) {
+                                      float eps, float temp_coef, int temp_every, const float* inv_freq, int head_dim,
+                                      int rotary_dim, cudaStream_t stream) {
     if (tokens <= 0) return SHISO_OK;
     if (q_cols <= 0 || k_cols <= 0 || v_cols <= 0 || v_col < q_cols || page_size <= 0 || temp_every < 0) return SHISO_ERR_SHAPE;
+    if (rotary_dim < 0 || rotary_dim % 2 || rotary_dim / 2 > JOINED_MAX_PAIRS) return SHISO_ERR_SHAPE;
+    if (rotary_dim > 0 && (!inv_freq || head_dim < rotary_dim || q_cols % head_dim || k_cols % head_dim)) return SHISO_ERR_SHAPE;
+    const Rotation rot = {inv_freq, head_dim, rotary_dim};
     const int n = act_dtype == SHISO_BF16 ? 8 : 4;
     const bool wide = q_cols % n == 0 && k_cols % n == 0 && v_col % n == 0 && v_cols % n == 0 && ld % n == 0 &&
+                      (rotary_dim == 0 || (head_dim % n == 0 && rotary_dim % (2 * n) == 0)) &&
                       ((((uintptr_t)proj) | ((uintptr_t)q_w) | ((uintptr_t)k_w) | ((uintptr_t)k_cache) | ((uintptr_t)v_cache)) & 15) == 0;
     const int threads = q_cols >= (wide ? 1024 * n / 2 : 1024) ? 256 : 128;
 #define JOINED_GO(AT, N)                                                                                                       \
     launch_kernel(joined_norm_store_kernel<AT, N>, tokens, threads, 0, stream, (AT*)proj, ld, q_cols, k_cols, v_col, v_cols, q_w, k_w, \
-                  positions, seq_of_token, table, table_width, (AT*)k_cache, (AT*)v_cache, page_size, eps, temp_coef, temp_every)
+                  positions, seq_of_token, table, table_width, (AT*)k_cache, (AT*)v_cache, page_size, eps, temp_coef, temp_every, rot)
     if (act_dtype == SHISO_F32) {
         if (wide) JOINED_GO(float, 4);
         else JOINED_GO(float, 1);

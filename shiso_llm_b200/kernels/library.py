@@ -68,9 +68,9 @@ _SIGNATURES = {
     "shiso_pool_kv": [P, P, I, P, P, P, P, I, P, P, I, I, I, I, I, I, P],
     "shiso_pooled_window_attention": [P, LL, I, P, P, P, P, P, P, I, P, P, P, LL, P, I, I, I, I, I, I, F, I, I, F, P],
     "shiso_prefill_attention_tc_open": [P, LL, P, P, P, I, P, P, P, LL, P, F, I, I, I, I, I, I, LL, F, I, P],
-    "shiso_prefill_attention_tc_kept": [P, LL, P, P, P, I, P, P, P, LL, I, I, I, I, I, I, LL, F, I, I, P],
+    "shiso_prefill_attention_tc_kept": [P, LL, P, P, P, I, P, P, P, LL, I, I, I, I, I, I, LL, F, I, I, P, P],
     "shiso_decode_attention_from_qkv_kept": [P, P, P, P, F, P, P, P, I, P, P, P, I, I, I, I, I, LL, F, I, I, I, I, P],
-    "shiso_decode_attention_fused_kept": [P, LL, P, P, P, I, P, P, P, I, I, I, I, I, LL, F, I, I, I, P],
+    "shiso_decode_attention_fused_kept": [P, LL, P, P, P, I, P, P, P, I, I, I, I, I, LL, F, I, I, I, P, P],
     "shiso_add_layernorm": [P, P, P, P, P, P, I, I, I, F, P],
     "shiso_group_rmsnorm": [P, I, LL, P, LL, P, P, I, I, I, I, I, F, P],
     "shiso_causal_conv": [P, LL, I, P, P, P, LL, P, P, P, P, I, I, I, I, I, P],
@@ -85,9 +85,9 @@ _SIGNATURES = {
     "shiso_latent_prefill_supported": [I, I],
     "shiso_latent_prefill": [P, P, P, I, P, P, P, I, I, I, I, I, I, F, P],
     "shiso_head_prepare_store": [P, LL, I, I, I, I, P, P, P, P, P, P, I, P, P, I, I, I, I, I, I, I, F, F, I, I, P],
-    "shiso_masked_attention": [P, LL, I, P, P, P, I, P, P, P, LL, P, LL, P, I, I, I, I, I, I, F, F, I, I, I, I, I, P, I, P],
+    "shiso_masked_attention": [P, LL, I, P, P, P, I, P, P, P, LL, P, LL, P, I, I, I, I, I, I, F, F, I, I, I, I, I, P, I, P, P],
     "shiso_masked_attention_tiles_supported": [I, I],
-    "shiso_masked_attention_tiles": [P, LL, P, P, P, I, P, P, P, LL, P, LL, P, I, I, I, I, I, I, I, F, F, I, I, I, I, I, P],
+    "shiso_masked_attention_tiles": [P, LL, P, P, P, I, P, P, P, LL, P, LL, P, I, I, I, I, I, I, I, F, F, I, I, I, I, I, P, P],
     "shiso_norm_into": [P, P, I, P, P, I, I, F, P],
     "shiso_polynorm": [P, LL, I, P, P, I, I, F, P],
     "shiso_gemm_stream_glu": [P, P, P, I, I, I, I, I, F, I, P],
@@ -99,7 +99,11 @@ _SIGNATURES = {
     "shiso_add_dyt": [P, P, P, P, P, P, F, P, I, I, I, P],
     "shiso_stream_add": [P, P, P, I, P, I, P, I, P, I, I, P],
     "shiso_glu_act": [P, P, I, I, I, I, F, P],
-    "shiso_joined_norm_store": [P, LL, I, I, I, I, I, P, P, P, P, P, I, P, P, I, I, F, F, I, P],
+    "shiso_joined_norm_store": [P, LL, I, I, I, I, I, P, P, P, P, P, I, P, P, I, I, F, F, I, P, I, I, P],
+    "shiso_stream_concat": [P, P, I, P, I, P, P, I, I, I, P],
+    "shiso_normed_pair": [P, P, I, P, P, F, F, P, P, P, F, P, P, I, I, P],
+    "shiso_delta_rule": [P, P, P, P, P, LL, LL, LL, LL, LL, I, P, P, P, LL, P, P, P, I, I, I, I, I, I, F, F, I, P],
+    "shiso_delta_output": [P, P, LL, I, P, P, LL, I, I, I, F, P],
 }
 
 

@@ -221,6 +221,29 @@ def stream_add(residual, deltas, vector, in_place=True):
     return out
 
 
+def stream_concat(residual, deltas, first, out_dtype):
+    """``[residual + sum(deltas) | first]``, rows ``[T, 2 H]`` of ``out_dtype``: ``residual`` and ``first``
+    float32 ``[T, H]``, up to two blocks of rows ``deltas`` (float32 or bfloat16 each)."""
+    _check(residual, "residual", torch.float32, 2)
+    _check(first, "first rows", torch.float32, 2)
+    tokens, hidden = residual.shape
+    deltas = tuple(deltas)
+    if len(deltas) > 2:
+        raise KernelError(f"{len(deltas)} blocks of rows to add; the kernel takes two")
+    for d in (first, *deltas):
+        _check(d, "rows", None, 2)
+        if d.shape != residual.shape:
+            raise KernelError(f"rows of {tuple(d.shape)} beside a residual of {tuple(residual.shape)}")
+    out = torch.empty((tokens, 2 * hidden), dtype=out_dtype, device=residual.device)
+    d = list(deltas) + [None] * (2 - len(deltas))
+    status = library().shiso_stream_concat(
+        _ptr(residual), _ptr(d[0]), _code(d[0]) if d[0] is not None else 0, _ptr(d[1]), _code(d[1]) if d[1] is not None else 0,
+        _ptr(first), _ptr(out), _code(out), tokens, hidden, _stream(),
+    )
+    _done(status, "stream_concat", shape=(tokens, hidden))
+    return out
+
+
 def add_dyt(residual, deltas, alpha, w, b, out_dtype, rows=None):
     """``tanh(alpha * x) * w + b`` of ``x = residual + sum(deltas)``: ``residual`` float32 ``[T, H]``,
     up to two ``deltas`` ``[T, H]`` in the output type.  Without ``rows`` the sum is stored back into
@@ -1308,11 +1331,12 @@ def gate_rows(x, gate):
 
 
 def joined_norm_store(proj, heads, kv_heads, dim, vdim, q_w, k_w, eps, q_temperature, values_from_keys, step, k_cache, v_cache,
-                      block_table, page_size):
+                      block_table, page_size, inv_freq=None, rotary_dim=0):
     """Prepares ``proj[T, heads*dim | kv_heads*dim | (kv_heads*vdim) | ...]`` in place: ONE RMS norm over
     all query columns together (weight ``q_w[heads*dim]``) and one over all key columns
     (``k_w[kv_heads*dim]``); the queries times ``1 + coef * ln(floor((p + 1) / every) + 1)`` at
-    position ``p`` when ``q_temperature = (coef, every)``.  Queries are written back where they
+    position ``p`` when ``q_temperature = (coef, every)``; behind the norm, the half-split rotation of
+    every head's first ``rotary_dim`` entries by ``position * inv_freq``.  Queries are written back where they
     stood, normed keys go to the paged key cache, and the value cache gets the value columns or,
     with ``values_from_keys``, the key columns as they came.  Returns the query columns."""
     act = proj.dtype
@@ -1331,26 +1355,31 @@ def joined_norm_store(proj, heads, kv_heads, dim, vdim, q_w, k_w, eps, q_tempera
     _paged(v_cache, "v cache", act, page_size)
     if k_cache.shape[2:] != (kv_heads, dim) or v_cache.shape[2:] != (kv_heads, vdim):
         raise KernelError(f"caches of shape {tuple(k_cache.shape)} / {tuple(v_cache.shape)} for {kv_heads} heads of {dim} / {vdim}")
+    if rotary_dim:
+        _check(inv_freq, "inv_freq", torch.float32, 1)
+        if inv_freq.shape[0] != rotary_dim // 2:
+            raise KernelError(f"inv_freq has {inv_freq.shape[0]} entries for a rotation over {rotary_dim}")
     coef, every = q_temperature if q_temperature is not None else (0.0, 0)
     status = library().shiso_joined_norm_store(
         proj.data_ptr(), ld, _CODES[act], q_cols, k_cols, q_cols if values_from_keys else q_cols + k_cols, v_cols, _ptr(q_w), _ptr(k_w),
         _ptr(step.positions), _ptr(step.seq_of_token), _ptr(block_table), block_table.shape[1], _ptr(k_cache), _ptr(v_cache),
-        proj.shape[0], page_size, float(eps), float(coef), int(every), _stream(),
+        proj.shape[0], page_size, float(eps), float(coef), int(every), _ptr(inv_freq) if rotary_dim else 0, dim, int(rotary_dim), _stream(),
     )
     _done(status, "joined_norm_store", shape=(proj.shape[0], heads + kv_heads, dim))
     return proj[:, :q_cols]
 
 
 def masked_attention(q, heads, k_cache, v_cache, block_table, page_size, scale, mask, size, keep_first, step, *, sigmoid=False,
-                     key_bias=None, softcap=None, gate=None, general=False, gate_per_element=False):
+                     key_bias=None, softcap=None, gate=None, general=False, gate_per_element=False, sink=None, out=None):
     """Attention of every row over the keys its mask shows: ``mask`` "window" (the last ``size``
     positions and the first ``keep_first`` of the sequence) or "chunk" (the positions of the row's
     own run of ``size``, counted from 0).  Scores ``(q . k) * scale``, capped as
     ``softcap * tanh(score / softcap)`` when a cap is given; weights a softmax, or with ``sigmoid``
-    one ``sigmoid(score + key_bias[head])`` per key, not normalised.  ``gate[T, heads]`` (logits)
+    one ``sigmoid(score + key_bias[head])`` per key, not normalised.  ``sink`` (float32 ``[heads]``, softmax
+    only): ``exp(sink[head])`` joins a head's denominator, with no key and no value.  ``gate[T, heads]`` (logits)
     multiplies each head's output by its sigmoid; with ``gate_per_element`` it is ``[T, heads * vdim]``
     and every output entry has a gate of its own.  ``q`` and ``gate`` may be column ranges.
-    Returns ``[T, heads * vdim]``.  bfloat16 steps that hold prompt portions take the tiled
+    Returns ``[T, heads * vdim]`` (``out``, where rows to write are given).  bfloat16 steps that hold prompt portions take the tiled
     tensor-core kernel (key sizes in multiples of 16 up to 256, value sizes up to 128); steps of
     single tokens, float32 and other sizes take the general kernel, as does ``general=True``
     (tests compare the routes)."""
@@ -1366,10 +1395,19 @@ def masked_attention(q, heads, k_cache, v_cache, block_table, page_size, scale, 
         _check(key_bias, "key bias", torch.float32, 1)
         if key_bias.shape[0] != heads:
             raise KernelError(f"key bias has {key_bias.shape[0]} entries for {heads} heads")
+    if sink is not None:
+        _check(sink, "sink", torch.float32, 1)
+        if sink.shape[0] != heads or sigmoid:
+            raise KernelError(f"{sink.shape[0]} sinks for {heads} heads under {'sigmoid weights' if sigmoid else 'a softmax'}")
     gate_ld = _rows(gate, "gate", act, heads * (vdim if gate_per_element else 1)) if gate is not None else 0
     wide = int(bool(gate is not None and gate_per_element))
     tokens = q.shape[0]
-    out = torch.empty((tokens, heads * vdim), dtype=act, device=q.device)
+    if out is None:
+        out = torch.empty((tokens, heads * vdim), dtype=act, device=q.device)
+    else:
+        _check(out, "out", act, 2)
+        if out.shape != (tokens, heads * vdim):
+            raise KernelError(f"out of {tuple(out.shape)} for {tokens} rows of {heads} heads of {vdim}")
     lib = library()
     what = f"({mask}, {'sigmoid' if sigmoid else 'softmax'})"
     # A softmax over a window (with or without kept first tokens), heads of 64, no cap and no gate is
@@ -1388,7 +1426,7 @@ def masked_attention(q, heads, k_cache, v_cache, block_table, page_size, scale, 
         status = lib.shiso_decode_attention_fused_kept(
             q.data_ptr(), q_ld, _ptr(k_cache), _ptr(v_cache), _ptr(block_table), block_table.shape[1], _ptr(step.positions),
             _ptr(step.seq_of_token), _ptr(out), tokens, heads, kv_heads, dim, page_size, k_cache.shape[0], float(scale),
-            0 if size >= NO_WINDOW else int(size), int(keep_first), splits, _stream(),
+            0 if size >= NO_WINDOW else int(size), int(keep_first), splits, _ptr(sink), _stream(),
         )
         _done(status, f"decode_attention (fused) {what}", shape=(tokens, heads, dim))
         return gate_rows(out, gate) if wide else out
@@ -1405,7 +1443,7 @@ def masked_attention(q, heads, k_cache, v_cache, block_table, page_size, scale, 
         status = lib.shiso_prefill_attention_tc_kept(
             q.data_ptr(), q_ld, _ptr(k_cache), _ptr(v_cache), _ptr(block_table), block_table.shape[1], _ptr(step.q_start),
             _ptr(step.start_pos), _ptr(out), heads * vdim, tokens, step.num_seqs, tiles, heads, kv_heads, page_size,
-            k_cache.shape[0], float(scale), 0 if size >= NO_WINDOW else int(size), int(keep_first), _stream(),
+            k_cache.shape[0], float(scale), 0 if size >= NO_WINDOW else int(size), int(keep_first), _ptr(sink), _stream(),
         )
         _done(status, f"prefill_attention (tcgen05) {what}", shape=(tokens, heads, dim))
         return gate_rows(out, gate) if wide else out
@@ -1422,7 +1460,7 @@ def masked_attention(q, heads, k_cache, v_cache, block_table, page_size, scale, 
             q.data_ptr(), q_ld, _ptr(k_cache), _ptr(v_cache), _ptr(block_table), block_table.shape[1], _ptr(step.q_start),
             _ptr(step.start_pos), _ptr(out), heads * vdim, gate.data_ptr() if gate is not None else 0, gate_ld, _ptr(key_bias),
             step.num_seqs, tiles, heads, kv_heads, dim, vdim, page_size, float(scale), float(softcap or 0.0), _MASKS[mask], int(size),
-            int(keep_first), int(bool(sigmoid)), wide, _stream(),
+            int(keep_first), int(bool(sigmoid)), wide, _ptr(sink), _stream(),
         )
         _done(status, f"masked_attention_tiles {what}", shape=(tokens, heads, dim))
         return out
@@ -1436,7 +1474,7 @@ def masked_attention(q, heads, k_cache, v_cache, block_table, page_size, scale, 
         q.data_ptr(), q_ld, _CODES[act], _ptr(k_cache), _ptr(v_cache), _ptr(block_table), block_table.shape[1], _ptr(step.positions),
         _ptr(step.seq_of_token), _ptr(out), heads * vdim, gate.data_ptr() if gate is not None else 0, gate_ld, _ptr(key_bias),
         tokens, heads, kv_heads, dim, vdim, page_size, float(scale), float(softcap or 0.0), _MASKS[mask], int(size), int(keep_first),
-        int(bool(sigmoid)), splits, _ptr(scratch), wide, _stream(),
+        int(bool(sigmoid)), splits, _ptr(scratch), wide, _ptr(sink), _stream(),
     )
     _done(status, f"masked_attention {what}", 2 if splits > 1 else 1, shape=(tokens, heads, dim))
     return out
@@ -1460,6 +1498,46 @@ def norm_into(residual, y, w, eps, want_rows=True):
     if not want_rows:
         return None
     return residual if out is None else out
+
+
+def _normed_pair(left, right, wa, wb, scale, pair_eps, residual, rows, w, eps, out, total, out_rows):
+    for name, t in (("left", left), ("right", right)):
+        _check(t, f"{name} rows", left.dtype, 2)
+        if t.shape != left.shape:
+            raise KernelError(f"branches of {tuple(left.shape)} and {tuple(right.shape)}")
+    tokens, hidden = left.shape
+    for t in (wa, wb) if w is None else (wa, wb, w):
+        _check(t, "norm weight", torch.float32, 1)
+        if t.shape[0] != hidden:
+            raise KernelError(f"a norm weight of {t.shape[0]} entries for rows of {hidden}")
+    if residual is not None:
+        _check(residual, "residual", torch.float32, 2)
+        if residual.shape != left.shape:
+            raise KernelError(f"branches of {tuple(left.shape)} beside a residual of {tuple(residual.shape)}")
+    status = library().shiso_normed_pair(
+        _ptr(left), _ptr(right), _code(left), _ptr(wa), _ptr(wb), float(scale), float(pair_eps), _ptr(residual), _ptr(rows), _ptr(w), float(eps),
+        _ptr(out), _ptr(total), out_rows, hidden, _stream(),
+    )
+    _done(status, "normed_pair" if residual is None else "add normed_pair + rmsnorm", shape=(out_rows, hidden))
+
+
+def normed_pair(left, right, wa, wb, scale, pair_eps):
+    """``scale * (norm(left) * wa + norm(right) * wb)`` with RMS norms over whole rows: float32 ``[T, H]``."""
+    total = torch.empty(left.shape, dtype=torch.float32, device=left.device)
+    _normed_pair(left, right, wa, wb, scale, pair_eps, None, None, None, 0.0, None, total, left.shape[0])
+    return total
+
+
+def add_normed_pair_rmsnorm(residual, left, right, wa, wb, scale, pair_eps, w, eps, rows=None):
+    """``residual += normed_pair(...)`` (float32, in place) and the RMS norm of the sum, in the branches'
+    type.  With ``rows`` (int32) only those rows are summed and normalised and the residual stays."""
+    out_rows = residual.shape[0]
+    if rows is not None:
+        _check(rows, "rows", torch.int32, 1)
+        out_rows = rows.shape[0]
+    out = torch.empty((out_rows, residual.shape[1]), dtype=left.dtype, device=residual.device)
+    _normed_pair(left, right, wa, wb, scale, pair_eps, residual, rows, w, eps, out, None, out_rows)
+    return out
 
 
 def polynorm(z, coefficients, eps, out_dtype):
@@ -1604,6 +1682,55 @@ def state_recurrence(q, k, v, state, step, heads, groups, dim, vdim, *, silu_inp
     return out
 
 
+def delta_rule(q, k, v, b, a, dt_bias, a_log, state, step, heads, groups, dim, vdim, q_scale, unit_eps):
+    """The gated delta rule over each sequence's rows in order, with a state ``S[dim, vdim]`` per head
+    (``state``, float32 ``[slots, heads, dim, vdim]``): ``S <- g S``, ``u = beta (v - S^T k)``,
+    ``S <- S + k u^T``, ``o = S^T q``.  ``q, k [T, groups * dim]`` are brought to unit length per head
+    (``x / sqrt(sum x^2 + unit_eps)``, q times ``q_scale`` too), head ``h`` reading group
+    ``h // (heads / groups)``; ``v [T, heads * vdim]``; ``beta = sigmoid(b)``, ``g = exp(-exp(a_log)
+    softplus(a + dt_bias))`` from ``b, a [T, heads]``.  All may be column ranges.  Returns float32
+    ``[T, heads * vdim]``."""
+    act = q.dtype
+    tokens = q.shape[0]
+    q_ld, k_ld = _rows(q, "q", act, groups * dim), _rows(k, "k", act, groups * dim)
+    v_ld = _rows(v, "v", act, heads * vdim)
+    b_ld, a_ld = _rows(b, "b", act, heads), _rows(a, "a", act, heads)
+    if state.shape[1:] != (heads, dim, vdim):
+        raise KernelError(f"a state of shape {tuple(state.shape)} for {heads} heads of {dim} x {vdim}")
+    stride = _slot_rows(state, "recurrent state", torch.float32)
+    for name, t in (("dt bias", dt_bias), ("a_log", a_log)):
+        _check(t, name, torch.float32, 1)
+        if t.shape[0] != heads:
+            raise KernelError(f"{name} has {t.shape[0]} entries for {heads} heads")
+    out = torch.empty((tokens, heads * vdim), dtype=torch.float32, device=q.device)
+    status = library().shiso_delta_rule(
+        q.data_ptr(), k.data_ptr(), v.data_ptr(), b.data_ptr(), a.data_ptr(), q_ld, k_ld, v_ld, b_ld, a_ld, _CODES[act], _ptr(dt_bias),
+        _ptr(a_log), state.data_ptr(), stride, _ptr(step.q_start), _ptr(step.state_slots), _ptr(out), tokens, step.num_seqs, heads,
+        groups, dim, vdim, float(q_scale), float(unit_eps), _sm_count(), _stream(),
+    )
+    _done(status, "delta_rule", shape=(tokens, heads, dim, vdim))
+    return out
+
+
+def delta_output(x, gate, weight, heads, eps, out):
+    """``out[t, h] = x[t, h] / rms(x[t, h]) * weight * silu(gate[t, h])`` per head: ``x`` float32
+    ``[T, heads * vdim]``, ``weight`` float32 ``[vdim]``, ``gate`` and ``out`` ``[T, heads * vdim]`` of one type
+    (column ranges may be given)."""
+    _check(x, "x", torch.float32, 2)
+    _check(weight, "norm weight", torch.float32, 1)
+    tokens, width = x.shape
+    gate_ld = _rows(gate, "gate", out.dtype, width)
+    out_ld = _rows(out, "out", out.dtype, width)
+    vdim = weight.shape[0]
+    if width != heads * vdim or gate.shape[0] != tokens or out.shape[0] != tokens:
+        raise KernelError(f"rows of {width} for {heads} heads of {vdim}")
+    status = library().shiso_delta_output(
+        _ptr(x), gate.data_ptr(), gate_ld, _code(out), _ptr(weight), out.data_ptr(), out_ld, tokens, heads, vdim, float(eps), _stream(),
+    )
+    _done(status, "delta_output", shape=(tokens, heads, vdim))
+    return out
+
+
 # --------------------------------------------------------------------------- latent attention
 
 
@@ -1735,12 +1862,18 @@ def latent_attention(q_lat, rank, k_cache, block_table, page_size, scale, step, 
 # --------------------------------------------------------------------------- mixture of experts
 
 
-def moe_route(logits, top, group_count, group_keep, scale, sigmoid=False, renormalize=False, correction=None, renorm_eps=0.0):
+_ROUTE_SCORES = {"softmax": 0, "sigmoid": 1, "chosen_softmax": 2}
+
+
+def moe_route(logits, top, group_count, group_keep, scale, sigmoid=False, renormalize=False, correction=None, renorm_eps=0.0,
+              scores=None):
     """For every row of ``logits`` (float32 ``[T, E]``, a column range may be given): scores (softmax
     over all experts, or sigmoids), the ``top`` largest among the experts of the ``group_keep`` best
     of ``group_count`` groups of neighbours (a group's value is its largest), ranked by score +
     ``correction[e]`` where a correction (float32 ``[E]``) is given, and their weights: the scores
-    themselves (divided by their sum + ``renorm_eps`` with ``renormalize``) times ``scale``.  Returns
+    themselves (divided by their sum + ``renorm_eps`` with ``renormalize``) times ``scale``.
+    ``scores = "chosen_softmax"``: the logits themselves are ranked, and the weights are the softmax
+    over the chosen logits only, times ``scale``.  Returns
     ids int32 and weights float32, both ``[T, top]``, best first."""
     ld = _rows(logits, "router logits", torch.float32)
     tokens, experts = logits.shape
@@ -1752,22 +1885,25 @@ def moe_route(logits, top, group_count, group_keep, scale, sigmoid=False, renorm
     weights = torch.empty((tokens, top), dtype=torch.float32, device=logits.device)
     status = library().shiso_moe_route(
         logits.data_ptr(), ld, _ptr(correction), _ptr(ids), _ptr(weights), tokens, experts, int(top), int(group_count), int(group_keep),
-        float(scale), int(bool(sigmoid)), int(bool(renormalize)), float(renorm_eps), _stream(),
+        float(scale), _ROUTE_SCORES[scores or ("sigmoid" if sigmoid else "softmax")], int(bool(renormalize)), float(renorm_eps), _stream(),
     )
     _done(status, "moe_route", shape=(tokens, experts, top))
     return ids, weights
 
 
+UNGATED_RELU2 = "relu2"
 MOE_MAX_EXPERTS = 256  # router outputs the grouping kernels keep in shared memory
 
 
 def routed_experts(x, ids, weights, gate_up, down, extra=None, act="silu", limit=0.0, extra_gate=None, identity=0):
     """``out[t] = extra[t] + sum_j weights[t, j] * expert_{ids[t, j]}(x[t])`` with gated experts
     ``down[e] pair(gate x, up x)`` (``act`` / ``limit``: the pairs of ``glu_act``), ``gate_up[e] =
-    [gate; up]``: ``x[T, H]``, ``gate_up[E, 2F, H]``, ``down[E, H, F]``.  Ids ``E .. E + identity - 1`` are
+    [gate; up]``: ``x[T, H]``, ``gate_up[E, 2F, H]``, ``down[E, H, F]``; with ``act = "relu2"`` ungated
+    experts ``down[e] relu(up x)^2`` and ``gate_up[E, F, H]`` holds the up matrices.  Ids ``E .. E + identity - 1`` are
     identity experts: one adds ``weights[t, j] * x[t]``.  ``extra_gate`` (float32 ``[T, 1]``, a column
     range may be given) multiplies ``extra[t]`` by its sigmoid.  The (row, choice) pairs are grouped
     by expert on the device; nothing about the routing reaches the host."""
+    gated = act != UNGATED_RELU2
     _check(x, "x", None, 2)
     _check(ids, "expert ids", torch.int32, 2)
     _check(weights, "expert weights", torch.float32, 2)
@@ -1775,15 +1911,16 @@ def routed_experts(x, ids, weights, gate_up, down, extra=None, act="silu", limit
     _check(down, "down matrices", gate_up.dtype, 3)
     tokens, hidden = x.shape
     experts, two_ff, _ = gate_up.shape
+    ff = two_ff // 2 if gated else two_ff
     top = ids.shape[1]
-    if ids.shape != (tokens, top) or weights.shape != ids.shape or gate_up.shape[2] != hidden or down.shape != (experts, hidden, two_ff // 2):
+    if ids.shape != (tokens, top) or weights.shape != ids.shape or gate_up.shape[2] != hidden or down.shape != (experts, hidden, ff):
         raise KernelError("ids, weights or expert matrices of the wrong shape")
     if extra is not None:
         _check(extra, "extra", x.dtype, 2)
         if extra.shape != x.shape:
             raise KernelError(f"extra rows of {tuple(extra.shape)} beside {tuple(x.shape)}")
-    if act not in _GLU_ACTS:
-        raise KernelError(f"gated pair {act!r}: expected one of {sorted(_GLU_ACTS)}")
+    if gated and act not in _GLU_ACTS:
+        raise KernelError(f"gated pair {act!r}: expected one of {sorted(_GLU_ACTS)} or {UNGATED_RELU2!r}")
     gate_ld = 0
     if extra_gate is not None:
         if extra is None:
@@ -1791,7 +1928,7 @@ def routed_experts(x, ids, weights, gate_up, down, extra=None, act="silu", limit
         gate_ld = _rows(extra_gate, "extra gate", torch.float32, 1)
         if extra_gate.shape[0] != tokens:
             raise KernelError(f"{extra_gate.shape[0]} gates for {tokens} rows")
-    ff, total = two_ff // 2, tokens * top
+    total = tokens * top
     if identity < 0 or experts + identity > MOE_MAX_EXPERTS:
         raise KernelError(f"{experts} experts and {identity} identity experts; the grouping kernels take {MOE_MAX_EXPERTS} in all")
     ints = torch.empty((experts + identity + 3 * total,), dtype=torch.int32, device=x.device)
@@ -1801,7 +1938,7 @@ def routed_experts(x, ids, weights, gate_up, down, extra=None, act="silu", limit
     status = library().shiso_routed_experts(
         _ptr(x), _code(x), _ptr(ids), _ptr(weights), _ptr(gate_up), _ptr(down), _code(gate_up), _ptr(extra),
         extra_gate.data_ptr() if extra_gate is not None else 0, gate_ld, _ptr(out), _ptr(ints),
-        _ptr(mid), _ptr(y), tokens, hidden, ff, experts, int(identity), top, _GLU_ACTS[act], float(limit), _stream(),
+        _ptr(mid), _ptr(y), tokens, hidden, ff, experts, int(identity), top, _GLU_ACTS[act] if gated else 3, float(limit), _stream(),
     )
     _done(status, "routed_experts", 6, shape=(tokens, top, experts, ff, hidden))
     return out

@@ -201,6 +201,21 @@ class DeferredLinear:
         return self.ops.linear(self.x, self.w, self.out_dtype)
 
 
+class NormedPair:
+    """A mixer output that is not formed yet: ``scale * (norm(left) * left_w + norm(right) * right_w)``,
+    the RMS norms of two branches' rows over the model width (``eps`` inside the root).
+
+    The next norm of the stream adds it to the residual and normalises the sum in one kernel when
+    it can (``takes_pairs``: its ``add_apply`` is handed this object as the block output).
+    ``materialize()`` gives the float32 rows."""
+
+    def __init__(self, ops, left, right, left_w, right_w, scale: float, eps: float):
+        self.ops, self.left, self.right, self.left_w, self.right_w, self.scale, self.eps = ops, left, right, left_w, right_w, scale, eps
+
+    def materialize(self) -> torch.Tensor:
+        return self.ops.normed_pair(self.left, self.right, self.left_w, self.right_w, self.scale, self.eps)
+
+
 class DeferredNorm:
     """The normed rows a mixer or feed-forward is about to read, not computed yet:
     ``norm(residual + pending)`` of a stream.
@@ -338,6 +353,9 @@ class Stream:
             if not getattr(norm, "takes_several", False):
                 raise RuntimeError(f"{type(norm).__name__} adds one block output at a time, {len(delta)} are waiting")
             return norm.add_apply(self.residual, tuple(d.materialize() if isinstance(d, DeferredLinear) else d for d in delta))
+        if isinstance(delta, NormedPair) and not getattr(norm, "takes_pairs", False):
+            self.residual = norm.env.ops.stream_add(self.residual, (delta.materialize(),), None)
+            return norm.apply(self.residual)
         if isinstance(delta, DeferredLinear):
             fused = getattr(norm, "add_apply_linear", None)
             if fused is not None:
@@ -345,10 +363,12 @@ class Stream:
             delta = delta.materialize()
         return norm.add_apply(self.residual, delta)
 
-    def take_pending(self) -> Optional[torch.Tensor]:
+    def take_pending(self, norm: Optional[Norm] = None) -> Optional[torch.Tensor]:
         """The block output still waiting to be added, as a tensor (or None); a tuple of tensors
-        where a layer left several."""
+        where a layer left several.  A ``NormedPair`` stays one where ``norm`` says it takes those."""
         delta, self.pending = self.pending, None
+        if isinstance(delta, NormedPair):
+            return delta if norm is not None and getattr(norm, "takes_pairs", False) else delta.materialize()
         if isinstance(delta, tuple):
             return tuple(d.materialize() if isinstance(d, DeferredLinear) else d for d in delta)
         if isinstance(delta, DeferredLinear):

@@ -25,6 +25,7 @@ from .base import FEED_FORWARDS, DeferredLinear, FeedForward, project
 MAX_EXPERTS = 256  # what the routing kernel keeps of a token's scores in a warp's registers ...
 MAX_TOP = 16  # ... and how many choices it makes per token
 GLU_ACTIVATIONS = ("silu", "gelu_tanh", "swish_clamped")
+UNGATED_RELU2 = "relu2"  # experts without a gate: W_down relu(W_up x)^2
 
 
 @FEED_FORWARDS.register("swiglu")
@@ -144,6 +145,11 @@ class RoutedExperts(FeedForward):
     the shared feed-forward's output is multiplied by ``sigmoid(W_sg x)``, one number per token;
     its row rides on the router's product.
 
+    ``scores = "chosen_softmax"``: the logits themselves are ranked (``router_bias`` names a vector added to
+    them, for the choice and the weights alike), and a token's weights are the softmax over its chosen
+    logits only.  ``activation = "relu2"`` makes the experts ungated, ``W_down relu(W_up x)^2``, with names
+    ``up`` and ``down`` each.
+
     The expert matrices are stacked ``[experts, 2 ff, hidden]`` (gate over up) and
     ``[experts, hidden, ff]`` when bound; a step's (token, choice) pairs are grouped by expert
     on the device and each group runs as row tiles of one launch, so nothing about the routing
@@ -164,17 +170,20 @@ class RoutedExperts(FeedForward):
         self.renorm_eps = float(p.get("renorm_eps", 0.0))
         self.identity = int(p.get("identity", 0))
         self.correction_name = p.get("correction")
+        self.router_bias_name = p.get("router_bias")
         self.shared_gate_name = p.get("shared_gate")
         self.activation = p.get("activation", "silu")
         self.limit = float(p.get("limit") or 0.0)
-        if self.activation not in GLU_ACTIVATIONS or (self.activation == "swish_clamped" and self.limit <= 0.0):
-            raise UnsupportedShape("expert activation", (self.activation, self.limit), f"one of {GLU_ACTIVATIONS}; a clamped pair needs a positive limit")
+        known = self.activation in GLU_ACTIVATIONS or self.activation == UNGATED_RELU2
+        if not known or (self.activation == "swish_clamped" and self.limit <= 0.0):
+            raise UnsupportedShape("expert activation", (self.activation, self.limit), f"one of {GLU_ACTIVATIONS} or {UNGATED_RELU2!r}; a clamped pair needs a positive limit")
+        self.in_names = ("up",) if self.activation == UNGATED_RELU2 else ("gate", "up")
         if not 0 <= self.identity < self.experts:
             raise UnsupportedShape("identity experts", self.identity, f"fewer than the router's {self.experts} outputs")
         if self.shared_gate_name is not None and p.get("shared") is None:
             raise UnsupportedShape("shared_gate", self.shared_gate_name, "a gate on a shared feed-forward that is absent")
-        if self.scores not in ("softmax", "sigmoid"):
-            raise UnsupportedShape("router scores", self.scores, "expected 'softmax' or 'sigmoid'")
+        if self.scores not in ("softmax", "sigmoid", "chosen_softmax"):
+            raise UnsupportedShape("router scores", self.scores, "expected 'softmax', 'sigmoid' or 'chosen_softmax'")
         if not 0 < self.top <= self.experts or self.experts % self.group_count or not 0 < self.group_keep <= self.group_count:
             raise UnsupportedShape("router", (self.experts, self.top, self.group_count, self.group_keep), "top <= experts, groups must divide the experts, keep <= groups")
         if self.group_keep * (self.experts // self.group_count) < self.top:
@@ -186,7 +195,7 @@ class RoutedExperts(FeedForward):
         if len(self.expert_names) != self.experts - self.identity:
             raise ValueError(f"{len(self.expert_names)} sets of names for {self.experts - self.identity} experts with matrices")
         self.shared = FEED_FORWARDS.build(p["shared"], env) if p.get("shared") is not None else None
-        self.router = self.gate_up = self.down = self.correction = None
+        self.router = self.router_bias = self.gate_up = self.down = self.correction = None
 
     def sub_parts(self):
         return [self.shared] if self.shared is not None else []
@@ -194,12 +203,14 @@ class RoutedExperts(FeedForward):
     def tensor_specs(self):
         specs = [TensorSpec(self.router_name, (self.experts, self.hidden))]
         for names in self.expert_names:
-            specs += [TensorSpec(names["gate"], (self.inter, self.hidden)), TensorSpec(names["up"], (self.inter, self.hidden)),
-                      TensorSpec(names["down"], (self.hidden, self.inter))]
+            specs += [TensorSpec(names[k], (self.inter, self.hidden)) for k in self.in_names]
+            specs.append(TensorSpec(names["down"], (self.hidden, self.inter)))
         if self.shared is not None:
             specs += self.shared.tensor_specs()
         if self.correction_name is not None:
             specs.append(TensorSpec(self.correction_name, (self.experts,), VECTOR, NORMAL, init_std=0.02))
+        if self.router_bias_name is not None:
+            specs.append(TensorSpec(self.router_bias_name, (self.experts,), VECTOR, NORMAL, init_std=0.02))
         if self.shared_gate_name is not None:
             specs.append(TensorSpec(self.shared_gate_name, (1, self.hidden)))
         return specs
@@ -213,19 +224,24 @@ class RoutedExperts(FeedForward):
             # (rows up to a multiple of eight are zeros: the tensor-memory products for long portions take such matrices)
             pad = torch.zeros((-(self.experts + 1) % 8, self.hidden), dtype=gate.dtype, device=gate.device)
             self.router = torch.cat([self.router, gate, pad], dim=0).contiguous()
+        if self.router_bias_name is not None:  # for the router's rows; the gate's and the padding have none
+            bias = tensors[self.router_bias_name].to(torch.float32)
+            self.router_bias = torch.cat([bias, bias.new_zeros(self.router.shape[0] - self.experts)]).contiguous()
         self.correction = tensors[self.correction_name] if self.correction_name is not None else None
-        mats = [tensors[n[k]] for n in self.expert_names for k in ("gate", "up", "down")]
+        mats = [tensors[n[k]] for n in self.expert_names for k in (*self.in_names, "down")]
         wide = len({m.dtype for m in mats}) > 1
         pick = (lambda m: m.float()) if wide else (lambda m: m)
-        self.gate_up = torch.stack([torch.cat([pick(tensors[n["gate"]]), pick(tensors[n["up"]])], dim=0) for n in self.expert_names]).contiguous()
+        self.gate_up = torch.stack([torch.cat([pick(tensors[n[k]]) for k in self.in_names], dim=0) for n in self.expert_names]).contiguous()
         self.down = torch.stack([pick(tensors[n["down"]]) for n in self.expert_names]).contiguous()
         if self.shared is not None:
             self.shared.bind(tensors)
 
     def forward(self, x, step):
         ops = self.env.ops
-        logits = ops.linear(x, self.router, torch.float32)
+        logits = ops.linear(x, self.router, torch.float32, self.router_bias)
         more = {}
+        if self.scores == "chosen_softmax":
+            more["scores"] = self.scores
         if self.correction is not None:
             more["correction"] = self.correction
         if self.renorm_eps:

@@ -9,7 +9,7 @@ projected (bias included), before any norm, so ``vdim = dim``.  Then, per query 
     rotation, with one ``[dim]`` weight for the queries and one for the keys (shared by the
     heads) or, without names for them, no weight at all (a unit norm); or ``"joined"``: ONE RMS
     norm over all query heads' entries together and one over all key heads', with weights of
-    ``[heads * dim]`` and ``[kv_heads * dim]`` (no rotation goes with it);
+    ``[heads * dim]`` and ``[kv_heads * dim]``, taken before the rotation (if any);
   * the position encoding on the first ``rotary_dim`` entries (half-split pairs; cosine and sine
     times the encoding's ``magnitude``).
 
@@ -23,7 +23,8 @@ position ``i`` sees (``mask``):
     position 0 of the sequence wherever a prompt was cut;
   * ``{"kind": "causal"}``: every ``j <= i`` (a window that never ends; the cache keeps everything).
 
-``weights``: ``"softmax"`` over the visible keys, or ``"sigmoid"``: every visible key weighs
+``weights``: ``"softmax"`` over the visible keys - with ``sink``, a ``[heads]`` tensor, the denominator
+holds ``exp(sink[head])`` once more, a share that has no key and no value - or ``"sigmoid"``: every visible key weighs
 ``sigmoid(score + key_bias[head])`` and nothing is normalised.  ``gate`` names a ``[heads,
 hidden]`` matrix: head ``a``'s output is multiplied by ``sigmoid((W_g h)_a)``; with ``gate_per =
 "element"`` the matrix is ``[heads * vdim, hidden]`` and every entry of the concatenated heads has
@@ -32,7 +33,8 @@ a gate of its own.  Output: ``W_o`` on the concatenated heads.
 The projections are joined into one matrix ``[q | k | v | gate]`` when bound, so one product
 feeds the kernel that prepares the heads in place and stores keys and values.  The cache keeps
 the last ``size`` positions (a chunk never reaches further back than that) and, for a window
-that keeps first tokens, the pages that hold those.
+that keeps first tokens, the pages that hold those.  The mixer also serves as a branch of
+``parallel_mixer`` (without projection biases): it then reads its columns of the joint product.
 """
 
 from __future__ import annotations
@@ -52,7 +54,7 @@ EVERYTHING = 1 << 30  # the size of a window that never ends
 class MaskedAttention(Mixer):
     """``params``: ``hidden_size``, ``num_heads``, ``num_kv_heads``, ``head_dim``, ``v_head_dim``,
     ``scale``, ``mask``, ``weights``, optionally ``softcap``, ``head_norm`` (+ ``eps``, ``q_norm``,
-    ``k_norm``), ``position``, ``key_bias``, ``gate`` (+ ``gate_per``), ``values``, ``q_temperature``,
+    ``k_norm``), ``position``, ``key_bias``, ``sink``, ``gate`` (+ ``gate_per``), ``values``, ``q_temperature``,
     ``q_bias`` / ``k_bias`` / ``v_bias``, and the names ``q_proj``, ``k_proj``, ``v_proj``, ``out_proj``."""
 
     def __init__(self, spec, env):
@@ -104,8 +106,8 @@ class MaskedAttention(Mixer):
             raise UnsupportedShape("q_temperature", dict(temperature), "the positions are counted in runs of at least 1")
         self.position = POSITION_ENCODINGS.build(p.get("position") or PartSpec("none"), env, self.dim)
         joined = self.head_norm == "joined"
-        if joined and self.position.rotary()[1]:
-            raise UnsupportedShape("position", p["position"].kind, "the kernel of the joined norm does not rotate")
+        if joined and float(getattr(self.position, "magnitude", 1.0)) != 1.0:
+            raise UnsupportedShape("position", p["position"].kind, "the kernel of the joined norm rotates without a magnitude on cosine and sine")
         if (self.values == "keys" or self.q_temperature is not None) and not joined:
             raise UnsupportedShape("head_norm", self.head_norm, "values that are the keys and a query temperature come with the joined norm's kernel")
         if joined and (p.get("q_norm") is None or p.get("k_norm") is None):
@@ -113,11 +115,13 @@ class MaskedAttention(Mixer):
         if getattr(self.position, "interleaved", False):
             raise UnsupportedShape("position", p["position"].kind, "the kernel that prepares the heads rotates half-split pairs")
         self.names = {k: p.get(k) for k in ("q_proj", "k_proj", "v_proj", "out_proj", "q_bias", "k_bias", "v_bias", "q_norm", "k_norm",
-                                             "key_bias", "gate")}
+                                             "key_bias", "sink", "gate")}
         if self.names["key_bias"] is not None and self.weights != "sigmoid":
             raise UnsupportedShape("key_bias", self.names["key_bias"], "a bias per head on the scores changes nothing under a softmax")
+        if self.names["sink"] is not None and self.weights != "softmax":
+            raise UnsupportedShape("sink", self.names["sink"], "only a softmax has a denominator for it")
         self.in_matrix = self.in_bias = self.out_matrix = None
-        self.q_weight = self.k_weight = self.key_bias = None
+        self.q_weight = self.k_weight = self.key_bias = self.sink = None
 
     @property
     def q_cols(self):
@@ -130,6 +134,14 @@ class MaskedAttention(Mixer):
     @property
     def gate_cols(self):
         return self.heads * (self.vdim if self.gate_per == "element" else 1)
+
+    @property
+    def in_width(self):
+        return self.q_cols + self.kv_cols + (self.gate_cols if self.names["gate"] is not None else 0)
+
+    @property
+    def out_width(self):
+        return self.heads * self.vdim
 
     def sub_parts(self):
         return [self.position]
@@ -152,6 +164,8 @@ class MaskedAttention(Mixer):
                 specs.append(TensorSpec(n[key], (heads * self.dim if joined else self.dim,), VECTOR, ONES))
         if n["key_bias"] is not None:
             specs.append(TensorSpec(n["key_bias"], (self.heads,), VECTOR, ZEROS))
+        if n["sink"] is not None:
+            specs.append(TensorSpec(n["sink"], (self.heads,), VECTOR, NORMAL, init_std=1.0))
         if n["gate"] is not None:
             specs.append(TensorSpec(n["gate"], (self.gate_cols, self.hidden)))
         return specs
@@ -176,30 +190,52 @@ class MaskedAttention(Mixer):
         self.q_weight = tensors[n["q_norm"]] if n["q_norm"] is not None else None
         self.k_weight = tensors[n["k_norm"]] if n["k_norm"] is not None else None
         self.key_bias = tensors[n["key_bias"]] if n["key_bias"] is not None else None
+        self.sink = tensors[n["sink"]] if n["sink"] is not None else None
 
     def cache_spec(self):
         return PagedKV(self.kv_heads, self.dim, None if self.causal else self.size, self.vdim, keep_first=self.keep_first)
+
+    def _attend(self, proj, step, cache, out=None):
+        """Prepares the heads of the projected rows in place, stores keys and values, and attends;
+        ``out``: rows to write (of their own when None)."""
+        ops = self.env.ops
+        inv_freq, rotary_dim = self.position.rotary()
+        table = step.block_tables[cache.group]
+        gate = proj[:, self.q_cols + self.kv_cols :] if self.names["gate"] is not None else None
+        more = {"gate_per_element": True} if gate is not None and self.gate_per == "element" else {}
+        if self.sink is not None:
+            more["sink"] = self.sink
+        if out is not None:
+            more["out"] = out
+        if self.head_norm == "joined":
+            turn = {"inv_freq": inv_freq, "rotary_dim": rotary_dim} if rotary_dim else {}
+            q = ops.joined_norm_store(
+                proj, self.heads, self.kv_heads, self.dim, self.vdim, self.q_weight, self.k_weight, self.eps, self.q_temperature,
+                self.values == "keys", step, cache.k, cache.v, table, cache.page_size, **turn,
+            )
+        else:
+            q = ops.head_prepare_store(
+                proj, self.heads, self.kv_heads, self.dim, self.vdim, self.q_weight, self.k_weight, self.eps, self.head_norm,
+                inv_freq, rotary_dim, float(getattr(self.position, "magnitude", 1.0)), step, cache.k, cache.v, table, cache.page_size,
+            )
+        return ops.masked_attention(
+            q, self.heads, cache.k, cache.v, table, cache.page_size, self.scale, self.mask, self.size, self.keep_first, step,
+            sigmoid=self.weights == "sigmoid", key_bias=self.key_bias, softcap=self.softcap, gate=gate, **more,
+        )
+
+    def mix(self, proj, step, cache, out, out_scale=1.0):
+        """``proj[T, in_width]`` (rows may be strided) -> ``out[T, out_width]``."""
+        if self.in_bias is not None or out_scale != 1.0:
+            raise RuntimeError("as a branch this mixer has no projection biases and its output no scale")
+        self._attend(proj, step, cache, out)
 
     def forward(self, x, step, cache):
         ops = self.env.ops
         proj = ops.linear(x, self.in_matrix, self.env.dtype, self.in_bias)
         inv_freq, rotary_dim = self.position.rotary()
-        table = step.block_tables[cache.group]
         from_qkv = getattr(ops, "decode_attention_from_qkv", None)
-        gate = proj[:, self.q_cols + self.kv_cols :] if self.names["gate"] is not None else None
-        more = {"gate_per_element": True} if gate is not None and self.gate_per == "element" else {}
-        if self.head_norm == "joined":
-            q = ops.joined_norm_store(
-                proj, self.heads, self.kv_heads, self.dim, self.vdim, self.q_weight, self.k_weight, self.eps, self.q_temperature,
-                self.values == "keys", step, cache.k, cache.v, table, cache.page_size,
-            )
-            out = ops.masked_attention(
-                q, self.heads, cache.k, cache.v, table, cache.page_size, self.scale, self.mask, self.size, self.keep_first, step,
-                sigmoid=self.weights == "sigmoid", key_bias=self.key_bias, softcap=self.softcap, gate=gate, **more,
-            )
-            return DeferredLinear(ops, out, self.out_matrix, self.env.dtype)
         if (
-            from_qkv is not None and self.mask == "window" and self.weights == "softmax" and self.softcap is None
+            from_qkv is not None and self.mask == "window" and self.weights == "softmax" and self.softcap is None and self.sink is None
             and self.names["gate"] is None and self.head_norm == "before" and self.q_weight is not None and self.k_weight is not None
             and self.dim == self.vdim and float(getattr(self.position, "magnitude", 1.0)) == 1.0
         ):
@@ -207,16 +243,8 @@ class MaskedAttention(Mixer):
             # attention in the one launch the framework's other attention layers take (None otherwise)
             attn = from_qkv(
                 proj, self.heads, self.kv_heads, self.dim, self.q_weight, self.k_weight, self.eps, inv_freq, rotary_dim, step,
-                cache.k, cache.v, table, cache.page_size, True, self.scale, self.size, keep_first=self.keep_first,
+                cache.k, cache.v, step.block_tables[cache.group], cache.page_size, True, self.scale, self.size, keep_first=self.keep_first,
             )
             if attn is not None:
                 return DeferredLinear(ops, attn, self.out_matrix, self.env.dtype)
-        q = ops.head_prepare_store(
-            proj, self.heads, self.kv_heads, self.dim, self.vdim, self.q_weight, self.k_weight, self.eps, self.head_norm,
-            inv_freq, rotary_dim, float(getattr(self.position, "magnitude", 1.0)), step, cache.k, cache.v, table, cache.page_size,
-        )
-        out = ops.masked_attention(
-            q, self.heads, cache.k, cache.v, table, cache.page_size, self.scale, self.mask, self.size, self.keep_first, step,
-            sigmoid=self.weights == "sigmoid", key_bias=self.key_bias, softcap=self.softcap, gate=gate, **more,
-        )
-        return DeferredLinear(ops, out, self.out_matrix, self.env.dtype)
+        return DeferredLinear(ops, self._attend(proj, step, cache), self.out_matrix, self.env.dtype)

@@ -13,7 +13,7 @@ from typing import Optional
 import torch
 
 from ..weights.spec import NORMAL, VECTOR, TensorSpec
-from .base import BLOCKS, EMBEDDINGS, HEADS, NORMS, BuildEnv, DeferredLinear, Stream
+from .base import BLOCKS, EMBEDDINGS, HEADS, NORMS, BuildEnv, Stream
 from .plan import ModelPlan
 
 
@@ -29,7 +29,7 @@ def stream_value(stream: Stream) -> torch.Tensor:
         return x.clone()
     total = x.clone()
     for part in waiting if isinstance(waiting, tuple) else (waiting,):
-        if isinstance(part, DeferredLinear):
+        if hasattr(part, "materialize"):
             part = part.materialize()
         total += part.to(x.dtype)
     return total
@@ -64,7 +64,10 @@ class Model:
                 name, row = entry.add_vector
                 self.entry_vectors[name] = max(self.entry_vectors.get(name, 0), int(row) + 1)
         self.vectors = {}
-        self.keeps_first = any(entry.add_first for entry in plan.order)
+        # matrices that take the stream and the embedding's output side by side back to the width
+        self.entry_mixes = tuple(dict.fromkeys(entry.mix_first for entry in plan.order if entry.mix_first is not None))
+        self.mixes = {}
+        self.keeps_first = any(entry.add_first or entry.mix_first is not None for entry in plan.order)
         self.bound = False
 
     # ------------------------------------------------------------------ weights
@@ -78,12 +81,15 @@ class Model:
             specs += part.tensor_specs()
         for name, rows in self.entry_vectors.items():
             specs.append(TensorSpec(name, (rows, self.plan.hidden_size), VECTOR, NORMAL))
+        for name in self.entry_mixes:
+            specs.append(TensorSpec(name, (self.plan.hidden_size, 2 * self.plan.hidden_size)))
         return specs
 
     def bind(self, tensors: dict[str, torch.Tensor]) -> None:
         for part in self.parts():
             part.bind(tensors)
         self.vectors = {name: tensors[name] for name in self.entry_vectors}
+        self.mixes = {name: tensors[name] for name in self.entry_mixes}
         self.bound = True
 
     @property
@@ -113,7 +119,8 @@ class Model:
     # ------------------------------------------------------------------ additions between entries
 
     def _add_to_stream(self, stream: Stream, entry, first):
-        """What ``entry`` adds to the stream before its layer: the block output that was waiting, the
+        """What ``entry`` does to the stream before its layer: ``mix_first``'s product over the stream and the
+        embedding's rows side by side (the block output that was waiting is added on the way in), and / or additions: the block output that was waiting, the
         embedding's rows (``first``) and a row of a tensor, in one kernel.  Returns the embedding's
         rows, which the first call keeps apart (it then writes the sums to rows of their own)."""
         ops = self.env.ops
@@ -125,6 +132,16 @@ class Model:
             vector = self.vectors[name][row]
         waiting = stream.take_pending()
         deltas = list(waiting) if isinstance(waiting, tuple) else ([waiting] if waiting is not None else [])
+        if entry.mix_first is not None:
+            if first is None:  # the stream is the embedding's output itself, and is not written again
+                first = stream.residual
+            side_by_side = ops.stream_concat(stream.residual, tuple(deltas), first, self.env.dtype)
+            # (a vector of the entry rides as the product's bias)
+            stream.residual = ops.linear(side_by_side, self.mixes[entry.mix_first], torch.float32, None if entry.add_first else vector)
+            stream.current = None
+            if entry.add_first:
+                ops.stream_add(stream.residual, (first,), vector)
+            return first
         if entry.add_first:
             if first is None:
                 raise RuntimeError("the first run entry cannot add the embedding's rows to themselves")
@@ -157,7 +174,7 @@ class Model:
             layer_hook(-1, stream)
         first = None
         for pos, entry in enumerate(self.plan.order):
-            if entry.add_first or entry.add_vector is not None:
+            if entry.add_first or entry.add_vector is not None or entry.mix_first is not None:
                 first = self._add_to_stream(stream, entry, first)
             elif self.keeps_first and first is None and pos == 0:
                 first = stream.residual.clone()  # the first block adds to the residual in place
@@ -176,7 +193,7 @@ class Model:
             # (handed over unevaluated to a head that says it takes that: its product may apply the row scale itself)
             return self.head.forward(stream.normed(self.final_norm, deferred=getattr(self.head, "takes_deferred_norm", False)))
         rows = step.want_rows
-        delta = stream.take_pending()
+        delta = stream.take_pending(self.final_norm)
         if delta is not None:
             normed = self.final_norm.add_apply(stream.residual, delta, rows)
         else:

@@ -22,11 +22,13 @@ from __future__ import annotations
 import torch
 
 from ..weights.spec import NORMAL, ONES, VECTOR, TensorSpec
-from .base import NORMS, Norm
+from .base import NORMS, Norm, NormedPair
 
 
 @NORMS.register("rmsnorm")
 class RMSNorm(Norm):
+    takes_pairs = True
+
     def __init__(self, spec, env):
         super().__init__(spec, env)
         self.tensor_name = spec.params["tensor"]
@@ -61,6 +63,9 @@ class RMSNorm(Norm):
         return self.env.ops.rmsnorm(x, self.weight, self.eps, self.env.dtype)
 
     def add_apply(self, residual, delta, rows=None):
+        if isinstance(delta, NormedPair):
+            return self.env.ops.add_normed_pair_rmsnorm(
+                residual, delta.left, delta.right, delta.left_w, delta.right_w, delta.scale, delta.eps, self.weight, self.eps, rows)
         return self.env.ops.add_rmsnorm(residual, delta, self.weight, self.eps, self.env.dtype, rows)
 
     def add_normed(self, residual, y, want_rows=True):

@@ -60,13 +60,15 @@ class RunEntry:
     embedding's output (the rows as they stood before the first entry), and with
     ``add_vector = (tensor name, row)`` one row of a ``[rows, hidden]`` tensor, the same for
     every token - what a model does that runs a stretch of layers several times and tells
-    the passes apart.
+    the passes apart.  ``mix_first = tensor name`` (``[hidden, 2 hidden]``) comes before both: the stream
+    becomes that matrix times the stream and the embedding's output side by side.
     """
 
     layer: int
     cache_of: Optional[int] = None
     add_first: bool = False
     add_vector: Optional[tuple] = None
+    mix_first: Optional[str] = None
 
 
 @dataclass(frozen=True)

@@ -656,12 +656,14 @@ def latent_attention(q_lat, rank, k_cache, block_table, page_size, scale, step):
 # --------------------------------------------------------------------------- mixture of experts
 
 
-def moe_route(logits, top, group_count, group_keep, scale, sigmoid=False, renormalize=False, correction=None, renorm_eps=0.0):
+def moe_route(logits, top, group_count, group_keep, scale, sigmoid=False, renormalize=False, correction=None, renorm_eps=0.0,
+              scores=None):
     """Expert ids (int32 ``[T, top]``, best first) and weights (float32) of every row.  Groups and
-    experts are ranked by score + ``correction``; the weights are the scores themselves."""
+    experts are ranked by score + ``correction``; the weights are the scores themselves.  ``scores =
+    "chosen_softmax"``: the logits are ranked, and the weights are the softmax over the chosen ones."""
     T, E = logits.shape
     z = logits.to(F64)
-    s = _sigmoid(z) if sigmoid else torch.softmax(z, dim=-1)
+    s = z if scores == "chosen_softmax" else _sigmoid(z) if sigmoid else torch.softmax(z, dim=-1)
     choice = s if correction is None else s + correction.to(F64)
     per = E // group_count
     best = choice.reshape(T, group_count, per).max(-1).values
@@ -672,7 +674,9 @@ def moe_route(logits, top, group_count, group_keep, scale, sigmoid=False, renorm
     masked = torch.where(allowed, choice, torch.full_like(s, float("-inf")))
     ids = torch.sort(masked, dim=-1, descending=True, stable=True).indices[:, :top]
     w = torch.gather(s, 1, ids)
-    if renormalize:
+    if scores == "chosen_softmax":
+        w = torch.softmax(w, dim=-1)
+    elif renormalize:
         w = w / (w.sum(-1, keepdim=True) + renorm_eps)
     return ids.to(torch.int32), (w * scale).to(torch.float32)
 
@@ -697,7 +701,7 @@ def routed_experts(x, ids, weights, gate_up, down, extra=None, act="silu", limit
                 out[t] += float(weights[t, j]) * x64[t]
                 continue
             y = gate_up[e].to(F64) @ x64[t]
-            mid = _glu(y[:inter], y[inter:], act, limit)
+            mid = torch.relu(y) ** 2 if act == "relu2" else _glu(y[:inter], y[inter:], act, limit)
             out[t] += float(weights[t, j]) * (down[e].to(F64) @ mid)
     return out.to(x.dtype)
 
@@ -736,11 +740,11 @@ def head_prepare_store(proj, heads, kv_heads, dim, vdim, q_w, k_w, eps, norm_ord
 
 
 def joined_norm_store(proj, heads, kv_heads, dim, vdim, q_w, k_w, eps, q_temperature, values_from_keys, step, k_cache, v_cache,
-                      block_table, page_size):
+                      block_table, page_size, inv_freq=None, rotary_dim=0):
     """``proj[T, heads*dim | kv_heads*dim | (kv_heads*vdim) | ...]``: one RMS norm over all query
     columns together (weight ``q_w[heads*dim]``) and one over all key columns; the queries times
-    ``1 + coef * ln(floor((p + 1) / every) + 1)`` when ``q_temperature = (coef, every)``; queries
-    written back in place, keys to the cache; the values are the key columns as they came
+    ``1 + coef * ln(floor((p + 1) / every) + 1)`` when ``q_temperature = (coef, every)``; then the
+    half-split rotation of every head's first ``rotary_dim`` entries; queries written back in place, keys to the cache; the values are the key columns as they came
     (``values_from_keys``) or the value columns."""
     T = proj.shape[0]
     x = proj.to(F64)
@@ -758,6 +762,9 @@ def joined_norm_store(proj, heads, kv_heads, dim, vdim, q_w, k_w, eps, q_tempera
         v = proj[:, q_cols : q_cols + k_cols].clone()
     else:
         v = proj[:, q_cols + k_cols : q_cols + k_cols + kv_heads * vdim]
+    if rotary_dim:
+        q = _rotate_rows(q.reshape(T, heads, dim), step.positions, inv_freq, rotary_dim).reshape(T, q_cols)
+        k = _rotate_rows(k.reshape(T, kv_heads, dim), step.positions, inv_freq, rotary_dim)
     proj[:, :q_cols] = q.to(proj.dtype)
     rows = _cache_rows(block_table, step.seq_of_token, step.positions, page_size)
     k_cache.view(-1, kv_heads, dim)[rows] = k.reshape(T, kv_heads, dim).to(k_cache.dtype)
@@ -766,12 +773,12 @@ def joined_norm_store(proj, heads, kv_heads, dim, vdim, q_w, k_w, eps, q_tempera
 
 
 def masked_attention(q, heads, k_cache, v_cache, block_table, page_size, scale, mask, size, keep_first, step, *, sigmoid=False,
-                     key_bias=None, softcap=None, gate=None, general=False, gate_per_element=False):
+                     key_bias=None, softcap=None, gate=None, general=False, gate_per_element=False, sink=None, out=None):
     T = q.shape[0]
     kv_heads, dim, vdim = k_cache.shape[2], k_cache.shape[3], v_cache.shape[3]
     q64 = q.to(F64).reshape(T, heads, dim)
     kf, vf = k_cache.view(-1, kv_heads, dim), v_cache.view(-1, kv_heads, vdim)
-    out = torch.zeros(T, heads, vdim, dtype=F64)
+    given, out = out, torch.zeros(T, heads, vdim, dtype=F64)
     seq, pos = step.seq_of_token.tolist(), step.positions.tolist()
     for t in range(T):
         i = pos[t]
@@ -792,6 +799,8 @@ def masked_attention(q, heads, k_cache, v_cache, block_table, page_size, scale, 
                 s = softcap * torch.tanh(s / softcap)
             if sigmoid:
                 w = torch.sigmoid(s + (float(key_bias[h]) if key_bias is not None else 0.0))
+            elif sink is not None:  # one more entry of the softmax, without a value
+                w = torch.softmax(torch.cat([s, sink[h].to(F64).reshape(1)]), dim=0)[:-1]
             else:
                 w = torch.softmax(s, dim=0)
             out[t, h] = w @ v[:, g, :]
@@ -799,7 +808,8 @@ def masked_attention(q, heads, k_cache, v_cache, block_table, page_size, scale, 
                 out[t, h] *= torch.sigmoid(gate[t, h * vdim : (h + 1) * vdim].to(F64))
             elif gate is not None:
                 out[t, h] *= torch.sigmoid(gate[t, h].to(F64))
-    return out.reshape(T, heads * vdim).to(q.dtype)
+    out = out.reshape(T, heads * vdim).to(q.dtype)
+    return out if given is None else given.copy_(out)
 
 
 def norm_into(residual, y, w, eps, want_rows=True):
@@ -809,6 +819,66 @@ def norm_into(residual, y, w, eps, want_rows=True):
     if not want_rows:
         return None
     return residual if y.dtype == torch.float32 else residual.to(y.dtype)
+
+
+def _unit_rms(x, eps):
+    x = x.to(F64)
+    return x / torch.sqrt((x * x).mean(-1, keepdim=True) + eps)
+
+
+def normed_pair(left, right, wa, wb, scale, pair_eps):
+    return (scale * (_unit_rms(left, pair_eps) * wa.to(F64) + _unit_rms(right, pair_eps) * wb.to(F64))).to(torch.float32)
+
+
+def add_normed_pair_rmsnorm(residual, left, right, wa, wb, scale, pair_eps, w, eps, rows=None):
+    delta = normed_pair(left, right, wa, wb, scale, pair_eps)
+    if rows is None:
+        residual += delta
+        return rmsnorm(residual, w, eps, left.dtype)
+    idx = rows.long()
+    return rmsnorm(residual[idx] + delta[idx], w, eps, left.dtype)
+
+
+def stream_concat(residual, deltas, first, out_dtype):
+    x = residual.to(F64)
+    for d in deltas:
+        x = x + d.to(F64)
+    return torch.cat([x, first.to(F64)], dim=-1).to(out_dtype)
+
+
+def delta_rule(q, k, v, b, a, dt_bias, a_log, state, step, heads, groups, dim, vdim, q_scale, unit_eps):
+    """Per head ``S[dim, vdim]``: ``S <- g S``, ``u = beta (v - S^T k)``, ``S <- S + k u^T``, ``o = S^T q``,
+    with unit keys and queries (``q`` times ``q_scale``).  Returns float32 ``[T, heads * vdim]``."""
+    T, per = q.shape[0], heads // groups
+
+    def unit(x):
+        x = x.to(F64).reshape(T, groups, dim)
+        return (x / torch.sqrt((x * x).sum(-1, keepdim=True) + unit_eps)).repeat_interleave(per, dim=1)
+
+    q64, k64, v64 = unit(q) * q_scale, unit(k), v.to(F64).reshape(T, heads, vdim)
+    z = a.to(F64) + dt_bias.to(F64)
+    g = torch.exp(-torch.exp(a_log.to(F64)) * torch.where(z > 30.0, z, torch.log1p(torch.exp(torch.clamp(z, max=30.0)))))
+    beta = _sigmoid(b.to(F64))
+    o = torch.zeros(T, heads, vdim, dtype=F64)
+    q_start, slots = step.q_start.tolist(), step.state_slots.tolist()
+    for s in range(step.num_seqs):
+        if q_start[s + 1] == q_start[s]:
+            continue
+        S = state[slots[s]].to(F64)
+        for t in range(q_start[s], q_start[s + 1]):
+            S = g[t][:, None, None] * S
+            u = beta[t][:, None] * (v64[t] - torch.einsum("hij,hi->hj", S, k64[t]))
+            S = S + k64[t][:, :, None] * u[:, None, :]
+            o[t] = torch.einsum("hij,hi->hj", S, q64[t])
+        state[slots[s]] = S.to(state.dtype)
+    return o.reshape(T, heads * vdim).to(torch.float32)
+
+
+def delta_output(x, gate, weight, heads, eps, out):
+    T = x.shape[0]
+    g = gate.to(F64)
+    y = (_unit_rms(x.reshape(T, heads, -1), eps) * weight.to(F64)).reshape(T, -1) * g * _sigmoid(g)
+    return out.copy_(y.to(out.dtype))
 
 
 def polynorm(z, coefficients, eps, out_dtype):
