@@ -354,7 +354,7 @@ def compare_designs(args) -> dict:
 
         def top(kind):
             return [{"kernel": r["kernel"], "shape": r["shape"], "launches": r["launches_per_step"], "us": round(r["us_per_step"], 1)}
-                    for r in report[kind]["rows"][:14]]
+                    for r in report[kind]["rows"][:24]]
 
         designs[name] = {
             "parameters": parameters,

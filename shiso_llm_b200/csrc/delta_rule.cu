@@ -7,44 +7,41 @@
 // g = exp(-exp(a_log_h) softplus(a + dt_bias_h)) from one logit each per row and head.  q and k may
 // be shared by the heads of a group (head h reads group h / (heads / groups)).
 //
-// A column of S needs both S^T k and S^T q; they are taken in ONE pass over the old state, since
-//     u = beta (v - g p),   o = g r + u (k . q)   with p = S_old^T k, r = S_old^T q,
-// so a row costs one exchange across lanes, not two that wait for one another.
+// Steps with portions of prompts: the rows of a sequence are taken EIGHT at a time.  Unrolled over
+// a block of rows with old state S, and with G_i = g_1 .. g_i and D_ij = g_(j+1) .. g_i (products, never
+// quotients),
 //
-// delta_rule_kernel: one CTA walks the rows of one (head, sequence, range of value columns) in
-// order.  Eight lanes hold a column, each dim / 8 of its rows in runs of four (rows 32 j + 4 lane .. + 3:
-// 16-byte words of shared memory, eight lanes a full 128-byte line, the columns of a warp reading the
-// same words), as pairs of floats for the two-wide multiply-add.  What is added to what depends on
-// dim only - never on how the sequence was cut into steps, on the batch, or on how many columns a CTA
-// was given.  Four warps that hold no state stage the rows sixteen at a time, a warp a row: copies
-// (cp.async) of the rows after next are on their way while the next are normalised and the current
-// ones walked; outputs leave through shared memory, written by the same warps.
+//     u_i = beta_i (v_i - G_i S^T k_i - sum_(j<i) D_ij (k_i . k_j) u_j)
+//     o_i = G_i S^T q_i + sum_(j<=i) D_ij (q_i . k_j) u_j
+//     S  <- G_8 S + sum_j D_8j k_j u_j^T.
 //
-// delta_output_kernel: each head's float outputs divided by their root mean square, times a weight
-// shared by the heads, times silu(gate).
+// With A_ij = beta_i D_ij (k_i . k_j) below the diagonal, w_i = beta_i v_i - beta_i G_i S^T k_i and
+// T = (I + A)^-1 (a unit triangle, by substitution) this is u = T w and o = G S^T q + M w with
+// M = (D o (Q K^T)) T: everything that couples the rows is eight-by-eight, the same for all columns
+// of the state, and found beforehand.
 //
-// delta_step_kernel: a step of single rows (decode) in ONE launch: the causal convolutions of q, k and
-// v with silu and their windows, unit vectors, the state, the output norm and the gate.
+//   delta_prepare_kernel  per (block of rows, group): unit vectors, the dot products between them,
+//                         decays, the two triangles per head, beta v; float, in the order the next reads.
+//   delta_blocks_kernel   per (head, sequence, range of value columns), block after block: S^T k and
+//                         S^T q of all eight rows from the old state, ONE exchange across lanes for the
+//                         sixteen results, the triangles, the state.  Walked row by row the state waits
+//                         for an exchange across lanes per row; and a lane that holds four columns uses
+//                         each key and query it reads from shared memory four times.
+//   delta_output_kernel   each head's outputs divided by their root mean square, times a weight shared
+//                         by the heads, times silu(gate).
+//
+// Blocks are counted from a portion's start, so another cut of a prompt adds the same numbers up in
+// another order (float throughout; a sequence's sums never depend on the rest of the batch).
+//
+// Steps of single rows (decode): delta_step_kernel, ONE launch for the convolutions of q, k and v with
+// silu and their windows, unit vectors, the state, the output norm and the gate.
 #include "common.cuh"
 
 namespace {
 
-constexpr int DR_ROWS = 16;      // rows a stage holds
-constexpr int DR_STAGERS = 128;  // threads behind the ones that hold state
-constexpr int DR_STAGE_WARPS = DR_STAGERS / 32;
-
-struct DeltaArgs {
-    const void *q, *k, *v, *b, *a;
-    long long q_ld, k_ld, v_ld, b_ld, a_ld;
-    const float *dt_bias, *a_log;
-    float* state;
-    long long slot_stride;
-    const int *q_start, *state_slots;
-    float* out;
-    int heads, groups, dim, vdim, cols;
-    int bulk;  // rows may be fetched 16 bytes at a time (widths, strides and addresses allow it)
-    float q_scale, unit_eps;
-};
+constexpr int DB = 8;            // rows a block
+constexpr int DC = 2 * DB * DB + 2 * DB + 4;  // a (head, block)'s coefficients: D_8i T_ij, M_ij, beta_i G_i, G_i, G_8 (and padding)
+constexpr int D_MAX_DIM = 256;
 
 __device__ __forceinline__ uint64_t fma2(uint64_t a, uint64_t b, uint64_t c) {
     uint64_t d;
@@ -63,9 +60,8 @@ __device__ __forceinline__ uint64_t pair_of(float lo, float hi) {
 }
 __device__ __forceinline__ void halves_of(uint64_t v, float& lo, float& hi) { asm("mov.b64 {%0, %1}, %2;" : "=f"(lo), "=f"(hi) : "l"(v)); }
 
-__device__ __forceinline__ void cp16(void* dst, const void* src, bool valid) {
-    const int bytes = valid ? 16 : 0;
-    asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"((uint32_t)__cvta_generic_to_shared(dst)), "l"(src), "r"(bytes) : "memory");
+__device__ __forceinline__ void cp16(void* dst, const void* src) {
+    asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"((uint32_t)__cvta_generic_to_shared(dst)), "l"(src) : "memory");
 }
 
 __device__ __forceinline__ float decay_of(float a_logit, float dt_bias, float rate) {
@@ -76,235 +72,530 @@ __device__ __forceinline__ float decay_of(float a_logit, float dt_bias, float ra
 __device__ __forceinline__ float sigmoid_of(float z) { return 1.0f / (1.0f + expf(-z)); }
 __device__ __forceinline__ float silu_of(float z) { return z / (1.0f + expf(-z)); }
 
-// RPT: key rows a lane holds (dim rounded up to a multiple of 32, divided by 8).
-template <typename AT, int RPT>
-__global__ void __launch_bounds__(RPT > 16 ? 256 : RPT > 8 ? 384 : 640) delta_rule_kernel(const DeltaArgs a) {
-    constexpr int DP = 8 * RPT;  // key rows with padding (zeros: their state stays zero)
-    constexpr int EPV = 16 / (int)sizeof(AT);
-    const int h = blockIdx.x, s = blockIdx.y, col0 = blockIdx.z * a.cols;
-    const int workers = a.cols * 8;
-    const bool stager = (int)threadIdx.x >= workers;
-    const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
-    const int part = lane & 7, local = warp * 4 + (lane >> 3), col = col0 + local;
-    const int dim = a.dim, vdim = a.vdim, cols = a.cols, g = h / (a.heads / a.groups);
-    extern __shared__ __align__(16) float sm[];
-    // two stages: q [ROWS][DP], k [ROWS][DP], v [ROWS][cols], (g, beta, k . q, -) [ROWS][4]; two blocks of outputs
-    // [ROWS][cols]; two raw areas: q [ROWS][dim], k [ROWS][dim], v [ROWS][cols] as they came
-    const int stage_floats = DR_ROWS * (2 * DP + cols + 4);
-    float* outs = sm + 2 * stage_floats;
-    AT* raw = reinterpret_cast<AT*>(outs + 2 * DR_ROWS * cols);
-    const int raw_elems = DR_ROWS * (2 * dim + cols);
-    __shared__ float logits[2][DR_ROWS][2];
-    const float rate = expf(a.a_log[h]), dt_bias = a.dt_bias[h];
-    pdl_wait();
-    const int first = a.q_start[s], n = a.q_start[s + 1] - first;
-    if (n <= 0) return;
-    const int batches = (n + DR_ROWS - 1) / DR_ROWS;
-    const AT* qp = (const AT*)a.q + (size_t)first * a.q_ld + (size_t)g * dim;
-    const AT* kp = (const AT*)a.k + (size_t)first * a.k_ld + (size_t)g * dim;
-    const AT* vp = (const AT*)a.v + (size_t)first * a.v_ld + (size_t)h * vdim + col0;
+// Block b of sequence s is number q_start[s] / 8 + s + b of the step: enough room for every sequence's
+// last, ragged block, and no prefix sum to find it.
+__device__ __forceinline__ int first_block(const int* q_start, int s) { return q_start[s] / DB + s; }
 
-    if (stager) {
-        const int me = (int)threadIdx.x - workers, mywarp = me >> 5;
-        const AT* bp = (const AT*)a.b + (size_t)first * a.b_ld + h;
-        const AT* ap = (const AT*)a.a + (size_t)first * a.a_ld + h;
-        float* op = a.out + (size_t)first * a.heads * vdim + (size_t)h * vdim + col0;
-        float b_logit = 0.0f, a_logit = 0.0f;
-        auto fetch = [&](int batch) {
-            const int base = batch * DR_ROWS, count = min(DR_ROWS, n - base);
-            if (a.bulk) {
-                AT* rq = raw + (batch & 1) * raw_elems;
-                AT* rk = rq + DR_ROWS * dim;
-                AT* rv = rk + DR_ROWS * dim;
-                const int pieces = dim / EPV, vpieces = cols / EPV;
-                for (int i = me; i < DR_ROWS * pieces; i += DR_STAGERS) {
-                    const int t = i / pieces, c = (i - t * pieces) * EPV;
-                    const bool ok = t < count;
-                    cp16(rq + t * dim + c, ok ? qp + (size_t)(base + t) * a.q_ld + c : qp, ok);
-                    cp16(rk + t * dim + c, ok ? kp + (size_t)(base + t) * a.k_ld + c : kp, ok);
-                }
-                for (int i = me; i < DR_ROWS * vpieces; i += DR_STAGERS) {
-                    const int t = i / vpieces, c = (i - t * vpieces) * EPV;
-                    const bool ok = t < count && col0 + c < vdim;
-                    cp16(rv + t * cols + c, ok ? vp + (size_t)(base + t) * a.v_ld + c : vp, ok);
-                }
-            }
-            asm volatile("cp.async.commit_group;" ::: "memory");
-            if (me < count) {
-                b_logit = to_f32(bp[(size_t)(base + me) * a.b_ld]);
-                a_logit = to_f32(ap[(size_t)(base + me) * a.a_ld]);
-            }
-        };
-        auto convert = [&](int batch) {  // a warp a row
-            const int base = batch * DR_ROWS, count = min(DR_ROWS, n - base);
-            const AT* rq = raw + (batch & 1) * raw_elems;
-            const AT* rk = rq + DR_ROWS * dim;
-            const AT* rv = rk + DR_ROWS * dim;
-            float* sq = sm + (batch & 1) * stage_floats;
-            float* sk = sq + DR_ROWS * DP;
-            float* sv = sk + DR_ROWS * DP;
-            float* sc = sv + DR_ROWS * cols;
-            for (int t = mywarp; t < count; t += DR_STAGE_WARPS) {
-                const AT* q_row = a.bulk ? rq + t * dim : qp + (size_t)(base + t) * a.q_ld;
-                const AT* k_row = a.bulk ? rk + t * dim : kp + (size_t)(base + t) * a.k_ld;
-                const AT* v_row = a.bulk ? rv + t * cols : vp + (size_t)(base + t) * a.v_ld;
-                float qv[RPT / 4], kv[RPT / 4];
-                float qq = 0.0f, kk = 0.0f, qk = 0.0f;
-#pragma unroll
-                for (int i = 0; i < RPT / 4; ++i) {
-                    const int c = lane + 32 * i;
-                    qv[i] = c < dim ? to_f32(q_row[c]) : 0.0f;
-                    kv[i] = c < dim ? to_f32(k_row[c]) : 0.0f;
-                    qq += qv[i] * qv[i];
-                    kk += kv[i] * kv[i];
-                    qk += qv[i] * kv[i];
-                }
-                qq = warp_sum(qq);
-                kk = warp_sum(kk);
-                qk = warp_sum(qk);
-                const float iq = rsqrtf(qq + a.unit_eps) * a.q_scale, ik = rsqrtf(kk + a.unit_eps);
-#pragma unroll
-                for (int i = 0; i < RPT / 4; ++i) {
-                    sq[t * DP + lane + 32 * i] = qv[i] * iq;
-                    sk[t * DP + lane + 32 * i] = kv[i] * ik;
-                }
-                for (int c = lane; c < cols; c += 32) sv[t * cols + c] = col0 + c < vdim ? to_f32(v_row[c]) : 0.0f;
-                if (lane == 0)
-                    *reinterpret_cast<float4*>(sc + t * 4) = make_float4(decay_of(logits[batch & 1][t][1], dt_bias, rate),
-                                                                         sigmoid_of(logits[batch & 1][t][0]), qk * iq * ik, 0.0f);
-            }
-        };
-        auto flush = [&](int batch) {
-            const int base = batch * DR_ROWS, count = min(DR_ROWS, n - base);
-            const float* so = outs + (batch & 1) * DR_ROWS * cols;
-            for (int i = me; i < count * cols; i += DR_STAGERS) {
-                const int t = i / cols, c = i - t * cols;
-                if (col0 + c < vdim) op[(size_t)(base + t) * a.heads * vdim + c] = so[i];
-            }
-        };
-        fetch(0);
-        for (int batch = 0; batch < batches; ++batch) {
-            asm volatile("cp.async.wait_group 0;" ::: "memory");
-            if (me < DR_ROWS) logits[batch & 1][me][0] = b_logit, logits[batch & 1][me][1] = a_logit;
-            asm volatile("bar.sync 1, %0;" ::"n"(DR_STAGERS) : "memory");
-            // (the other raw area was converted before the last of the block's barriers)
-            if (batch + 1 < batches) fetch(batch + 1);
-            convert(batch);
-            if (batch >= 2) flush(batch - 2);
-            __syncthreads();  // this batch is staged; the batch before it has been walked
-        }
-        if (batches >= 2) flush(batches - 2);
-        __syncthreads();
-        flush(batches - 1);
-        pdl_trigger();
-        return;
-    }
+// --------------------------------------------------------------------------- what couples a block's rows
 
-    const bool live = col < vdim;
-    float* slot = a.state + (size_t)a.state_slots[s] * a.slot_stride + (size_t)h * dim * vdim;
-    uint64_t S[RPT / 2];
+struct PrepareArgs {
+    const void *q, *k, *v, *b, *a;
+    long long q_ld, k_ld, v_ld, b_ld, a_ld;
+    const float *dt_bias, *a_log;
+    const int* q_start;
+    float* kq;    // [groups][blocks][k: 8 x DP | q: 8 x DP]
+    float* coef;  // [heads][blocks][DC]
+    float* bv;    // [heads][blocks][chunks of 8 columns][8 rows][8 columns]: beta v
+    int num_seqs, blocks, heads, groups, dim, dp, vdim, chunks;
+    float q_scale, unit_eps;
+};
+
+template <typename AT>
+__global__ void __launch_bounds__(DB * 32) delta_prepare_kernel(const PrepareArgs a) {
+    constexpr int PER = D_MAX_DIM / 32;
+    __shared__ float ks[DB][D_MAX_DIM];
+    __shared__ float kk[DB][DB], qk[DB][DB];
+    __shared__ float tri[DB][DB * DB], inv[DB][DB * DB];  // per warp: A, then T, of the head it works on
+    __shared__ float gs[DB][DB];
+    __shared__ int s_seq;
+    pdl_begin();
+    const int blk = blockIdx.x, g = blockIdx.y, lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+    if (threadIdx.x == 0) s_seq = -1;
+    __syncthreads();
+    for (int s = threadIdx.x; s < a.num_seqs; s += blockDim.x)
+        if (first_block(a.q_start, s) <= blk && blk < first_block(a.q_start, s) + (a.q_start[s + 1] - a.q_start[s] + DB - 1) / DB) s_seq = s;
+    __syncthreads();
+    const int s = s_seq;
+    if (s < 0) return;
+    const int base = a.q_start[s] + (blk - first_block(a.q_start, s)) * DB;
+    const int count = min(DB, a.q_start[s + 1] - base);
+    // a warp a row: unit vectors (rows beyond the portion are zeros)
+    const size_t row = (size_t)base + min(warp, count - 1);
+    const bool mine = warp < count;
+    const AT* qp = (const AT*)a.q + row * a.q_ld + (size_t)g * a.dim;
+    const AT* kp = (const AT*)a.k + row * a.k_ld + (size_t)g * a.dim;
+    float qv[PER], kv[PER];
+    float qq = 0.0f, kn = 0.0f;
 #pragma unroll
-    for (int r = 0; r < RPT; r += 2) {
-        const int row = (r >> 2) * 32 + part * 4 + (r & 3);
-        S[r / 2] = pair_of(live && row < dim ? slot[(size_t)row * vdim + col] : 0.0f,
-                           live && row + 1 < dim ? slot[(size_t)(row + 1) * vdim + col] : 0.0f);
+    for (int i = 0; i < PER; ++i) {
+        const int c = lane + 32 * i;
+        const bool ok = mine && c < a.dim;
+        qv[i] = ok ? to_f32(qp[c]) : 0.0f;
+        kv[i] = ok ? to_f32(kp[c]) : 0.0f;
+        qq += qv[i] * qv[i];
+        kn += kv[i] * kv[i];
     }
-    for (int batch = 0; batch < batches; ++batch) {
-        __syncthreads();
-        const int count = min(DR_ROWS, n - batch * DR_ROWS);
-        const float* sq = sm + (batch & 1) * stage_floats;
-        const float* sk = sq + DR_ROWS * DP;
-        const float* sv = sk + DR_ROWS * DP + local;
-        const float4* sc = reinterpret_cast<const float4*>(sk + DR_ROWS * DP + DR_ROWS * cols);
-        float* so = outs + (batch & 1) * DR_ROWS * cols + local;
-        const ulonglong2* kt = reinterpret_cast<const ulonglong2*>(sk) + part;
-        const ulonglong2* qt = reinterpret_cast<const ulonglong2*>(sq) + part;
-        uint64_t K[RPT / 2], Q[RPT / 2];
+    const float iq = rsqrtf(warp_sum(qq) + a.unit_eps) * a.q_scale, ik = rsqrtf(warp_sum(kn) + a.unit_eps);
+    float* kq = a.kq + ((size_t)g * a.blocks + blk) * 2 * DB * a.dp;
 #pragma unroll
-        for (int j = 0; j < RPT / 4; ++j) {
-            const ulonglong2 k2 = kt[8 * j], q2 = qt[8 * j];
-            K[2 * j] = k2.x, K[2 * j + 1] = k2.y;
-            Q[2 * j] = q2.x, Q[2 * j + 1] = q2.y;
-        }
-#pragma unroll 2
-        for (int t = 0; t < count; ++t) {
-            uint64_t p0 = 0, p1 = 0, r0 = 0, r1 = 0;  // (pairs of zeros)
-#pragma unroll
-            for (int j = 0; j < RPT / 2; j += 2) {
-                p0 = fma2(S[j], K[j], p0);
-                r0 = fma2(S[j], Q[j], r0);
-                p1 = fma2(S[j + 1], K[j + 1], p1);
-                r1 = fma2(S[j + 1], Q[j + 1], r1);
-            }
-            const float4 c4 = sc[t];  // decay, beta, k . q
-            const float v = sv[t * cols];
-            // the next row's keys and queries are asked for under the exchange below
-            uint64_t Kn[RPT / 2];
-            const int next = min(t + 1, count - 1);
-#pragma unroll
-            for (int j = 0; j < RPT / 4; ++j) {
-                const ulonglong2 k2 = kt[next * (DP / 4) + 8 * j], q2 = qt[next * (DP / 4) + 8 * j];
-                Kn[2 * j] = k2.x, Kn[2 * j + 1] = k2.y;
-                Q[2 * j] = q2.x, Q[2 * j + 1] = q2.y;
-            }
-            float pa, pb, pc, pd, ra, rb, rc, rd;
-            halves_of(p0, pa, pb);
-            halves_of(p1, pc, pd);
-            halves_of(r0, ra, rb);
-            halves_of(r1, rc, rd);
-            float p = (pa + pb) + (pc + pd), r = (ra + rb) + (rc + rd);
-#pragma unroll
-            for (int o = 1; o < 8; o <<= 1) {
-                p += __shfl_xor_sync(0xffffffffu, p, o);
-                r += __shfl_xor_sync(0xffffffffu, r, o);
-            }
-            const float u = c4.y * fmaf(-c4.x, p, v);
-            if (part == 0) so[t * cols] = fmaf(u, c4.z, c4.x * r);
-            const uint64_t u2 = pair_of(u, u), g2 = pair_of(c4.x, c4.x);
-#pragma unroll
-            for (int j = 0; j < RPT / 2; ++j) S[j] = fma2(K[j], u2, mul2(g2, S[j]));
-#pragma unroll
-            for (int j = 0; j < RPT / 2; ++j) K[j] = Kn[j];
+    for (int i = 0; i < PER; ++i) {
+        const int c = lane + 32 * i;
+        qv[i] *= iq;
+        kv[i] *= ik;
+        ks[warp][c] = kv[i];
+        if (c < a.dp) {
+            kq[warp * a.dp + c] = kv[i];
+            kq[(DB + warp) * a.dp + c] = qv[i];
         }
     }
     __syncthreads();
-    pdl_trigger();
+    // the products between the rows: warp i's row against rows j <= i
+    for (int j = 0; j <= warp; ++j) {
+        float x = 0.0f, y = 0.0f;
 #pragma unroll
-    for (int r = 0; r < RPT; r += 2) {
-        const int row = (r >> 2) * 32 + part * 4 + (r & 3);
-        float lo, hi;
-        halves_of(S[r / 2], lo, hi);
-        if (live && row < dim) slot[(size_t)row * vdim + col] = lo;
-        if (live && row + 1 < dim) slot[(size_t)(row + 1) * vdim + col] = hi;
+        for (int i = 0; i < PER; ++i) {
+            const float other = ks[j][lane + 32 * i];
+            x = fmaf(kv[i], other, x);
+            y = fmaf(qv[i], other, y);
+        }
+        x = warp_sum(x);
+        y = warp_sum(y);
+        if (lane == 0) kk[warp][j] = x, qk[warp][j] = y;
+    }
+    __syncthreads();
+    // a warp a head
+    const int per = a.heads / a.groups;
+    for (int hh = warp; hh < per; hh += DB) {
+        const int h = g * per + hh;
+        float decay = 1.0f, beta = 0.0f;
+        if (lane < count) {
+            decay = decay_of(to_f32(((const AT*)a.a)[((size_t)base + lane) * a.a_ld + h]), a.dt_bias[h], expf(a.a_log[h]));
+            beta = sigmoid_of(to_f32(((const AT*)a.b)[((size_t)base + lane) * a.b_ld + h]));
+        }
+        float* A = tri[warp];
+        float* T = inv[warp];
+        if (lane < DB) gs[warp][lane] = decay;
+        __syncwarp();
+        auto between = [&](int i, int j) {  // g_(j+1) .. g_i
+            float d = 1.0f;
+            for (int m = j + 1; m <= i; ++m) d *= gs[warp][m];
+            return d;
+        };
+#pragma unroll
+        for (int e = lane; e < DB * DB; e += 32) {
+            const int i = e / DB, j = e % DB;
+            const float b_i = __shfl_sync(0xffffffffu, beta, i);
+            A[e] = j < i ? b_i * between(i, j) * kk[i][j] : 0.0f;
+        }
+        __syncwarp();
+        if (lane < DB) {  // column `lane` of (I + A)^-1
+            float x[DB];
+#pragma unroll
+            for (int i = 0; i < DB; ++i) {
+                x[i] = i == lane ? 1.0f : 0.0f;
+#pragma unroll
+                for (int j = 0; j < i; ++j) x[i] = fmaf(-A[i * DB + j], x[j], x[i]);
+                T[i * DB + lane] = x[i];
+            }
+        }
+        __syncwarp();
+        float* out = a.coef + ((size_t)h * a.blocks + blk) * DC;
+#pragma unroll
+        for (int e = lane; e < DB * DB; e += 32) {
+            const int i = e / DB, j = e % DB;
+            out[e] = between(DB - 1, i) * T[e];
+            float m = 0.0f;
+            for (int l = j; l <= i; ++l) m = fmaf(between(i, l) * qk[i][l], T[l * DB + j], m);
+            out[DB * DB + e] = m;
+        }
+        if (lane < DB) {
+            const float so_far = between(lane, -1);
+            out[2 * DB * DB + lane] = beta * so_far;
+            out[2 * DB * DB + DB + lane] = so_far;
+            if (lane == DB - 1) out[2 * DB * DB + 2 * DB] = so_far;
+        }
+        const AT* vp = (const AT*)a.v + (size_t)base * a.v_ld + (size_t)h * a.vdim;
+        float* bv = a.bv + ((size_t)h * a.blocks + blk) * a.chunks * DB * DB;
+        for (int t = 0; t < DB; ++t) {
+            const float b_t = __shfl_sync(0xffffffffu, beta, t);
+            for (int c = lane; c < a.chunks * DB; c += 32)
+                bv[(c / DB) * DB * DB + t * DB + c % DB] = t < count && c < a.vdim ? b_t * to_f32(vp[(size_t)t * a.v_ld + c]) : 0.0f;
+        }
+        __syncwarp();
     }
 }
 
-template <typename AT>
-int launch_delta_rule(const DeltaArgs& args, int num_seqs, int sm_count, cudaStream_t stream) {
-    DeltaArgs a = args;
-    const int rpt = (a.dim + 31) / 32 * 4;  // key rows in runs of 32: four to each of a column's eight lanes
-    // value columns per CTA: fewer while SMs would stay idle, but at least 16 (every CTA's staging
-    // warps bring and normalise its head's keys and queries themselves), or what the head has
-    int cols = rpt > 16 ? 16 : rpt > 8 ? 32 : 64;  // (the registers of a lane bound the block)
-    while (cols > 16 && (long long)a.heads * num_seqs * ((a.vdim + cols - 1) / cols) < sm_count) cols /= 2;
-    while (cols > 8 && cols / 2 >= a.vdim) cols /= 2;
-    a.cols = cols;
-    const int epv = 16 / (int)sizeof(AT);
-    a.bulk = a.dim % epv == 0 && a.vdim % epv == 0 && a.q_ld % epv == 0 && a.k_ld % epv == 0 && a.v_ld % epv == 0 &&
-             (((uintptr_t)a.q | (uintptr_t)a.k | (uintptr_t)a.v) & 15) == 0;
-    const dim3 grid(a.heads, num_seqs, (a.vdim + cols - 1) / cols), block(cols * 8 + DR_STAGERS);
-#define DR_CASE(R)                                                                                                    \
-    if (rpt <= R) {                                                                                                   \
-        const size_t smem = (size_t)2 * DR_ROWS * (2 * 8 * R + cols + 4 + cols) * sizeof(float) +                     \
-                            (size_t)2 * DR_ROWS * (2 * a.dim + cols) * sizeof(AT);                                    \
-        auto kern = delta_rule_kernel<AT, R>;                                                                         \
-        if (smem > 48 * 1024) cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);    \
-        launch_kernel(kern, grid, block, smem, stream, a);                                                            \
-        return launch_status();                                                                                       \
+// --------------------------------------------------------------------------- the state, block after block
+
+struct BlocksArgs {
+    const float *kq, *coef, *bv;
+    float* state;
+    long long slot_stride;
+    const int *q_start, *state_slots;
+    float* out;  // [T, heads * vdim]
+    int blocks, heads, groups, dim, vdim, chunks;
+    int wide;  // a state row's four neighbouring columns may be moved at once
+};
+
+constexpr int D_STAGES = 3;
+
+// RPL: key rows a lane holds; 16 lanes hold four columns, a warp eight (a chunk), rows 64 j + 4 lane .. + 3.
+template <int RPL>
+__global__ void __launch_bounds__(256) delta_blocks_kernel(const BlocksArgs a) {
+    constexpr int DP = 16 * RPL, KQ = 2 * DB * DP;
+    const int h = blockIdx.x, s = blockIdx.y, warps = blockDim.x >> 5;
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, quad = lane >> 4, l16 = lane & 15;
+    const int chunk0 = blockIdx.z * warps, chunk = chunk0 + warp;
+    const int col0 = chunk * DB + quad * 4;
+    const int dim = a.dim, vdim = a.vdim, g = h / (a.heads / a.groups);
+    extern __shared__ __align__(16) float sm[];
+    const int stage_floats = KQ + DC + warps * DB * DB;
+    float* wsm = sm + D_STAGES * stage_floats + warp * 3 * DB * DB;  // this warp's w: [8 columns][8 rows]
+    float* usm = wsm + DB * DB;                                      // and D_8 u: [8 rows][8 columns] twice over, (u, u)
+    pdl_wait();
+    const int first = a.q_start[s], n = a.q_start[s + 1] - first;
+    if (n <= 0) return;
+    const int nb = (n + DB - 1) / DB;
+    const size_t blk0 = (size_t)first_block(a.q_start, s);
+    const float* kq_src = a.kq + ((size_t)g * a.blocks + blk0) * KQ;
+    const float* coef_src = a.coef + ((size_t)h * a.blocks + blk0) * DC;
+    const float* bv_src = a.bv + (((size_t)h * a.blocks + blk0) * a.chunks + chunk0) * DB * DB;
+    const int my_chunks = min(warps, a.chunks - chunk0);
+    auto load = [&](int b) {
+        if (b < nb) {
+            float* st = sm + (b % D_STAGES) * stage_floats;
+            const float* src = kq_src + (size_t)b * KQ;
+            for (int i = threadIdx.x; i < KQ / 4; i += blockDim.x) cp16(st + 4 * i, src + 4 * i);
+            src = coef_src + (size_t)b * DC;
+            for (int i = threadIdx.x; i < DC / 4; i += blockDim.x) cp16(st + KQ + 4 * i, src + 4 * i);
+            src = bv_src + (size_t)b * a.chunks * DB * DB;
+            for (int i = threadIdx.x; i < my_chunks * DB * DB / 4; i += blockDim.x) cp16(st + KQ + DC + 4 * i, src + 4 * i);
+        }
+        asm volatile("cp.async.commit_group;" ::: "memory");
+    };
+#pragma unroll
+    for (int b = 0; b < D_STAGES - 1; ++b) load(b);
+
+    const bool live = chunk < a.chunks && col0 < vdim;
+    float* slot = a.state + (size_t)a.state_slots[s] * a.slot_stride + (size_t)h * dim * vdim;
+    uint64_t S[4][RPL / 2];
+#pragma unroll
+    for (int r = 0; r < RPL; r += 2) {
+        float v[2][4];
+#pragma unroll
+        for (int e = 0; e < 2; ++e) {
+            const int row = (r >> 2) * 64 + l16 * 4 + (r & 3) + e;
+            v[e][0] = v[e][1] = v[e][2] = v[e][3] = 0.0f;
+            if (live && row < dim) {
+                if (a.wide) {
+                    const float4 x = *reinterpret_cast<const float4*>(slot + (size_t)row * vdim + col0);
+                    v[e][0] = x.x, v[e][1] = x.y, v[e][2] = x.z, v[e][3] = x.w;
+                } else {
+#pragma unroll
+                    for (int c = 0; c < 4; ++c)
+                        if (col0 + c < vdim) v[e][c] = slot[(size_t)row * vdim + col0 + c];
+                }
+            }
+        }
+#pragma unroll
+        for (int c = 0; c < 4; ++c) S[c][r / 2] = pair_of(v[0][c], v[1][c]);
     }
-    DR_CASE(4) DR_CASE(8) DR_CASE(12) DR_CASE(16) DR_CASE(24) DR_CASE(32)
-#undef DR_CASE
-    return SHISO_ERR_SHAPE;
+    const int tok = l16 >> 1, pair_col = quad * 4 + (l16 & 1) * 2;  // this lane's row and two columns of the chunk between exchange and update
+    const int out_col = chunk * DB + pair_col;
+    float* out = a.out + (size_t)first * a.heads * vdim + (size_t)h * vdim + out_col;
+    const bool out_pair = (vdim & 1) == 0;
+
+    for (int b = 0; b < nb; ++b) {
+        asm volatile("cp.async.wait_group %0;" ::"n"(D_STAGES - 2) : "memory");
+        __syncthreads();  // block b has landed for everybody, and nobody reads block b - 1 any more
+        load(b + D_STAGES - 1);
+        const float* st = sm + (b % D_STAGES) * stage_floats;
+        const ulonglong2* kt = reinterpret_cast<const ulonglong2*>(st) + l16;  // row t's piece j: kt[t * DP / 4 + 16 j]
+        const ulonglong2* qt = kt + DB * DP / 4;
+        const float* coef = st + KQ;
+        if (chunk < a.chunks) {
+            // ---- S^T k and S^T q of the eight rows: this lane's share of 8 x 4 columns x 2
+            float val[64];
+#pragma unroll
+            for (int t = 0; t < DB; ++t) {
+                uint64_t K[RPL / 2], Q[RPL / 2];
+#pragma unroll
+                for (int j = 0; j < RPL / 4; ++j) {
+                    const ulonglong2 k2 = kt[t * (DP / 4) + 16 * j], q2 = qt[t * (DP / 4) + 16 * j];
+                    K[2 * j] = k2.x, K[2 * j + 1] = k2.y;
+                    Q[2 * j] = q2.x, Q[2 * j + 1] = q2.y;
+                }
+#pragma unroll
+                for (int c = 0; c < 4; ++c) {
+                    uint64_t p = mul2(S[c][0], K[0]), r = mul2(S[c][0], Q[0]);
+#pragma unroll
+                    for (int j = 1; j < RPL / 2; ++j) {
+                        p = fma2(S[c][j], K[j], p);
+                        r = fma2(S[c][j], Q[j], r);
+                    }
+                    float lo, hi;
+                    halves_of(p, lo, hi);
+                    val[(t * 4 + c) * 2] = lo + hi;
+                    halves_of(r, lo, hi);
+                    val[(t * 4 + c) * 2 + 1] = lo + hi;
+                }
+            }
+            // ---- one exchange: every step sends half of what a lane still holds; lane l ends up with the sums 4 l .. 4 l + 3
+#pragma unroll
+            for (int o = 8; o > 0; o >>= 1) {
+                const bool upper = (l16 & o) != 0;
+#pragma unroll
+                for (int i = 0; i < 4 * o; ++i) {
+                    const float keep = upper ? val[i + 4 * o] : val[i], send = upper ? val[i] : val[i + 4 * o];
+                    val[i] = keep + __shfl_xor_sync(0xffffffffu, send, o);
+                }
+            }
+            // ---- the triangles: row `tok`, two columns
+            const float2 bv = *reinterpret_cast<const float2*>(st + KQ + DC + warp * DB * DB + tok * DB + pair_col);
+            const float bg = coef[2 * DB * DB + tok], so_far = coef[2 * DB * DB + DB + tok];
+            wsm[pair_col * DB + tok] = fmaf(-bg, val[0], bv.x);
+            wsm[(pair_col + 1) * DB + tok] = fmaf(-bg, val[2], bv.y);
+            __syncwarp();
+            float u0 = 0.0f, u1 = 0.0f, o0 = so_far * val[1], o1 = so_far * val[3];
+            const float4* t4 = reinterpret_cast<const float4*>(coef + tok * DB);
+            const float4* m4 = reinterpret_cast<const float4*>(coef + DB * DB + tok * DB);
+            const float4* w0 = reinterpret_cast<const float4*>(wsm + pair_col * DB);
+            const float4* w1 = w0 + DB / 4;
+#pragma unroll
+            for (int j = 0; j < DB / 4; ++j) {
+                const float4 t = t4[j], m = m4[j], x = w0[j], y = w1[j];
+                u0 = fmaf(t.x, x.x, fmaf(t.y, x.y, fmaf(t.z, x.z, fmaf(t.w, x.w, u0))));
+                u1 = fmaf(t.x, y.x, fmaf(t.y, y.y, fmaf(t.z, y.z, fmaf(t.w, y.w, u1))));
+                o0 = fmaf(m.x, x.x, fmaf(m.y, x.y, fmaf(m.z, x.z, fmaf(m.w, x.w, o0))));
+                o1 = fmaf(m.x, y.x, fmaf(m.y, y.y, fmaf(m.z, y.z, fmaf(m.w, y.w, o1))));
+            }
+            *reinterpret_cast<float4*>(usm + (tok * DB + pair_col) * 2) = make_float4(u0, u0, u1, u1);
+            if (b * DB + tok < n) {
+                float* o = out + (size_t)(b * DB + tok) * a.heads * vdim;
+                if (out_pair && out_col < vdim) {
+                    *reinterpret_cast<float2*>(o) = make_float2(o0, o1);
+                } else {
+                    if (out_col < vdim) o[0] = o0;
+                    if (out_col + 1 < vdim) o[1] = o1;
+                }
+            }
+            __syncwarp();
+            // ---- the state
+            const float last = coef[2 * DB * DB + 2 * DB];
+            const uint64_t last2 = pair_of(last, last);
+#pragma unroll
+            for (int c = 0; c < 4; ++c)
+#pragma unroll
+                for (int j = 0; j < RPL / 2; ++j) S[c][j] = mul2(S[c][j], last2);
+#pragma unroll
+            for (int t = 0; t < DB; ++t) {
+                const ulonglong2* up = reinterpret_cast<const ulonglong2*>(usm + (t * DB + quad * 4) * 2);
+                const ulonglong2 ua = up[0], ub = up[1];
+                const uint64_t u[4] = {ua.x, ua.y, ub.x, ub.y};
+#pragma unroll
+                for (int j = 0; j < RPL / 4; ++j) {
+                    const ulonglong2 k2 = kt[t * (DP / 4) + 16 * j];
+#pragma unroll
+                    for (int c = 0; c < 4; ++c) {
+                        S[c][2 * j] = fma2(k2.x, u[c], S[c][2 * j]);
+                        S[c][2 * j + 1] = fma2(k2.y, u[c], S[c][2 * j + 1]);
+                    }
+                }
+            }
+        }
+    }
+    pdl_trigger();
+    if (!live) return;
+#pragma unroll
+    for (int r = 0; r < RPL; r += 2) {
+        float v[2][4];
+#pragma unroll
+        for (int c = 0; c < 4; ++c) halves_of(S[c][r / 2], v[0][c], v[1][c]);
+#pragma unroll
+        for (int e = 0; e < 2; ++e) {
+            const int row = (r >> 2) * 64 + l16 * 4 + (r & 3) + e;
+            if (row >= dim) continue;
+            if (a.wide) {
+                *reinterpret_cast<float4*>(slot + (size_t)row * vdim + col0) = make_float4(v[e][0], v[e][1], v[e][2], v[e][3]);
+            } else {
+#pragma unroll
+                for (int c = 0; c < 4; ++c)
+                    if (col0 + c < vdim) slot[(size_t)row * vdim + col0 + c] = v[e][c];
+            }
+        }
+    }
+}
+
+template <int RPL>
+int launch_delta_blocks(const BlocksArgs& a, int num_seqs, int sm_count, cudaStream_t stream) {
+    // a CTA's warps share the keys and queries they read: as many as leave a CTA for every SM, at least two
+    int warps = 8;
+    while (warps > 2 && (long long)a.heads * num_seqs * ((a.chunks + warps - 1) / warps) < sm_count) warps /= 2;
+    while (warps > 1 && warps / 2 >= a.chunks) warps /= 2;
+    const size_t smem = (size_t)(D_STAGES * (2 * DB * 16 * RPL + DC + warps * DB * DB) + warps * 3 * DB * DB) * sizeof(float);
+    auto kern = delta_blocks_kernel<RPL>;
+    if (smem > 48 * 1024) cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+    launch_kernel(kern, dim3(a.heads, num_seqs, (a.chunks + warps - 1) / warps), dim3(warps * 32), smem, stream, a);
+    return launch_status();
+}
+
+// --------------------------------------------------------------------------- steps of single rows
+
+struct StepArgs {
+    const void *x, *gate, *b, *a;  // x: the columns [q | k | v] before their convolution
+    long long ld;                  // between two rows of all four
+    const float *taps, *dt_bias, *a_log, *norm_w;
+    float *window, *state;
+    long long window_stride, slot_stride;
+    const int *q_start, *state_slots;
+    void* out;
+    long long out_ld;
+    int heads, groups, dim, vdim, n_taps;
+    float q_scale, unit_eps, eps;
+};
+
+constexpr int DS_THREADS = 256;
+constexpr int DS_HELD = 16;  // state rows a thread keeps between its two passes
+
+// One CTA per (group, sequence): the group's q and k channels and its heads' v channels are nobody
+// else's, so their windows move on here.  N: value columns a thread takes at once.
+template <typename AT, int N>
+__global__ void __launch_bounds__(DS_THREADS) delta_step_kernel(const StepArgs a) {
+    __shared__ float scratch[33];
+    __shared__ float red[2][DS_THREADS * N];
+    extern __shared__ __align__(16) float ch[];  // q [dim], k [dim], v [heads of the group][vdim], then u and o of a head [vdim] each
+    pdl_wait();
+    const int g = blockIdx.x, s = blockIdx.y, tid = threadIdx.x;
+    const int row = a.q_start[s];
+    if (a.q_start[s + 1] <= row) return;
+    const int dim = a.dim, vdim = a.vdim, per = a.heads / a.groups, channels = 2 * a.groups * dim + a.heads * vdim;
+    const int slot = a.state_slots[s], mine = 2 * dim + per * vdim;
+    float* su = ch + mine;
+    float* so = su + vdim;
+    const AT* x = (const AT*)a.x + (size_t)row * a.ld;
+    float* window = a.window + (size_t)slot * a.window_stride;
+    float qq = 0.0f, kn = 0.0f;
+    for (int i = tid; i < mine; i += DS_THREADS) {
+        const int c = i < dim ? g * dim + i : i < 2 * dim ? (a.groups + g) * dim + i - dim : 2 * a.groups * dim + g * per * vdim + i - 2 * dim;
+        const float* taps = a.taps + (size_t)c * a.n_taps;
+        const float in = to_f32(x[c]);
+        float acc = taps[a.n_taps - 1] * in;
+        for (int j = 0; j < a.n_taps - 1; ++j) {
+            float* at = window + (size_t)j * channels + c;
+            acc = fmaf(taps[j], *at, acc);
+            if (j > 0) at[-(long long)channels] = *at;
+        }
+        window[(size_t)(a.n_taps - 2) * channels + c] = in;
+        acc = to_f32(from_f32<AT>(silu_of(acc)));  // (rounded where the convolution's own kernel rounds)
+        ch[i] = acc;
+        if (i < dim) qq += acc * acc;
+        else if (i < 2 * dim) kn += acc * acc;
+    }
+    qq = block_sum(qq, scratch);
+    kn = block_sum(kn, scratch);
+    const float iq = rsqrtf(qq + a.unit_eps) * a.q_scale, ik = rsqrtf(kn + a.unit_eps);
+    float qk = 0.0f;
+    for (int i = tid; i < dim; i += DS_THREADS) {
+        const float q = ch[i] * iq, k = ch[dim + i] * ik;
+        ch[i] = q;
+        ch[dim + i] = k;
+        qk += q * k;
+    }
+    qk = block_sum(qk, scratch);  // (its barriers stand between the writes above and the reads below)
+    const float *sq = ch, *sk = ch + dim;
+    const int spans = (vdim + N - 1) / N;
+    const int lanes = min(spans, DS_THREADS), parts = DS_THREADS / lanes;  // threads over the columns, and shares of the key rows
+    const int span = tid % lanes, part = tid / lanes;
+    for (int hh = 0; hh < per; ++hh) {
+        const int h = g * per + hh;
+        const float decay = decay_of(to_f32(((const AT*)a.a)[(size_t)row * a.ld + h]), a.dt_bias[h], expf(a.a_log[h]));
+        const float beta = sigmoid_of(to_f32(((const AT*)a.b)[(size_t)row * a.ld + h]));
+        const float* sv = ch + 2 * dim + hh * vdim;
+        float* S = a.state + (size_t)slot * a.slot_stride + (size_t)h * dim * vdim;
+        for (int base = 0; base < spans; base += lanes) {
+            const int c0 = (base + span) * N;
+            const bool live = part < parts && base + span < spans;
+            auto fetch = [&](int r, float (&v)[N]) {
+                if constexpr (N == 4) {
+                    const float4 f = *reinterpret_cast<const float4*>(S + (size_t)r * vdim + c0);
+                    v[0] = f.x, v[1] = f.y, v[2] = f.z, v[3] = f.w;
+                } else {
+                    v[0] = S[(size_t)r * vdim + c0];
+                }
+            };
+            float held[DS_HELD][N], p[N], o[N];
+#pragma unroll
+            for (int e = 0; e < N; ++e) p[e] = o[e] = 0.0f;
+            if (live) {
+#pragma unroll
+                for (int i = 0; i < DS_HELD; ++i) {
+                    const int r = part + i * parts;
+#pragma unroll
+                    for (int e = 0; e < N; ++e) held[i][e] = 0.0f;
+                    if (r < dim) fetch(r, held[i]);
+                }
+#pragma unroll
+                for (int i = 0; i < DS_HELD; ++i) {
+                    const int r = part + i * parts;
+                    const float k = r < dim ? sk[r] : 0.0f, q = r < dim ? sq[r] : 0.0f;
+#pragma unroll
+                    for (int e = 0; e < N; ++e) p[e] = fmaf(held[i][e], k, p[e]), o[e] = fmaf(held[i][e], q, o[e]);
+                }
+                for (int r = part + DS_HELD * parts; r < dim; r += parts) {
+                    float v[N];
+                    fetch(r, v);
+#pragma unroll
+                    for (int e = 0; e < N; ++e) p[e] = fmaf(v[e], sk[r], p[e]), o[e] = fmaf(v[e], sq[r], o[e]);
+                }
+#pragma unroll
+                for (int e = 0; e < N; ++e) red[0][(part * lanes + span) * N + e] = p[e], red[1][(part * lanes + span) * N + e] = o[e];
+            }
+            __syncthreads();
+            for (int i = tid; i < lanes * N; i += DS_THREADS) {
+                const int c = base * N + i;
+                if (c >= vdim) continue;
+                float ps = 0.0f, os = 0.0f;
+                for (int j = 0; j < parts; ++j) ps += red[0][j * lanes * N + i], os += red[1][j * lanes * N + i];
+                const float u = beta * fmaf(-decay, ps, sv[c]);
+                su[c] = u;
+                so[c] = fmaf(u, qk, decay * os);
+            }
+            __syncthreads();
+            if (live) {
+                float u[N];
+#pragma unroll
+                for (int e = 0; e < N; ++e) u[e] = su[c0 + e];
+                auto put = [&](int r, const float (&v)[N]) {
+                    const float k = sk[r];
+                    if constexpr (N == 4)
+                        *reinterpret_cast<float4*>(S + (size_t)r * vdim + c0) =
+                            make_float4(fmaf(k, u[0], decay * v[0]), fmaf(k, u[1], decay * v[1]), fmaf(k, u[2], decay * v[2]), fmaf(k, u[3], decay * v[3]));
+                    else
+                        S[(size_t)r * vdim + c0] = fmaf(k, u[0], decay * v[0]);
+                };
+#pragma unroll
+                for (int i = 0; i < DS_HELD; ++i) {
+                    const int r = part + i * parts;
+                    if (r < dim) put(r, held[i]);
+                }
+                for (int r = part + DS_HELD * parts; r < dim; r += parts) {
+                    float v[N];
+                    fetch(r, v);
+                    put(r, v);
+                }
+            }
+        }
+        // the head's output norm and gate
+        float ss = 0.0f;
+        for (int c = tid; c < vdim; c += DS_THREADS) ss += so[c] * so[c];
+        const float inv = rsqrtf(block_sum(ss, scratch) / (float)vdim + a.eps);
+        const AT* gate = (const AT*)a.gate + (size_t)row * a.ld + (size_t)h * vdim;
+        AT* out = (AT*)a.out + (size_t)row * a.out_ld + (size_t)h * vdim;
+        for (int c = tid; c < vdim; c += DS_THREADS) out[c] = from_f32<AT>(so[c] * inv * a.norm_w[c] * silu_of(to_f32(gate[c])));
+        __syncthreads();  // u, o and the shares are written again by the next head
+    }
+    pdl_trigger();
+}
+
+template <typename AT>
+int launch_delta_step(const StepArgs& a, int num_seqs, cudaStream_t stream) {
+    const size_t smem = (size_t)(2 * a.dim + (a.heads / a.groups + 2) * a.vdim) * sizeof(float);
+    if (smem > 160 * 1024) return SHISO_ERR_SHAPE;
+    const bool wide = a.vdim % 4 == 0 && a.slot_stride % 4 == 0 && ((uintptr_t)a.state & 15) == 0;
+    auto kern = wide ? delta_step_kernel<AT, 4> : delta_step_kernel<AT, 1>;
+    if (smem > 32 * 1024) cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+    launch_kernel(kern, dim3(a.groups, num_seqs), dim3(DS_THREADS), smem, stream, a);
+    return launch_status();
 }
 
 // --------------------------------------------------------------------------- output norm and gate
@@ -358,19 +649,54 @@ delta_output_kernel(const float* __restrict__ x, const AT* __restrict__ gate, lo
 
 }  // namespace
 
+
 // q, k [T, groups * dim], v [T, heads * vdim], b, a [T, heads] (rows may be strided, `*_ld` elements
-// apart); state float [slots, heads, dim, vdim]; out float [T, heads * vdim].
+// apart); state float [slots, heads, dim, vdim]; out float [T, heads * vdim]; scratch: 16-byte aligned.
 SHISO_API int shiso_delta_rule(const void* q, const void* k, const void* v, const void* b, const void* a_logit, long long q_ld,
                                long long k_ld, long long v_ld, long long b_ld, long long a_ld, int act_dtype, const float* dt_bias,
                                const float* a_log, float* state, long long slot_stride, const int* q_start, const int* state_slots,
-                               float* out, int tokens, int num_seqs, int heads, int groups, int dim, int vdim, float q_scale,
-                               float unit_eps, int sm_count, cudaStream_t stream) {
+                               float* scratch, float* out, int tokens, int num_seqs, int heads, int groups, int dim, int vdim,
+                               float q_scale, float unit_eps, int sm_count, cudaStream_t stream) {
     if (tokens <= 0 || num_seqs <= 0) return SHISO_OK;
-    if (heads <= 0 || groups <= 0 || heads % groups || dim <= 0 || dim > 256 || vdim <= 0 || num_seqs > 65535) return SHISO_ERR_SHAPE;
-    const DeltaArgs args = {q, k, v, b, a_logit, q_ld, k_ld, v_ld, b_ld, a_ld, dt_bias, a_log, state, slot_stride,
-                            q_start, state_slots, out, heads, groups, dim, vdim, 0, 0, q_scale, unit_eps};
-    if (act_dtype == SHISO_F32) return launch_delta_rule<float>(args, num_seqs, sm_count, stream);
-    if (act_dtype == SHISO_BF16) return launch_delta_rule<__nv_bfloat16>(args, num_seqs, sm_count, stream);
+    if (heads <= 0 || groups <= 0 || heads % groups || dim <= 0 || dim > D_MAX_DIM || vdim <= 0 || num_seqs > 65535 || groups > 65535)
+        return SHISO_ERR_SHAPE;
+    if (((uintptr_t)scratch | (uintptr_t)out) & 15) return SHISO_ERR_ALIGN;
+    const int blocks = tokens / DB + num_seqs, dp = (dim + 63) / 64 * 64, chunks = (vdim + DB - 1) / DB;
+    float* kq = scratch;
+    float* coef = kq + (size_t)groups * blocks * 2 * DB * dp;
+    float* bv = coef + (size_t)heads * blocks * DC;
+    const PrepareArgs prep = {q, k, v, b, a_logit, q_ld, k_ld, v_ld, b_ld, a_ld, dt_bias, a_log, q_start, kq, coef, bv,
+                              num_seqs, blocks, heads, groups, dim, dp, vdim, chunks, q_scale, unit_eps};
+    const dim3 grid(blocks, groups);
+    if (act_dtype == SHISO_F32) launch_kernel(delta_prepare_kernel<float>, grid, DB * 32, 0, stream, prep);
+    else if (act_dtype == SHISO_BF16) launch_kernel(delta_prepare_kernel<__nv_bfloat16>, grid, DB * 32, 0, stream, prep);
+    else return SHISO_ERR_DTYPE;
+    const int status = launch_status();
+    if (status != SHISO_OK) return status;
+    const int wide = vdim % 4 == 0 && slot_stride % 4 == 0 && ((uintptr_t)state & 15) == 0;
+    const BlocksArgs walk = {kq, coef, bv, state, slot_stride, q_start, state_slots, out, blocks, heads, groups, dim, vdim, chunks, wide};
+    switch (dp) {
+        case 64: return launch_delta_blocks<4>(walk, num_seqs, sm_count, stream);
+        case 128: return launch_delta_blocks<8>(walk, num_seqs, sm_count, stream);
+        case 192: return launch_delta_blocks<12>(walk, num_seqs, sm_count, stream);
+        default: return launch_delta_blocks<16>(walk, num_seqs, sm_count, stream);
+    }
+}
+
+// A step of one row per sequence.  x: the columns [q | k | v] of the projected rows, gate, b and a further
+// columns of the same rows (`ld` elements apart); taps float [channels, n_taps]; window float
+// [slots, n_taps - 1, channels]; out [T, heads * vdim], rows out_ld apart.
+SHISO_API int shiso_delta_step(const void* x, const void* gate, const void* b, const void* a_logit, long long ld, int act_dtype,
+                               const float* taps, const float* dt_bias, const float* a_log, const float* norm_w, float* window,
+                               long long window_stride, float* state, long long slot_stride, const int* q_start,
+                               const int* state_slots, void* out, long long out_ld, int num_seqs, int heads, int groups, int dim,
+                               int vdim, int n_taps, float q_scale, float unit_eps, float eps, cudaStream_t stream) {
+    if (num_seqs <= 0) return SHISO_OK;
+    if (heads <= 0 || groups <= 0 || heads % groups || dim <= 0 || vdim <= 0 || n_taps < 2 || num_seqs > 65535) return SHISO_ERR_SHAPE;
+    const StepArgs args = {x, gate, b, a_logit, ld, taps, dt_bias, a_log, norm_w, window, state, window_stride, slot_stride, q_start,
+                           state_slots, out, out_ld, heads, groups, dim, vdim, n_taps, q_scale, unit_eps, eps};
+    if (act_dtype == SHISO_F32) return launch_delta_step<float>(args, num_seqs, stream);
+    if (act_dtype == SHISO_BF16) return launch_delta_step<__nv_bfloat16>(args, num_seqs, stream);
     return SHISO_ERR_DTYPE;
 }
 

@@ -102,7 +102,8 @@ _SIGNATURES = {
     "shiso_joined_norm_store": [P, LL, I, I, I, I, I, P, P, P, P, P, I, P, P, I, I, F, F, I, P, I, I, P],
     "shiso_stream_concat": [P, P, I, P, I, P, P, I, I, I, P],
     "shiso_normed_pair": [P, P, I, P, P, F, F, P, P, P, F, P, P, I, I, P],
-    "shiso_delta_rule": [P, P, P, P, P, LL, LL, LL, LL, LL, I, P, P, P, LL, P, P, P, I, I, I, I, I, I, F, F, I, P],
+    "shiso_delta_step": [P, P, P, P, LL, I, P, P, P, P, P, LL, P, LL, P, P, P, LL, I, I, I, I, I, I, F, F, F, P],
+    "shiso_delta_rule": [P, P, P, P, P, LL, LL, LL, LL, LL, I, P, P, P, LL, P, P, P, P, I, I, I, I, I, I, F, F, I, P],
     "shiso_delta_output": [P, P, LL, I, P, P, LL, I, I, I, F, P],
 }
 

@@ -1689,7 +1689,7 @@ def delta_rule(q, k, v, b, a, dt_bias, a_log, state, step, heads, groups, dim, v
     (``x / sqrt(sum x^2 + unit_eps)``, q times ``q_scale`` too), head ``h`` reading group
     ``h // (heads / groups)``; ``v [T, heads * vdim]``; ``beta = sigmoid(b)``, ``g = exp(-exp(a_log)
     softplus(a + dt_bias))`` from ``b, a [T, heads]``.  All may be column ranges.  Returns float32
-    ``[T, heads * vdim]``."""
+    ``[T, heads * vdim]``.  Two launches: what couples eight neighbouring rows, then the state."""
     act = q.dtype
     tokens = q.shape[0]
     q_ld, k_ld = _rows(q, "q", act, groups * dim), _rows(k, "k", act, groups * dim)
@@ -1703,12 +1703,46 @@ def delta_rule(q, k, v, b, a, dt_bias, a_log, state, step, heads, groups, dim, v
         if t.shape[0] != heads:
             raise KernelError(f"{name} has {t.shape[0]} entries for {heads} heads")
     out = torch.empty((tokens, heads * vdim), dtype=torch.float32, device=q.device)
+    blocks, padded, chunks = tokens // 8 + step.num_seqs, -(-dim // 64) * 64, -(-vdim // 8)  # (as the kernels lay it out)
+    scratch = torch.empty((blocks * (groups * 16 * padded + heads * (148 + chunks * 64)),), dtype=torch.float32, device=q.device)
     status = library().shiso_delta_rule(
         q.data_ptr(), k.data_ptr(), v.data_ptr(), b.data_ptr(), a.data_ptr(), q_ld, k_ld, v_ld, b_ld, a_ld, _CODES[act], _ptr(dt_bias),
-        _ptr(a_log), state.data_ptr(), stride, _ptr(step.q_start), _ptr(step.state_slots), _ptr(out), tokens, step.num_seqs, heads,
+        _ptr(a_log), state.data_ptr(), stride, _ptr(step.q_start), _ptr(step.state_slots), _ptr(scratch), _ptr(out), tokens, step.num_seqs, heads,
         groups, dim, vdim, float(q_scale), float(unit_eps), _sm_count(), _stream(),
     )
-    _done(status, "delta_rule", shape=(tokens, heads, dim, vdim))
+    _done(status, "delta_rule", 2, shape=(tokens, heads, dim, vdim))
+    return out
+
+
+def delta_step(proj, conv_cols, taps, dt_bias, a_log, norm_w, window, state, step, heads, groups, dim, vdim, q_scale, unit_eps, eps, out):
+    """For a step of one row per sequence: ``causal_conv`` of the first ``conv_cols`` columns ``[q | k | v]`` of
+    ``proj[T, q | k | v | gate | b | a]`` (rows may be strided), ``delta_rule`` and ``delta_output`` in one
+    launch.  Writes ``out[T, heads * vdim]`` and returns it, or None (nothing done) for a step that holds
+    longer portions."""
+    if not getattr(step, "all_decode", False):
+        return None
+    act, tokens, v_cols = proj.dtype, proj.shape[0], heads * vdim
+    ld = _rows(proj, "projected rows", act, conv_cols + v_cols + 2 * heads)
+    out_ld = _rows(out, "out", act, v_cols)
+    if conv_cols != 2 * groups * dim + v_cols or out.shape[0] != tokens:
+        raise KernelError(f"{conv_cols} columns for {groups} heads of {dim} twice and {heads} of {vdim}")
+    for name, t, n in (("dt bias", dt_bias, heads), ("a_log", a_log, heads), ("norm weight", norm_w, vdim)):
+        _check(t, name, torch.float32, 1)
+        if t.shape[0] != n:
+            raise KernelError(f"{name} has {t.shape[0]} entries where {n} are expected")
+    _check(taps, "conv taps", torch.float32, 2)
+    n_taps = taps.shape[1]
+    if taps.shape[0] != conv_cols or window.shape[1:] != (n_taps - 1, conv_cols) or state.shape[1:] != (heads, dim, vdim):
+        raise KernelError(f"taps {tuple(taps.shape)}, window {tuple(window.shape)} and state {tuple(state.shape)} do not fit")
+    window_stride, slot_stride = _slot_rows(window, "conv state", torch.float32), _slot_rows(state, "recurrent state", torch.float32)
+    at, size = proj.data_ptr(), proj.element_size()
+    gate, b, a = (at + size * (conv_cols + o) for o in (0, v_cols, v_cols + heads))
+    status = library().shiso_delta_step(
+        at, gate, b, a, ld, _CODES[act], _ptr(taps), _ptr(dt_bias), _ptr(a_log), _ptr(norm_w), window.data_ptr(), window_stride,
+        state.data_ptr(), slot_stride, _ptr(step.q_start), _ptr(step.state_slots), out.data_ptr(), out_ld, step.num_seqs, heads, groups,
+        dim, vdim, n_taps, float(q_scale), float(unit_eps), float(eps), _stream(),
+    )
+    _done(status, "delta_step", shape=(tokens, heads, dim, vdim))
     return out
 
 

@@ -121,6 +121,12 @@ class GatedDelta(Mixer):
         ops = self.env.ops
         window, state = cache
         c, qk, v, h = self.conv_cols, self.qk_cols, self.v_cols, self.heads
+        in_one = getattr(ops, "delta_step", None)
+        if in_one is not None and in_one(
+            proj, c, self.conv, self.dt_bias, self.a_log, self.norm, window.state, state.state, step, self.heads, self.kv_heads,
+            self.dim, self.vdim, self.dim**-0.5, self.unit_eps, self.eps, out,
+        ) is not None:
+            return  # a step of single rows: everything in one launch
         gate, b, a = proj[:, c : c + v], proj[:, c + v : c + v + h], proj[:, c + v + h : c + v + 2 * h]
         qkv = ops.causal_conv(proj[:, :c], self.conv, None, window.state, step, silu=True)
         raw = ops.delta_rule(

@@ -164,8 +164,12 @@ def choose(logits, top):
     return order, z / z.sum()
 
 
-def mixture(tensors, prefix, mlp, h):
+def mixture(tensors, prefix, mlp, h, margins=None):
+    """``margins``, a list, gets per row how far the last chosen logit lies above the best one left out."""
     logits = h @ _w(tensors, f"{prefix}.router").T + _w(tensors, f"{prefix}.router.b")
+    if margins is not None:
+        ranked, top = torch.sort(logits, dim=-1, descending=True).values, mlp["router"]["top"]
+        margins.append(ranked[:, top - 1] - ranked[:, top] if top < logits.shape[1] else torch.full((h.shape[0],), float("inf"), dtype=F64))
     out = torch.zeros_like(h)
     for t in range(h.shape[0]):
         ids, weights = choose(logits[t], mlp["router"]["top"])
@@ -191,7 +195,7 @@ def run_order(document):
     return order + [(i, None) for i in range(loop["stop"], n)]
 
 
-def plain_layers(document, tensors, tokens, hook=None):
+def plain_layers(document, tensors, tokens, hook=None, margins=None):
     """The stream after the last layer; ``hook(run, x)`` sees it after every layer run."""
     eps = document["norm"]["eps"]
     x0 = tensors["embed"][torch.as_tensor(tokens)].to(F64) * (document.get("embedding") or {}).get("scale", 1.0)
@@ -202,12 +206,12 @@ def plain_layers(document, tensors, tokens, hook=None):
         layer = document["layers"][i]
         x = x + parallel_mixer(tensors, f"l{i}.mix", layer["mixer"], centred_norm(x, tensors, f"l{i}.norm1", eps), eps)
         if layer.get("mlp") is not None:
-            x = x + mixture(tensors, f"l{i}.mlp", layer["mlp"], centred_norm(x, tensors, f"l{i}.norm2", eps))
+            x = x + mixture(tensors, f"l{i}.mlp", layer["mlp"], centred_norm(x, tensors, f"l{i}.norm2", eps), margins)
         if hook is not None:
             hook(run, x)
     return x
 
 
-def plain_logits(document, tensors, tokens, hook=None):
-    x = plain_layers(document, tensors, tokens, hook)
+def plain_logits(document, tensors, tokens, hook=None, margins=None):
+    x = plain_layers(document, tensors, tokens, hook, margins)
     return centred_norm(x, tensors, "final.norm", document["norm"]["eps"]) @ _w(tensors, "head").T
