@@ -90,13 +90,13 @@ struct PrepareArgs {
     float q_scale, unit_eps;
 };
 
-template <typename AT>
+// PER: entries of a query or key a lane holds (dim in multiples of 32, divided by 32).
+template <typename AT, int PER>
 __global__ void __launch_bounds__(DB * 32) delta_prepare_kernel(const PrepareArgs a) {
-    constexpr int PER = D_MAX_DIM / 32;
-    __shared__ float ks[DB][D_MAX_DIM];
+    __shared__ float ks[DB][32 * PER];
     __shared__ float kk[DB][DB], qk[DB][DB];
-    __shared__ float tri[DB][DB * DB], inv[DB][DB * DB];  // per warp: A, then T, of the head it works on
-    __shared__ float gs[DB][DB];
+    __shared__ float gs[DB][DB], bs[DB][DB];               // decay and beta of eight heads' rows
+    __shared__ float sA[DB][DB * DB], sD[DB][DB * DB], sT[DB][DB * DB];  // a warp's head: A, D, (I + A)^-1
     __shared__ int s_seq;
     pdl_begin();
     const int blk = blockIdx.x, g = blockIdx.y, lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
@@ -109,6 +109,22 @@ __global__ void __launch_bounds__(DB * 32) delta_prepare_kernel(const PrepareArg
     if (s < 0) return;
     const int base = a.q_start[s] + (blk - first_block(a.q_start, s)) * DB;
     const int count = min(DB, a.q_start[s + 1] - base);
+    const int per = a.heads / a.groups;
+    // decays and betas of eight heads, a thread a (head, row); rows beyond the portion neither forget nor write
+    auto gates = [&](int hh0) {
+        const int hh = hh0 + threadIdx.x / DB, t = threadIdx.x % DB;
+        if (threadIdx.x < DB * DB && hh < per) {
+            const int h = g * per + hh;
+            float decay = 1.0f, beta = 0.0f;
+            if (t < count) {
+                decay = decay_of(to_f32(((const AT*)a.a)[((size_t)base + t) * a.a_ld + h]), a.dt_bias[h], expf(a.a_log[h]));
+                beta = sigmoid_of(to_f32(((const AT*)a.b)[((size_t)base + t) * a.b_ld + h]));
+            }
+            gs[hh - hh0][t] = decay;
+            bs[hh - hh0][t] = beta;
+        }
+    };
+    gates(0);
     // a warp a row: unit vectors (rows beyond the portion are zeros)
     const size_t row = (size_t)base + min(warp, count - 1);
     const bool mine = warp < count;
@@ -133,86 +149,113 @@ __global__ void __launch_bounds__(DB * 32) delta_prepare_kernel(const PrepareArg
         qv[i] *= iq;
         kv[i] *= ik;
         ks[warp][c] = kv[i];
-        if (c < a.dp) {
-            kq[warp * a.dp + c] = kv[i];
-            kq[(DB + warp) * a.dp + c] = qv[i];
-        }
+        kq[warp * a.dp + c] = kv[i];
+        kq[(DB + warp) * a.dp + c] = qv[i];
     }
+    for (int c = 32 * PER + lane; c < a.dp; c += 32) kq[warp * a.dp + c] = kq[(DB + warp) * a.dp + c] = 0.0f;
     __syncthreads();
-    // the products between the rows: warp i's row against rows j <= i
-    for (int j = 0; j <= warp; ++j) {
-        float x = 0.0f, y = 0.0f;
+    // the products between the rows, row `warp` against all eight: sixteen sums, one exchange (lane l
+    // ends up with sum l / 2: of k for l < 16, of q behind)
+    {
+        float x[2 * DB];
 #pragma unroll
-        for (int i = 0; i < PER; ++i) {
-            const float other = ks[j][lane + 32 * i];
-            x = fmaf(kv[i], other, x);
-            y = fmaf(qv[i], other, y);
-        }
-        x = warp_sum(x);
-        y = warp_sum(y);
-        if (lane == 0) kk[warp][j] = x, qk[warp][j] = y;
-    }
-    __syncthreads();
-    // a warp a head
-    const int per = a.heads / a.groups;
-    for (int hh = warp; hh < per; hh += DB) {
-        const int h = g * per + hh;
-        float decay = 1.0f, beta = 0.0f;
-        if (lane < count) {
-            decay = decay_of(to_f32(((const AT*)a.a)[((size_t)base + lane) * a.a_ld + h]), a.dt_bias[h], expf(a.a_log[h]));
-            beta = sigmoid_of(to_f32(((const AT*)a.b)[((size_t)base + lane) * a.b_ld + h]));
-        }
-        float* A = tri[warp];
-        float* T = inv[warp];
-        if (lane < DB) gs[warp][lane] = decay;
-        __syncwarp();
-        auto between = [&](int i, int j) {  // g_(j+1) .. g_i
-            float d = 1.0f;
-            for (int m = j + 1; m <= i; ++m) d *= gs[warp][m];
-            return d;
-        };
+        for (int j = 0; j < DB; ++j) {
+            x[j] = x[DB + j] = 0.0f;
 #pragma unroll
-        for (int e = lane; e < DB * DB; e += 32) {
-            const int i = e / DB, j = e % DB;
-            const float b_i = __shfl_sync(0xffffffffu, beta, i);
-            A[e] = j < i ? b_i * between(i, j) * kk[i][j] : 0.0f;
-        }
-        __syncwarp();
-        if (lane < DB) {  // column `lane` of (I + A)^-1
-            float x[DB];
-#pragma unroll
-            for (int i = 0; i < DB; ++i) {
-                x[i] = i == lane ? 1.0f : 0.0f;
-#pragma unroll
-                for (int j = 0; j < i; ++j) x[i] = fmaf(-A[i * DB + j], x[j], x[i]);
-                T[i * DB + lane] = x[i];
+            for (int i = 0; i < PER; ++i) {
+                const float other = ks[j][lane + 32 * i];
+                x[j] = fmaf(kv[i], other, x[j]);
+                x[DB + j] = fmaf(qv[i], other, x[DB + j]);
             }
         }
-        __syncwarp();
-        float* out = a.coef + ((size_t)h * a.blocks + blk) * DC;
 #pragma unroll
-        for (int e = lane; e < DB * DB; e += 32) {
-            const int i = e / DB, j = e % DB;
-            out[e] = between(DB - 1, i) * T[e];
-            float m = 0.0f;
-            for (int l = j; l <= i; ++l) m = fmaf(between(i, l) * qk[i][l], T[l * DB + j], m);
-            out[DB * DB + e] = m;
+        for (int o = 16; o > 1; o >>= 1) {
+            const bool upper = (lane & o) != 0;
+#pragma unroll
+            for (int i = 0; i < o / 2; ++i) {
+                const float keep = upper ? x[i + o / 2] : x[i], send = upper ? x[i] : x[i + o / 2];
+                x[i] = keep + __shfl_xor_sync(0xffffffffu, send, o);
+            }
         }
-        if (lane < DB) {
-            const float so_far = between(lane, -1);
-            out[2 * DB * DB + lane] = beta * so_far;
-            out[2 * DB * DB + DB + lane] = so_far;
-            if (lane == DB - 1) out[2 * DB * DB + 2 * DB] = so_far;
-        }
-        const AT* vp = (const AT*)a.v + (size_t)base * a.v_ld + (size_t)h * a.vdim;
-        float* bv = a.bv + ((size_t)h * a.blocks + blk) * a.chunks * DB * DB;
-        for (int t = 0; t < DB; ++t) {
-            const float b_t = __shfl_sync(0xffffffffu, beta, t);
-            for (int c = lane; c < a.chunks * DB; c += 32)
-                bv[(c / DB) * DB * DB + t * DB + c % DB] = t < count && c < a.vdim ? b_t * to_f32(vp[(size_t)t * a.v_ld + c]) : 0.0f;
-        }
-        __syncwarp();
+        const float sum = x[0] + __shfl_xor_sync(0xffffffffu, x[0], 1);
+        const int e = lane >> 1;
+        if ((lane & 1) == 0) (e < DB ? kk : qk)[warp][e % DB] = sum;
     }
+    for (int hh0 = 0; hh0 < per; hh0 += DB) {
+        if (hh0 > 0) {
+            __syncthreads();  // the heads before these are done with their gates
+            gates(hh0);
+        }
+        __syncthreads();
+        const int here = min(DB, per - hh0);
+        if (warp < here) {  // a warp a head
+            const int h = g * per + hh0 + warp;
+            float *A = sA[warp], *D = sD[warp], *T = sT[warp];
+            const float* gw = gs[warp];
+#pragma unroll
+            for (int e = lane; e < DB * DB; e += 32) {
+                const int i = e / DB, j = e % DB;
+                float d = 1.0f;  // g_(j+1) .. g_i
+#pragma unroll
+                for (int m = 1; m < DB; ++m)
+                    if (m > j && m <= i) d *= gw[m];
+                D[e] = d;
+                A[e] = j < i ? bs[warp][i] * d * kk[i][j] : 0.0f;
+            }
+            __syncwarp();
+            if (lane < DB) {  // column `lane` of (I + A)^-1
+                float x[DB];
+#pragma unroll
+                for (int i = 0; i < DB; ++i) {
+                    x[i] = i == lane ? 1.0f : 0.0f;
+#pragma unroll
+                    for (int j = 0; j < i; ++j) x[i] = fmaf(-A[i * DB + j], x[j], x[i]);
+                    T[i * DB + lane] = x[i];
+                }
+            }
+            __syncwarp();
+            float* out = a.coef + ((size_t)h * a.blocks + blk) * DC;
+#pragma unroll
+            for (int e = lane; e < DB * DB; e += 32) {
+                const int i = e / DB, j = e % DB;
+                out[e] = D[(DB - 1) * DB + i] * T[e];
+                float m = 0.0f;
+#pragma unroll
+                for (int l = 0; l < DB; ++l)  // (T is zero above the diagonal)
+                    if (l <= i) m = fmaf(D[i * DB + l] * qk[i][l], T[l * DB + j], m);
+                out[DB * DB + e] = m;
+            }
+            if (lane < DB) {
+                const float so_far = D[lane * DB] * gw[0];
+                out[2 * DB * DB + lane] = bs[warp][lane] * so_far;
+                out[2 * DB * DB + DB + lane] = so_far;
+                if (lane == DB - 1) out[2 * DB * DB + 2 * DB] = so_far;
+            }
+        }
+        // beta v of these heads, by everybody
+        for (int hh = 0; hh < here; ++hh) {
+            const int h = g * per + hh0 + hh;
+            const AT* vp = (const AT*)a.v + (size_t)base * a.v_ld + (size_t)h * a.vdim;
+            float* bv = a.bv + ((size_t)h * a.blocks + blk) * a.chunks * DB * DB;
+            for (int e = threadIdx.x; e < a.chunks * DB * DB; e += blockDim.x) {
+                const int t = e / (a.chunks * DB), c = e - t * a.chunks * DB;
+                bv[(c / DB) * DB * DB + t * DB + c % DB] = t < count && c < a.vdim ? bs[hh][t] * to_f32(vp[(size_t)t * a.v_ld + c]) : 0.0f;
+            }
+        }
+    }
+}
+
+template <typename AT>
+int launch_delta_prepare(const PrepareArgs& a, cudaStream_t stream) {
+    const dim3 grid(a.blocks, a.groups);
+    const int per = (a.dim + 31) / 32;
+#define DP_GO(P) launch_kernel(delta_prepare_kernel<AT, P>, grid, DB * 32, 0, stream, a)
+    if (per <= 1) DP_GO(1);
+    else if (per <= 2) DP_GO(2);
+    else if (per <= 4) DP_GO(4);
+    else DP_GO(8);
+#undef DP_GO
+    return launch_status();
 }
 
 // --------------------------------------------------------------------------- the state, block after block
@@ -229,19 +272,31 @@ struct BlocksArgs {
 
 constexpr int D_STAGES = 3;
 
-// RPL: key rows a lane holds; 16 lanes hold four columns, a warp eight (a chunk), rows 64 j + 4 lane .. + 3.
+// A run of RUN neighbouring floats as pairs.
+template <int RUN>
+__device__ __forceinline__ void read_run(const float* p, uint64_t* pairs) {
+    if constexpr (RUN == 4) {
+        const ulonglong2 v = *reinterpret_cast<const ulonglong2*>(p);
+        pairs[0] = v.x, pairs[1] = v.y;
+    } else {
+        pairs[0] = *reinterpret_cast<const uint64_t*>(p);
+    }
+}
+
+// RPL: key rows a lane holds.  A warp holds four columns, half a chunk; a lane's rows come in runs of four
+// (rows 128 j + 4 lane .. + 3, 16-byte words of shared memory) or, where RPL is no multiple of four, of two.
 template <int RPL>
 __global__ void __launch_bounds__(256) delta_blocks_kernel(const BlocksArgs a) {
-    constexpr int DP = 16 * RPL, KQ = 2 * DB * DP;
+    constexpr int DP = 32 * RPL, KQ = 2 * DB * DP, RUN = RPL % 4 == 0 ? 4 : 2;
     const int h = blockIdx.x, s = blockIdx.y, warps = blockDim.x >> 5;
-    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, quad = lane >> 4, l16 = lane & 15;
-    const int chunk0 = blockIdx.z * warps, chunk = chunk0 + warp;
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, quad = warp & 1;
+    const int chunk0 = blockIdx.z * (warps / 2), chunk = chunk0 + (warp >> 1);
     const int col0 = chunk * DB + quad * 4;
     const int dim = a.dim, vdim = a.vdim, g = h / (a.heads / a.groups);
     extern __shared__ __align__(16) float sm[];
-    const int stage_floats = KQ + DC + warps * DB * DB;
-    float* wsm = sm + D_STAGES * stage_floats + warp * 3 * DB * DB;  // this warp's w: [8 columns][8 rows]
-    float* usm = wsm + DB * DB;                                      // and D_8 u: [8 rows][8 columns] twice over, (u, u)
+    const int stage_floats = KQ + DC + warps / 2 * DB * DB;
+    float* wsm = sm + D_STAGES * stage_floats + warp * 3 * DB * 4;  // this warp's w: [4 columns][8 rows]
+    float* usm = wsm + DB * 4;                                      // and D_8 u: [8 rows][4 columns] twice over, (u, u)
     pdl_wait();
     const int first = a.q_start[s], n = a.q_start[s + 1] - first;
     if (n <= 0) return;
@@ -250,7 +305,7 @@ __global__ void __launch_bounds__(256) delta_blocks_kernel(const BlocksArgs a) {
     const float* kq_src = a.kq + ((size_t)g * a.blocks + blk0) * KQ;
     const float* coef_src = a.coef + ((size_t)h * a.blocks + blk0) * DC;
     const float* bv_src = a.bv + (((size_t)h * a.blocks + blk0) * a.chunks + chunk0) * DB * DB;
-    const int my_chunks = min(warps, a.chunks - chunk0);
+    const int my_chunks = min(warps / 2, a.chunks - chunk0);
     auto load = [&](int b) {
         if (b < nb) {
             float* st = sm + (b % D_STAGES) * stage_floats;
@@ -274,7 +329,7 @@ __global__ void __launch_bounds__(256) delta_blocks_kernel(const BlocksArgs a) {
         float v[2][4];
 #pragma unroll
         for (int e = 0; e < 2; ++e) {
-            const int row = (r >> 2) * 64 + l16 * 4 + (r & 3) + e;
+            const int row = r / RUN * (32 * RUN) + lane * RUN + r % RUN + e;
             v[e][0] = v[e][1] = v[e][2] = v[e][3] = 0.0f;
             if (live && row < dim) {
                 if (a.wide) {
@@ -290,18 +345,17 @@ __global__ void __launch_bounds__(256) delta_blocks_kernel(const BlocksArgs a) {
 #pragma unroll
         for (int c = 0; c < 4; ++c) S[c][r / 2] = pair_of(v[0][c], v[1][c]);
     }
-    const int tok = l16 >> 1, pair_col = quad * 4 + (l16 & 1) * 2;  // this lane's row and two columns of the chunk between exchange and update
-    const int out_col = chunk * DB + pair_col;
-    float* out = a.out + (size_t)first * a.heads * vdim + (size_t)h * vdim + out_col;
-    const bool out_pair = (vdim & 1) == 0;
+    const int tok = lane >> 2, mine = lane & 3;  // this lane's row and column between exchange and update
+    float* out = a.out + (size_t)first * a.heads * vdim + (size_t)h * vdim + col0 + mine;
+    const bool writes = chunk < a.chunks && col0 + mine < vdim;
 
     for (int b = 0; b < nb; ++b) {
         asm volatile("cp.async.wait_group %0;" ::"n"(D_STAGES - 2) : "memory");
         __syncthreads();  // block b has landed for everybody, and nobody reads block b - 1 any more
         load(b + D_STAGES - 1);
         const float* st = sm + (b % D_STAGES) * stage_floats;
-        const ulonglong2* kt = reinterpret_cast<const ulonglong2*>(st) + l16;  // row t's piece j: kt[t * DP / 4 + 16 j]
-        const ulonglong2* qt = kt + DB * DP / 4;
+        const float* kt = st + lane * RUN;  // row t's run j: kt[t * DP + 32 * RUN * j]
+        const float* qt = kt + DB * DP;
         const float* coef = st + KQ;
         if (chunk < a.chunks) {
             // ---- S^T k and S^T q of the eight rows: this lane's share of 8 x 4 columns x 2
@@ -310,10 +364,9 @@ __global__ void __launch_bounds__(256) delta_blocks_kernel(const BlocksArgs a) {
             for (int t = 0; t < DB; ++t) {
                 uint64_t K[RPL / 2], Q[RPL / 2];
 #pragma unroll
-                for (int j = 0; j < RPL / 4; ++j) {
-                    const ulonglong2 k2 = kt[t * (DP / 4) + 16 * j], q2 = qt[t * (DP / 4) + 16 * j];
-                    K[2 * j] = k2.x, K[2 * j + 1] = k2.y;
-                    Q[2 * j] = q2.x, Q[2 * j + 1] = q2.y;
+                for (int j = 0; j < RPL / RUN; ++j) {
+                    read_run<RUN>(kt + t * DP + 32 * RUN * j, K + j * (RUN / 2));
+                    read_run<RUN>(qt + t * DP + 32 * RUN * j, Q + j * (RUN / 2));
                 }
 #pragma unroll
                 for (int c = 0; c < 4; ++c) {
@@ -330,45 +383,32 @@ __global__ void __launch_bounds__(256) delta_blocks_kernel(const BlocksArgs a) {
                     val[(t * 4 + c) * 2 + 1] = lo + hi;
                 }
             }
-            // ---- one exchange: every step sends half of what a lane still holds; lane l ends up with the sums 4 l .. 4 l + 3
+            // ---- one exchange: every step sends half of what a lane still holds; lane l ends up with the sums 2 l and 2 l + 1
 #pragma unroll
-            for (int o = 8; o > 0; o >>= 1) {
-                const bool upper = (l16 & o) != 0;
+            for (int o = 16; o > 0; o >>= 1) {
+                const bool upper = (lane & o) != 0;
 #pragma unroll
-                for (int i = 0; i < 4 * o; ++i) {
-                    const float keep = upper ? val[i + 4 * o] : val[i], send = upper ? val[i] : val[i + 4 * o];
+                for (int i = 0; i < 2 * o; ++i) {
+                    const float keep = upper ? val[i + 2 * o] : val[i], send = upper ? val[i] : val[i + 2 * o];
                     val[i] = keep + __shfl_xor_sync(0xffffffffu, send, o);
                 }
             }
-            // ---- the triangles: row `tok`, two columns
-            const float2 bv = *reinterpret_cast<const float2*>(st + KQ + DC + warp * DB * DB + tok * DB + pair_col);
-            const float bg = coef[2 * DB * DB + tok], so_far = coef[2 * DB * DB + DB + tok];
-            wsm[pair_col * DB + tok] = fmaf(-bg, val[0], bv.x);
-            wsm[(pair_col + 1) * DB + tok] = fmaf(-bg, val[2], bv.y);
+            // ---- the triangles: row `tok`, column `mine`
+            const float bv = st[KQ + DC + (warp >> 1) * DB * DB + tok * DB + quad * 4 + mine];
+            wsm[mine * DB + tok] = fmaf(-coef[2 * DB * DB + tok], val[0], bv);
             __syncwarp();
-            float u0 = 0.0f, u1 = 0.0f, o0 = so_far * val[1], o1 = so_far * val[3];
+            float u = 0.0f, o = coef[2 * DB * DB + DB + tok] * val[1];
             const float4* t4 = reinterpret_cast<const float4*>(coef + tok * DB);
             const float4* m4 = reinterpret_cast<const float4*>(coef + DB * DB + tok * DB);
-            const float4* w0 = reinterpret_cast<const float4*>(wsm + pair_col * DB);
-            const float4* w1 = w0 + DB / 4;
+            const float4* w4 = reinterpret_cast<const float4*>(wsm + mine * DB);
 #pragma unroll
             for (int j = 0; j < DB / 4; ++j) {
-                const float4 t = t4[j], m = m4[j], x = w0[j], y = w1[j];
-                u0 = fmaf(t.x, x.x, fmaf(t.y, x.y, fmaf(t.z, x.z, fmaf(t.w, x.w, u0))));
-                u1 = fmaf(t.x, y.x, fmaf(t.y, y.y, fmaf(t.z, y.z, fmaf(t.w, y.w, u1))));
-                o0 = fmaf(m.x, x.x, fmaf(m.y, x.y, fmaf(m.z, x.z, fmaf(m.w, x.w, o0))));
-                o1 = fmaf(m.x, y.x, fmaf(m.y, y.y, fmaf(m.z, y.z, fmaf(m.w, y.w, o1))));
+                const float4 t = t4[j], m = m4[j], x = w4[j];
+                u = fmaf(t.x, x.x, fmaf(t.y, x.y, fmaf(t.z, x.z, fmaf(t.w, x.w, u))));
+                o = fmaf(m.x, x.x, fmaf(m.y, x.y, fmaf(m.z, x.z, fmaf(m.w, x.w, o))));
             }
-            *reinterpret_cast<float4*>(usm + (tok * DB + pair_col) * 2) = make_float4(u0, u0, u1, u1);
-            if (b * DB + tok < n) {
-                float* o = out + (size_t)(b * DB + tok) * a.heads * vdim;
-                if (out_pair && out_col < vdim) {
-                    *reinterpret_cast<float2*>(o) = make_float2(o0, o1);
-                } else {
-                    if (out_col < vdim) o[0] = o0;
-                    if (out_col + 1 < vdim) o[1] = o1;
-                }
-            }
+            *reinterpret_cast<float2*>(usm + (tok * 4 + mine) * 2) = make_float2(u, u);
+            if (writes && b * DB + tok < n) out[(size_t)(b * DB + tok) * a.heads * vdim] = o;
             __syncwarp();
             // ---- the state
             const float last = coef[2 * DB * DB + 2 * DB];
@@ -379,17 +419,17 @@ __global__ void __launch_bounds__(256) delta_blocks_kernel(const BlocksArgs a) {
                 for (int j = 0; j < RPL / 2; ++j) S[c][j] = mul2(S[c][j], last2);
 #pragma unroll
             for (int t = 0; t < DB; ++t) {
-                const ulonglong2* up = reinterpret_cast<const ulonglong2*>(usm + (t * DB + quad * 4) * 2);
+                const ulonglong2* up = reinterpret_cast<const ulonglong2*>(usm + t * 4 * 2);
                 const ulonglong2 ua = up[0], ub = up[1];
                 const uint64_t u[4] = {ua.x, ua.y, ub.x, ub.y};
 #pragma unroll
-                for (int j = 0; j < RPL / 4; ++j) {
-                    const ulonglong2 k2 = kt[t * (DP / 4) + 16 * j];
+                for (int j = 0; j < RPL / RUN; ++j) {
+                    uint64_t k2[RUN / 2];
+                    read_run<RUN>(kt + t * DP + 32 * RUN * j, k2);
 #pragma unroll
-                    for (int c = 0; c < 4; ++c) {
-                        S[c][2 * j] = fma2(k2.x, u[c], S[c][2 * j]);
-                        S[c][2 * j + 1] = fma2(k2.y, u[c], S[c][2 * j + 1]);
-                    }
+                    for (int i = 0; i < RUN / 2; ++i)
+#pragma unroll
+                        for (int c = 0; c < 4; ++c) S[c][j * (RUN / 2) + i] = fma2(k2[i], u[c], S[c][j * (RUN / 2) + i]);
                 }
             }
         }
@@ -403,7 +443,7 @@ __global__ void __launch_bounds__(256) delta_blocks_kernel(const BlocksArgs a) {
         for (int c = 0; c < 4; ++c) halves_of(S[c][r / 2], v[0][c], v[1][c]);
 #pragma unroll
         for (int e = 0; e < 2; ++e) {
-            const int row = (r >> 2) * 64 + l16 * 4 + (r & 3) + e;
+            const int row = r / RUN * (32 * RUN) + lane * RUN + r % RUN + e;
             if (row >= dim) continue;
             if (a.wide) {
                 *reinterpret_cast<float4*>(slot + (size_t)row * vdim + col0) = make_float4(v[e][0], v[e][1], v[e][2], v[e][3]);
@@ -418,14 +458,16 @@ __global__ void __launch_bounds__(256) delta_blocks_kernel(const BlocksArgs a) {
 
 template <int RPL>
 int launch_delta_blocks(const BlocksArgs& a, int num_seqs, int sm_count, cudaStream_t stream) {
-    // a CTA's warps share the keys and queries they read: as many as leave a CTA for every SM, at least two
+    // a CTA's warps share the keys and queries they bring in: as many as leave a CTA for every SM, at least four
     int warps = 8;
-    while (warps > 2 && (long long)a.heads * num_seqs * ((a.chunks + warps - 1) / warps) < sm_count) warps /= 2;
-    while (warps > 1 && warps / 2 >= a.chunks) warps /= 2;
-    const size_t smem = (size_t)(D_STAGES * (2 * DB * 16 * RPL + DC + warps * DB * DB) + warps * 3 * DB * DB) * sizeof(float);
+    while (warps > 4 && (long long)a.heads * num_seqs * ((2 * a.chunks + warps - 1) / warps) < sm_count) warps /= 2;
+    while (warps > 2 && warps / 2 >= 2 * a.chunks) warps /= 2;
+    const size_t smem = (size_t)(D_STAGES * (2 * DB * 32 * RPL + DC + warps / 2 * DB * DB) + warps * 3 * DB * 4) * sizeof(float);
     auto kern = delta_blocks_kernel<RPL>;
     if (smem > 48 * 1024) cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
-    launch_kernel(kern, dim3(a.heads, num_seqs, (a.chunks + warps - 1) / warps), dim3(warps * 32), smem, stream, a);
+    // (without the dependent-launch attribute: CTAs that become resident under the tail of the kernel
+    // before them pile up on the SMs that have room first, and a CTA here runs as long as the portion)
+    kern<<<dim3(a.heads, num_seqs, (2 * a.chunks + warps - 1) / warps), dim3(warps * 32), smem, stream>>>(a);
     return launch_status();
 }
 
@@ -450,7 +492,7 @@ constexpr int DS_HELD = 16;  // state rows a thread keeps between its two passes
 // One CTA per (group, sequence): the group's q and k channels and its heads' v channels are nobody
 // else's, so their windows move on here.  N: value columns a thread takes at once.
 template <typename AT, int N>
-__global__ void __launch_bounds__(DS_THREADS) delta_step_kernel(const StepArgs a) {
+__global__ void __launch_bounds__(DS_THREADS, 2) delta_step_kernel(const StepArgs a) {
     __shared__ float scratch[33];
     __shared__ float red[2][DS_THREADS * N];
     extern __shared__ __align__(16) float ch[];  // q [dim], k [dim], v [heads of the group][vdim], then u and o of a head [vdim] each
@@ -667,19 +709,17 @@ SHISO_API int shiso_delta_rule(const void* q, const void* k, const void* v, cons
     float* bv = coef + (size_t)heads * blocks * DC;
     const PrepareArgs prep = {q, k, v, b, a_logit, q_ld, k_ld, v_ld, b_ld, a_ld, dt_bias, a_log, q_start, kq, coef, bv,
                               num_seqs, blocks, heads, groups, dim, dp, vdim, chunks, q_scale, unit_eps};
-    const dim3 grid(blocks, groups);
-    if (act_dtype == SHISO_F32) launch_kernel(delta_prepare_kernel<float>, grid, DB * 32, 0, stream, prep);
-    else if (act_dtype == SHISO_BF16) launch_kernel(delta_prepare_kernel<__nv_bfloat16>, grid, DB * 32, 0, stream, prep);
-    else return SHISO_ERR_DTYPE;
-    const int status = launch_status();
+    int status = SHISO_ERR_DTYPE;
+    if (act_dtype == SHISO_F32) status = launch_delta_prepare<float>(prep, stream);
+    else if (act_dtype == SHISO_BF16) status = launch_delta_prepare<__nv_bfloat16>(prep, stream);
     if (status != SHISO_OK) return status;
     const int wide = vdim % 4 == 0 && slot_stride % 4 == 0 && ((uintptr_t)state & 15) == 0;
     const BlocksArgs walk = {kq, coef, bv, state, slot_stride, q_start, state_slots, out, blocks, heads, groups, dim, vdim, chunks, wide};
     switch (dp) {
-        case 64: return launch_delta_blocks<4>(walk, num_seqs, sm_count, stream);
-        case 128: return launch_delta_blocks<8>(walk, num_seqs, sm_count, stream);
-        case 192: return launch_delta_blocks<12>(walk, num_seqs, sm_count, stream);
-        default: return launch_delta_blocks<16>(walk, num_seqs, sm_count, stream);
+        case 64: return launch_delta_blocks<2>(walk, num_seqs, sm_count, stream);
+        case 128: return launch_delta_blocks<4>(walk, num_seqs, sm_count, stream);
+        case 192: return launch_delta_blocks<6>(walk, num_seqs, sm_count, stream);
+        default: return launch_delta_blocks<8>(walk, num_seqs, sm_count, stream);
     }
 }
 
