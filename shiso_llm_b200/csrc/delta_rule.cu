@@ -149,8 +149,10 @@ __global__ void __launch_bounds__(DB * 32) delta_prepare_kernel(const PrepareArg
         qv[i] *= iq;
         kv[i] *= ik;
         ks[warp][c] = kv[i];
-        kq[warp * a.dp + c] = kv[i];
-        kq[(DB + warp) * a.dp + c] = qv[i];
+        if (c < a.dp) {
+            kq[warp * a.dp + c] = kv[i];
+            kq[(DB + warp) * a.dp + c] = qv[i];
+        }
     }
     for (int c = 32 * PER + lane; c < a.dp; c += 32) kq[warp * a.dp + c] = kq[(DB + warp) * a.dp + c] = 0.0f;
     __syncthreads();

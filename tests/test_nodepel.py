@@ -402,3 +402,260 @@ def test_greedy_generation_through_the_scheduler(tmp_path, backend):
     assert [o.token_ids for o in outs] == want
     llm.engine.cache.check()
     assert llm.engine.cache.slots.free_slots == 2
+
+
+# --------------------------------------------------------------------------- mechanisms alone
+
+
+def plan_layer(left_doc, right_doc, width, mlp=None, eps=1e-5):
+    """The layer's specs as the plan builder makes them, with tensors named ``l0.*``."""
+    doc = {"architecture": "Nodepel", "vocab": 8, "width": width, "norm": {"eps": eps}, "layers": [layer(left_doc, right_doc, mlp)]}
+    return plan_from_document(doc)[2].layers[0]
+
+
+LEFT = left(6, 3, 10, 7, 0.4, 9, 6, 50.0)
+LEFT_ONE = left(5, 1, 8, 16, 0.5, 1, 8)
+RIGHT = right(6, 3, 9, 5, 4)
+RIGHT_ONE = right(2, 2, 16, 24, 1)
+RIGHT_WIDE_CONV = right(4, 1, 70, 12, 8)
+
+
+def side(which, left_doc, right_doc, width, eps=1e-5):
+    return MIXERS.build, plan_layer(left_doc, right_doc, width, eps=eps).mixer.params["branches"][which][0]
+
+
+@pytest.mark.parametrize("backend", BACKENDS)
+@pytest.mark.parametrize("which,doc", [("left", LEFT), ("left", LEFT_ONE), ("right", RIGHT), ("right", RIGHT_ONE), ("right", RIGHT_WIDE_CONV)],
+                         ids=["attention", "attention-window-of-one", "delta", "delta-one-tap", "delta-eight-taps"])
+def test_each_branch_alone_in_steps_and_batches(backend, which, doc):
+    for dtype in mixer_dtypes(backend):
+        if which == "right" and dtype == torch.bfloat16:
+            continue  # (a head's output may be small before its norm: bfloat16 is compared kernel by kernel)
+        env = build_env(backend, dtype)
+        build, spec = side(0 if which == "left" else 1, doc if which == "left" else LEFT, doc if which == "right" else RIGHT, 40)
+        mixer = build(spec, env)
+        w = bind(mixer, env, 11)
+        g = torch.Generator().manual_seed(1)
+        a, b = torch.randn(37, 40, generator=g).to(dtype), torch.randn(9, 40, generator=g).to(dtype)
+        fn = plain.attention if which == "left" else plain.gated_delta
+        want_a, want_b = (fn(w, f"l0.mix.{which}", doc, x.double(), 1e-5) for x in (a, b))
+        in_steps_and_batches(mixer, env, dtype, a, b, want_a, want_b, which, 4.0)
+
+
+@pytest.mark.parametrize("backend", BACKENDS)
+@pytest.mark.parametrize("left_doc,right_doc", [(LEFT, RIGHT), (LEFT_ONE, RIGHT_ONE)], ids=["odd-columns", "even-columns"])
+def test_both_branches_and_their_norms(backend, left_doc, right_doc):
+    env = build_env(backend, torch.float32)
+    mixer = MIXERS.build(plan_layer(left_doc, right_doc, 44).mixer, env)
+    w = bind(mixer, env, 12)
+    g = torch.Generator().manual_seed(2)
+    a, b = torch.randn(37, 44, generator=g), torch.randn(9, 44, generator=g)
+    m = {"left": left_doc, "right": right_doc}
+    want_a, want_b = (plain.parallel_mixer(w, "l0.mix", m, x.double(), 1e-5) for x in (a, b))
+    in_steps_and_batches(mixer, env, torch.float32, a, b, want_a, want_b, "both branches", 4.0)
+
+
+@pytest.mark.parametrize("backend", BACKENDS)
+@pytest.mark.parametrize("size", [5, 32, 70])
+def test_a_planted_key_on_either_side_of_the_window_edge(backend, size):
+    """One key is made to stand out (the key matrix is the query matrix and the asking row repeats its
+    direction): right before the asking row, just inside and just outside the window, far outside, on
+    either side of page borders; the asking row ends a portion or is decoded.  Inside it decides the
+    output, outside it must not be felt at all."""
+    env = build_env(backend, torch.float32)
+    doc = left(2, 2, 16, 12, 2.0, size, 8, 5000.0)
+    build, spec = side(0, doc, RIGHT, 32)
+    mixer = build(spec, env)
+    from shiso_llm_b200.weights import random_tensors
+    from shiso_llm_b200.weights.loader import target_dtype
+    specs = {s.name: s for s in mixer.tensor_specs()}
+    stored = random_tensors(list(specs.values()), 31, 0.3, "bfloat16", 0.1)
+    for k_name, q_name in {"l0.mix.left.k": "l0.mix.left.q", "l0.mix.left.k.norm": "l0.mix.left.q.norm"}.items():
+        stored[k_name] = stored[q_name].clone()
+    mixer.bind({k: v.to(env.device, target_dtype(specs[k], v.dtype, env.dtype)) for k, v in stored.items()})
+    w = {k: v.double() for k, v in stored.items()}
+    T = 150
+    g = torch.Generator().manual_seed(3)
+    base, probe = torch.randn(T, 32, generator=g) * 0.1, torch.randn(32, generator=g)
+    quiet = base.clone()
+    quiet[T - 1] = probe * 3.0
+    without = plain.attention(w, "l0.mix.left", doc, quiet.double(), 1e-5)[T - 1]
+    for back in sorted({1, size - 1, size, size + 1, 2 * size, 3, 4, 31, 32, 33, 120}):
+        h = quiet.clone()
+        h[T - 1 - back] = probe * 30.0
+        want = plain.attention(w, "l0.mix.left", doc, h.double(), 1e-5)
+        moved = (want[T - 1] - without).abs().max().item() / without.abs().max().item()
+        assert (moved > 0.02) == (back < size) or back == 0, (back, moved)
+        for tail in (0, 9):
+            feeder = Feeder(mixer, env, pages=64)
+            got = [feeder.step([("a", h[: T - tail - 7])])["a"], feeder.step([("a", h[T - tail - 7 : T - tail])])["a"]]
+            for t in range(T - tail, T):
+                got.append(feeder.step([("a", h[t : t + 1])])["a"])
+            close(torch.cat(got), want, torch.float32, f"window of {size}: planted {back} back, {tail} decoded", 4.0)
+
+
+@pytest.mark.parametrize("backend", BACKENDS)
+def test_the_sink_takes_its_share(backend):
+    """Sinks far above, near and far below the scores: a head whose sink dominates gives (nearly)
+    nothing, one whose sink is far below is an ordinary softmax; a sink that is scaled with the scores,
+    counted per key or left out differs."""
+    env = build_env(backend, torch.float32)
+    doc = left(4, 2, 12, 12, 0.3, 20, 12)
+    build, spec = side(0, doc, RIGHT, 32)
+    mixer = build(spec, env)
+    sinks = torch.tensor([30.0, 1.5, -2.0, -200.0])
+    w = bind(mixer, env, 7, 0.3, {"l0.mix.left.sink": lambda t: sinks})
+    g = torch.Generator().manual_seed(5)
+    h = torch.randn(50, 32, generator=g)
+    want = plain.attention(w, "l0.mix.left", doc, h.double(), 1e-5)
+    gone = plain.attention({**w, "l0.mix.left.sink": torch.full((4,), -1e9)}, "l0.mix.left", doc, h.double(), 1e-5)
+    assert (want - gone).abs().max().item() > 0.1 * want.abs().max().item()
+    feeder = Feeder(mixer, env)
+    got = [feeder.step([("a", h[:1])])["a"], feeder.step([("a", h[1:40])])["a"]]
+    got += [feeder.step([("a", h[t : t + 1])])["a"] for t in range(40, 50)]
+    close(torch.cat(got), want, torch.float32, "sinks", 2.0)
+
+
+@pytest.mark.parametrize("backend", BACKENDS)
+def test_a_lost_state_or_convolution_window_shows(backend):
+    """Decays of nearly one and a large first token: what it wrote is read for the whole sequence, so a
+    state or a convolution window dropped (or taken twice) at a portion's start changes every row
+    behind it; portions on either side of blocks of eight rows."""
+    env = build_env(backend, torch.float32)
+    doc = right(4, 2, 12, 10, 4)
+    build, spec = side(1, LEFT, doc, 24)
+    mixer = build(spec, env)
+    w = bind(mixer, env, 3, 0.4, {"l0.mix.right.A_log": lambda t: t * 0.0 - 9.0})
+    g = torch.Generator().manual_seed(4)
+    h = torch.randn(75, 24, generator=g) * 0.2
+    h[0] *= 40.0
+    want = plain.gated_delta(w, "l0.mix.right", doc, h.double(), 1e-5)
+    for sizes in ([75], [1], [2], [1, 2, 3], [7, 8, 9, 1], [16, 1, 15, 17], [3, 64]):
+        feeder, got, at, i = Feeder(mixer, env), [], 0, 0
+        while at < 75:
+            n = min(sizes[i % len(sizes)], 75 - at)
+            got.append(feeder.step([("a", h[at : at + n])])["a"])
+            at, i = at + n, i + 1
+        close(torch.cat(got), want, torch.float32, f"portions of {sizes}", 10.0)
+
+
+@pytest.mark.parametrize("backend", BACKENDS)
+def test_the_state_is_corrected_not_added_to(backend):
+    """The same key again and again with a step of nearly one and no forgetting: a second write with
+    the same value changes nothing, one with another value replaces it.  Plain linear attention would
+    add them up; a correction taken before the decay, or a read-out before the write, differs."""
+    env = build_env(backend, torch.float32)
+    ops, T, D, V = env.ops, 21, 8, 4
+    from types import SimpleNamespace
+    step = SimpleNamespace(num_seqs=1, q_start=torch.tensor([0, T], dtype=torch.int32, device=env.device),
+                           state_slots=torch.zeros(1, dtype=torch.int32, device=env.device))
+    g = torch.Generator().manual_seed(1)
+    key = torch.randn(1, D, generator=g).expand(T, D).contiguous()
+    v = torch.randn(T, V, generator=g)
+    v[5:13] = v[5]
+    one = torch.full((T, 1), 40.0)  # beta = 1
+    state = torch.zeros(1, 1, D, V, device=env.device)
+    out = ops.delta_rule(*(x.to(env.device) for x in (key, key, v, one, -one)), torch.zeros(1, device=env.device), torch.zeros(1, device=env.device),
+                         state, step, 1, 1, D, V, 1.0, 1e-12).double().cpu()
+    assert (out - v.double()).abs().max().item() <= 1e-5 * v.abs().max().item()  # every read-out is the latest value
+    # beta one half and a decay of one half each: u = (v - S k / 2) / 2 on the decayed state
+    half = torch.zeros(T, 1)
+    decay = torch.full((T, 1), 0.5)
+    want = plain.delta_rule(plain.unit_vector(key.double()), plain.unit_vector(key.double()), v.double(), torch.full((T,), 0.5, dtype=torch.float64), decay[:, 0].double())
+    state.zero_()
+    out = ops.delta_rule(*(x.to(env.device) for x in (key, key, v, half, half)), torch.zeros(1, device=env.device), torch.zeros(1, device=env.device),
+                         state, step, 1, 1, D, V, 1.0, 1e-6).double().cpu()
+    close(out, want, torch.float32, "beta and decay of one half")  # softplus(0) = ln 2, exp(-ln 2) = 1/2
+
+
+MLPS = {"shared": moe(7, 3, 14, 20), "plain": moe(7, 2, 9), "all-chosen": moe(4, 4, 8, 8), "one": moe(1, 1, 12, 6), "first-only": moe(9, 1, 5)}
+
+
+@pytest.mark.parametrize("backend", BACKENDS)
+@pytest.mark.parametrize("name", list(MLPS))
+def test_feed_forwards_alone(backend, name):
+    mlp = MLPS[name]
+    for dtype in mixer_dtypes(backend):
+        env = build_env(backend, dtype)
+        part = FEED_FORWARDS.build(plan_layer(LEFT, RIGHT, 36, mlp).feed_forward, env)
+        w = bind(part, env, 17, 0.3, {"l0.mlp.router.b": lambda t: t * 50.0})
+        g = torch.Generator().manual_seed(2)
+        for rows in (1, 5, 70):
+            h = (torch.randn(rows, 36, generator=g) * 1.5).to(dtype)
+            margins = []
+            want = plain.mixture(w, "l0.mlp", mlp, h.double(), margins)
+            y = part.forward(h.to(env.device), None)
+            y = (y.materialize() if hasattr(y, "materialize") else y).double().cpu()
+            sure = torch.ones(rows, dtype=torch.bool) if dtype == torch.float32 else margins[0] > CLOSE_CALL
+            assert torch.isfinite(y).all()
+            if sure.any():
+                close(y[sure], want[sure], dtype, f"{name} feed-forward, {rows} rows {dtype}", 4.0)
+
+
+@pytest.mark.parametrize("backend", BACKENDS)
+def test_the_softmax_over_the_chosen_logits(backend):
+    """Weights come from the chosen logits alone, whatever the others are, and logits so far apart that
+    a softmax over all of them would round the second choice to zero still choose it; ties fall to the
+    lower expert; logits may be a column range."""
+    env = build_env(backend, torch.float32)
+    logits = torch.tensor([[1.0, 3.0, 2.0, 2.5, -1.0], [0.5, 0.5, 0.5, 0.5, 0.5], [-300.0, 200.0, -150.0, -290.0, -400.0], [5.0, -5.0, 4.0, 4.5, 4.25]])
+    wide = torch.cat([logits, torch.full((4, 3), 999.0)], dim=1).to(env.device)
+    for z in (logits.to(env.device), wide[:, :5]):
+        ids, weights = env.ops.moe_route(z, 2, 1, 1, 1.0, scores="chosen_softmax")
+        assert ids.cpu().tolist() == [[1, 3], [0, 1], [1, 2], [0, 3]]
+        want = torch.stack([plain.choose(row.double(), 2)[1] for row in logits])
+        assert (weights.cpu().double() - want).abs().max().item() <= 1e-6
+        ids, weights = env.ops.moe_route(z, 5, 1, 1, 1.0, scores="chosen_softmax")
+        assert ids.cpu()[2].tolist() == [1, 2, 3, 0, 4] and abs(float(weights[0].sum()) - 1.0) < 1e-6
+
+
+@pytest.mark.parametrize("backend", BACKENDS)
+def test_the_pair_of_normed_branches(backend):
+    """The pair added to the stream under the next norm, with a row list (before the head), on its own,
+    and under a norm that knows no pairs; residual sums in float32."""
+    for dtype in mixer_dtypes(backend):
+        env = build_env(backend, dtype)
+        for width in (50, 64, 2056):
+            norm = NORMS.build(PartSpec("rmsnorm", {"tensor": "n", "size": width, "eps": 1e-5, "offset": 1.0}), env)
+            other = NORMS.build(PartSpec("layernorm", {"tensor": "n", "size": width, "eps": 1e-5}), env)
+            w = bind(norm, env, 3)
+            w_other = bind(other, env, 3)
+            g = torch.Generator().manual_seed(6)
+            x = (torch.randn(9, width, generator=g) * 3).to(env.device)
+            l, r = (torch.randn(9, width, generator=g).to(env.device, dtype) * s for s in (0.01, 7.0))
+            lw, rw = (1.0 + 0.3 * torch.randn(width, generator=g).to(env.device) for _ in range(2))
+            pair = NormedPair(env.ops, l, r, lw, rw, 0.5, 1e-5)
+            c = [t.double().cpu() for t in (x, l, r, lw, rw)]
+            delta = 0.5 * (plain.rms_norm(c[1], c[3], 1e-5) + plain.rms_norm(c[2], c[4], 1e-5))
+            close(pair.materialize().double().cpu(), delta, torch.float32, f"pair {width}", 2.0)
+            want = plain.centred_norm(c[0] + delta, w, "n", 1e-5)
+            stream = Stream(x.clone())
+            stream.add(pair)
+            close(stream.normed(norm).double().cpu(), want, dtype, f"pair under a norm {width}", 2.0)
+            assert (stream.residual.double().cpu() - c[0] - delta).abs().max().item() <= 1e-5 and stream.pending is None
+            residual = x.clone()
+            rows = torch.tensor([7, 2], dtype=torch.int32, device=env.device)
+            close(norm.add_apply(residual, pair, rows).double().cpu(), want[[7, 2]], dtype, "rows", 2.0)
+            assert torch.equal(residual, x)
+            stream = Stream(x.clone())
+            stream.add(pair)
+            y = c[0] + delta
+            y = (y - y.mean(-1, keepdim=True)) / torch.sqrt(y.var(-1, unbiased=False, keepdim=True) + 1e-5) * w_other["n"]
+            close(stream.normed(other).double().cpu(), y, dtype, "under a layer norm", 2.0)
+
+
+@pytest.mark.parametrize("backend", BACKENDS)
+def test_the_stream_beside_the_first_rows(backend):
+    for dtype in mixer_dtypes(backend):
+        env = build_env(backend, dtype)
+        g = torch.Generator().manual_seed(8)
+        for tokens, width in ((5, 50), (1, 64), (33, 132)):
+            x, first = (torch.randn(tokens, width, generator=g).to(env.device) for _ in range(2))
+            d0 = torch.randn(tokens, width, generator=g).to(env.device, dtype)
+            d1 = torch.randn(tokens, width, generator=g).to(env.device)
+            kept = x.clone()
+            for deltas in ((), (d0,), (d0, d1)):
+                got = env.ops.stream_concat(x, deltas, first, dtype)
+                total = sum((d.double() for d in deltas), x.double())
+                assert got.dtype == dtype and torch.equal(x, kept)
+                close(got.double().cpu(), torch.cat([total, first.double()], -1).cpu(), dtype, f"{tokens} x {width}, {len(deltas)} waiting")
