@@ -71,6 +71,9 @@ __device__ __forceinline__ float decay_of(float a_logit, float dt_bias, float ra
 }
 __device__ __forceinline__ float sigmoid_of(float z) { return 1.0f / (1.0f + expf(-z)); }
 __device__ __forceinline__ float silu_of(float z) { return z / (1.0f + expf(-z)); }
+// The same with the special-function unit's exponential and reciprocal: relative error about 2^-21, for
+// results that are rounded to bfloat16 at once.
+__device__ __forceinline__ float silu_sfu(float z) { return __fdividef(z, 1.0f + __expf(-z)); }
 
 // Block b of sequence s is number q_start[s] / 8 + s + b of the step: enough room for every sequence's
 // last, ragged block, and no prefix sum to find it.
@@ -360,15 +363,16 @@ __global__ void __launch_bounds__(256) delta_blocks_kernel(const BlocksArgs a) {
         const float* qt = kt + DB * DP;
         const float* coef = st + KQ;
         if (chunk < a.chunks) {
-            // ---- S^T k and S^T q of the eight rows: this lane's share of 8 x 4 columns x 2
+            // ---- S^T k and S^T q of the eight rows: this lane's share of 8 x 4 columns x 2.  Place t holds row
+            // t ^ tok: the rows a lane keeps in the exchange stand in the first places whatever the lane
             float val[64];
 #pragma unroll
             for (int t = 0; t < DB; ++t) {
                 uint64_t K[RPL / 2], Q[RPL / 2];
 #pragma unroll
                 for (int j = 0; j < RPL / RUN; ++j) {
-                    read_run<RUN>(kt + t * DP + 32 * RUN * j, K + j * (RUN / 2));
-                    read_run<RUN>(qt + t * DP + 32 * RUN * j, Q + j * (RUN / 2));
+                    read_run<RUN>(kt + (t ^ tok) * DP + 32 * RUN * j, K + j * (RUN / 2));
+                    read_run<RUN>(qt + (t ^ tok) * DP + 32 * RUN * j, Q + j * (RUN / 2));
                 }
 #pragma unroll
                 for (int c = 0; c < 4; ++c) {
@@ -387,7 +391,11 @@ __global__ void __launch_bounds__(256) delta_blocks_kernel(const BlocksArgs a) {
             }
             // ---- one exchange: every step sends half of what a lane still holds; lane l ends up with the sums 2 l and 2 l + 1
 #pragma unroll
-            for (int o = 16; o > 0; o >>= 1) {
+            for (int o = 16; o > 2; o >>= 1)  // over the rows
+#pragma unroll
+                for (int i = 0; i < 2 * o; ++i) val[i] += __shfl_xor_sync(0xffffffffu, val[i + 2 * o], o);
+#pragma unroll
+            for (int o = 2; o > 0; o >>= 1) {  // over the columns
                 const bool upper = (lane & o) != 0;
 #pragma unroll
                 for (int i = 0; i < 2 * o; ++i) {
@@ -677,8 +685,8 @@ delta_output_kernel(const float* __restrict__ x, const AT* __restrict__ gate, lo
                 const uint2 raw = *reinterpret_cast<const uint2*>(gr + c);
                 const float g0 = __uint_as_float(raw.x << 16), g1 = __uint_as_float(raw.x & 0xffff0000u);
                 const float g2 = __uint_as_float(raw.y << 16), g3 = __uint_as_float(raw.y & 0xffff0000u);
-                const __nv_bfloat162 lo = __floats2bfloat162_rn(v.x * inv * wv.x * silu_of(g0), v.y * inv * wv.y * silu_of(g1));
-                const __nv_bfloat162 hi = __floats2bfloat162_rn(v.z * inv * wv.z * silu_of(g2), v.w * inv * wv.w * silu_of(g3));
+                const __nv_bfloat162 lo = __floats2bfloat162_rn(v.x * inv * wv.x * silu_sfu(g0), v.y * inv * wv.y * silu_sfu(g1));
+                const __nv_bfloat162 hi = __floats2bfloat162_rn(v.z * inv * wv.z * silu_sfu(g2), v.w * inv * wv.w * silu_sfu(g3));
                 *reinterpret_cast<uint2*>(o + c) = make_uint2(*reinterpret_cast<const uint32_t*>(&lo), *reinterpret_cast<const uint32_t*>(&hi));
             } else {
                 const float4 gv = *reinterpret_cast<const float4*>(gr + c);

@@ -207,7 +207,7 @@ __global__ void causal_conv_kernel(const AT* __restrict__ x, long long x_ld, con
 }
 
 // The same for bfloat16 rows whose columns may be moved 16 bytes at a time, up to four taps: a thread
-// per (run of eight rows, eight neighbouring channels), all of the run's loads asked for first.  The
+// per (run of up to 64 rows, eight neighbouring channels), eight rows' loads asked for at once.  The
 // window is brought from rows or slot again where the run crosses into another sequence.  silu with
 // the special-function unit's exponential and reciprocal (relative error about 2^-21 on a result that
 // is rounded to 2^-9).
@@ -216,65 +216,76 @@ __global__ void __launch_bounds__(128)
 causal_conv_vec_kernel(const __nv_bfloat16* __restrict__ x, long long x_ld, const float* __restrict__ taps, const float* __restrict__ bias,
                        const float* __restrict__ state, long long slot_stride, const int* __restrict__ seq_of_token,
                        const int* __restrict__ q_start, const int* __restrict__ state_slots, __nv_bfloat16* __restrict__ y, int tokens,
-                       int channels, int silu) {
+                       int channels, int silu, int run_rows) {
     pdl_begin();
     const int groups = channels >> 3;
     const long long i = (long long)blockIdx.x * blockDim.x + threadIdx.x;
     const int run = (int)(i / groups), c0 = (int)(i % groups) * 8;
-    const int t0 = run * SHISO_CONV_ROWS, count = min(SHISO_CONV_ROWS, tokens - t0);
-    if (count <= 0) return;
+    const int run0 = run * run_rows, run_end = min(run0 + run_rows, tokens);
+    if (run0 >= tokens) return;
     auto unpack = [](const uint4& q, float (&v)[8]) {
         const uint32_t w[4] = {q.x, q.y, q.z, q.w};
 #pragma unroll
         for (int e = 0; e < 4; ++e) v[2 * e] = __uint_as_float(w[e] << 16), v[2 * e + 1] = __uint_as_float(w[e] & 0xffff0000u);
     };
     auto row_at = [&](int t) { return *reinterpret_cast<const uint4*>(x + (size_t)t * x_ld + c0); };
-    uint4 raw[SHISO_CONV_ROWS];
-#pragma unroll
-    for (int r = 0; r < SHISO_CONV_ROWS; ++r) raw[r] = row_at(t0 + min(r, count - 1));
     float tp[TAPS][8], w[TAPS - 1][8], b[8];
+    {
+        float flat[8 * TAPS];  // this thread's taps lie together: [8 channels][TAPS]
 #pragma unroll
-    for (int e = 0; e < 8; ++e) {
-        b[e] = bias ? bias[c0 + e] : 0.0f;
-#pragma unroll
-        for (int k = 0; k < TAPS; ++k) tp[k][e] = taps[(size_t)(c0 + e) * TAPS + k];
-    }
-    int current = -1;
-#pragma unroll
-    for (int r = 0; r < SHISO_CONV_ROWS; ++r) {
-        if (r >= count) break;
-        const int t = t0 + r, s = seq_of_token[t];
-        if (s != current) {  // the inputs before row t: rows of the same sequence in this step, or what its slot holds
-            current = s;
-            const int first = q_start[s];
-            const float* slot = state + (size_t)state_slots[s] * slot_stride;
-#pragma unroll
-            for (int k = 0; k < TAPS - 1; ++k) {
-                const int src = t - (TAPS - 1) + k;
-                if (src >= first) {
-                    unpack(row_at(src), w[k]);
-                } else {
-#pragma unroll
-                    for (int e = 0; e < 8; ++e) w[k][e] = slot[(size_t)(TAPS - 1 - (first - src)) * channels + c0 + e];
-                }
-            }
+        for (int k = 0; k < 2 * TAPS; ++k) {
+            const float4 f = reinterpret_cast<const float4*>(taps + (size_t)c0 * TAPS)[k];
+            flat[4 * k] = f.x, flat[4 * k + 1] = f.y, flat[4 * k + 2] = f.z, flat[4 * k + 3] = f.w;
         }
-        float in[8], out[8];
-        unpack(raw[r], in);
 #pragma unroll
         for (int e = 0; e < 8; ++e) {
-            float acc = fmaf(tp[TAPS - 1][e], in[e], b[e]);
+            b[e] = bias ? bias[c0 + e] : 0.0f;
 #pragma unroll
-            for (int k = 0; k < TAPS - 1; ++k) acc = fmaf(tp[k][e], w[k][e], acc);
-#pragma unroll
-            for (int k = 0; k + 1 < TAPS - 1; ++k) w[k][e] = w[k + 1][e];
-            w[TAPS - 2][e] = in[e];
-            out[e] = silu ? __fdividef(acc, 1.0f + __expf(-acc)) : acc;
+            for (int k = 0; k < TAPS; ++k) tp[k][e] = flat[e * TAPS + k];
         }
-        __nv_bfloat162 h[4];
+    }
+    int current = -1;
+    for (int t0 = run0; t0 < run_end; t0 += SHISO_CONV_ROWS) {
+        const int count = min(SHISO_CONV_ROWS, run_end - t0);
+        uint4 raw[SHISO_CONV_ROWS];
 #pragma unroll
-        for (int e = 0; e < 4; ++e) h[e] = __floats2bfloat162_rn(out[2 * e], out[2 * e + 1]);
-        *reinterpret_cast<uint4*>(y + (size_t)t * channels + c0) = *reinterpret_cast<const uint4*>(h);
+        for (int r = 0; r < SHISO_CONV_ROWS; ++r) raw[r] = row_at(t0 + min(r, count - 1));
+#pragma unroll
+        for (int r = 0; r < SHISO_CONV_ROWS; ++r) {
+            if (r >= count) break;
+            const int t = t0 + r, s = seq_of_token[t];
+            if (s != current) {  // the inputs before row t: rows of the same sequence in this step, or what its slot holds
+                current = s;
+                const int first = q_start[s];
+                const float* slot = state + (size_t)state_slots[s] * slot_stride;
+#pragma unroll
+                for (int k = 0; k < TAPS - 1; ++k) {
+                    const int src = t - (TAPS - 1) + k;
+                    if (src >= first) {
+                        unpack(row_at(src), w[k]);
+                    } else {
+#pragma unroll
+                        for (int e = 0; e < 8; ++e) w[k][e] = slot[(size_t)(TAPS - 1 - (first - src)) * channels + c0 + e];
+                    }
+                }
+            }
+            float in[8], out[8];
+            unpack(raw[r], in);
+#pragma unroll
+            for (int e = 0; e < 8; ++e) {
+                float acc = fmaf(tp[TAPS - 1][e], in[e], b[e]);
+#pragma unroll
+                for (int k = 0; k < TAPS - 1; ++k) acc = fmaf(tp[k][e], w[k][e], acc);
+#pragma unroll
+                for (int k = 0; k + 1 < TAPS - 1; ++k) w[k][e] = w[k + 1][e];
+                w[TAPS - 2][e] = in[e];
+                out[e] = silu ? __fdividef(acc, 1.0f + __expf(-acc)) : acc;
+            }
+            __nv_bfloat162 h[4];
+#pragma unroll
+            for (int e = 0; e < 4; ++e) h[e] = __floats2bfloat162_rn(out[2 * e], out[2 * e + 1]);
+            *reinterpret_cast<uint4*>(y + (size_t)t * channels + c0) = *reinterpret_cast<const uint4*>(h);
+        }
     }
 }
 
@@ -314,12 +325,15 @@ SHISO_API int shiso_causal_conv(const void* x, long long x_ld, int act_dtype, co
         launch_kernel(causal_conv_state_kernel<float>, sblocks, 256, 0, stream, (const float*)x, x_ld, state, slot_stride, q_start,
                       state_slots, num_seqs, channels, n_taps);
     } else if (act_dtype == SHISO_BF16) {
-        const bool wide = n_taps <= 4 && channels % 8 == 0 && x_ld % 8 == 0 && (((uintptr_t)x | (uintptr_t)y) & 15) == 0;
+        const bool wide = n_taps <= 4 && channels % 8 == 0 && x_ld % 8 == 0 && (((uintptr_t)x | (uintptr_t)y | (uintptr_t)taps) & 15) == 0;
         if (wide) {
-            const unsigned vblocks = ceil_div_u((long long)((tokens + SHISO_CONV_ROWS - 1) / SHISO_CONV_ROWS) * (channels / 8), 128);
+            // longer runs (a thread's taps are loaded once a run) while enough threads remain
+            int run_rows = SHISO_CONV_ROWS;
+            while (run_rows < 64 && (long long)tokens / (2 * run_rows) * (channels / 8) >= 32 * 1024) run_rows *= 2;
+            const unsigned vblocks = ceil_div_u((long long)((tokens + run_rows - 1) / run_rows) * (channels / 8), 128);
             auto kern = n_taps == 4 ? causal_conv_vec_kernel<4> : n_taps == 3 ? causal_conv_vec_kernel<3> : causal_conv_vec_kernel<2>;
             launch_kernel(kern, vblocks, 128, 0, stream, (const __nv_bfloat16*)x, x_ld, taps, bias, (const float*)state, slot_stride,
-                          seq_of_token, q_start, state_slots, (__nv_bfloat16*)y, tokens, channels, silu);
+                          seq_of_token, q_start, state_slots, (__nv_bfloat16*)y, tokens, channels, silu, run_rows);
         } else {
             launch_kernel(causal_conv_kernel<__nv_bfloat16>, blocks, 256, 0, stream, (const __nv_bfloat16*)x, x_ld, taps, bias,
                           (const float*)state, slot_stride, seq_of_token, q_start, state_slots, (__nv_bfloat16*)y, tokens, channels,
