@@ -12,7 +12,8 @@ everything.  A window entry that also reads the first positions of a sequence fo
 (``keep_first``) is a group of its own kind: its tables keep the pages of those positions
 and have their holes between them and the window.  Entries that hold one row per run of ``every`` positions (summaries of
 blocks) form groups of their own as well, with a pool sized for that many fewer rows.  Within a group every entry has its own K and V buffer
-``[num_pages, page_size, kv_heads, head_dim]`` (widths may differ between entries); a
+``[num_pages, page_size, kv_heads, head_dim]`` (widths may differ between entries, and an
+entry may have fewer value heads than key heads); a
 page id names the same rows in all of them, as the reference's pages do
 (crates/shiso-engine/src/kv.rs:18-31,97-109).
 
@@ -135,7 +136,7 @@ class CacheManager:
                 kv_dtype = need.dtype if need.dtype is not None else dtype
                 built[(pos, j)] = PagedKVView(
                     k=torch.zeros((buffer_pages, page_size, need.num_kv_heads, need.head_dim), dtype=kv_dtype, device=self.device),
-                    v=torch.zeros((buffer_pages, page_size, need.num_kv_heads, need.value_dim), dtype=kv_dtype, device=self.device),
+                    v=torch.zeros((buffer_pages, page_size, need.value_heads, need.value_dim), dtype=kv_dtype, device=self.device),
                     page_size=page_size,
                     group=group.index,
                     kv_heads=need.num_kv_heads,
@@ -178,7 +179,7 @@ class CacheManager:
             if isinstance(need, PagedKV):
                 itemsize = (need.dtype if need.dtype is not None else dtype).itemsize
                 # (an entry with a row per run of positions costs that much less per page of tokens)
-                page_bytes += -(-page_size * need.num_kv_heads * (need.head_dim + need.value_dim) * itemsize // need.every)
+                page_bytes += -(-page_size * (need.num_kv_heads * need.head_dim + need.value_heads * need.value_dim) * itemsize // need.every)
             elif isinstance(need, FixedState):
                 state_bytes += -(-need.nbytes // 16) * 16
         return page_bytes, state_bytes

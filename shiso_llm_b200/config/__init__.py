@@ -17,11 +17,13 @@ from . import zetavik  # registers Zetavik
 from . import volalorn  # registers Volalorn
 from . import povilorn  # registers Povilorn
 from . import nodepel  # registers Nodepel
+from . import raketar  # registers Raketar
 from .filulix import FilulixConfig
 from .zetavik import ZetavikConfig
 from .volalorn import VolalornConfig
 from .povilorn import PovilornConfig
 from .nodepel import NodepelConfig
+from .raketar import RaketarConfig
 from .lfm2 import Lfm2Config, feed_forward_width
 
 __all__ = [
@@ -33,6 +35,7 @@ __all__ = [
     "Lfm2Config",
     "NodepelConfig",
     "PovilornConfig",
+    "RaketarConfig",
     "UnknownArchitecture",
     "UnsupportedShape",
     "VolalornConfig",

@@ -12,7 +12,8 @@
 // tiles on the tensor cores.
 //
 // Routing: moe_route_kernel (a warp per row: scores, group-limited choice of the top experts by
-// score + correction, weights), moe_count / moe_place (rows grouped by expert with two passes of
+// score + correction, weights; a weight multiplies the expert's output, or, with weigh_input, its input -
+// the accumulators of the first product, ahead of the activation), moe_count / moe_place (rows grouped by expert with two passes of
 // integer atomics: which place a row gets inside its expert's range is arbitrary, its arithmetic is
 // not touched by it), moe_combine_kernel (a token's weighted sum over its choices, in the order of
 // the choices; a choice beyond the experts with matrices is an identity expert and adds the
@@ -53,6 +54,7 @@ struct TileGemmArgs {
     int M, N, K, batches;
     int act;      // the gated pair of a stacked gate/up matrix (GLU_*), or ACT_RELU2 on a plain one
     float limit;  // its clamp
+    const float* row_weight;  // with `gather`: row m's input counts row_weight[gather[m]] times (the accumulators are scaled), or nullptr
 };
 
 template <typename XT, typename WT, typename OT, bool GLU>
@@ -139,12 +141,13 @@ __global__ void __launch_bounds__(256) tile_gemm_kernel(const TileGemmArgs a) {
         if (m >= row_end) continue;
         float scale = 1.0f;
         if (a.gate) scale = 1.0f / (1.0f + expf(-to_f32(((const XT*)a.gate)[(size_t)m * a.gate_ld + batch])));
+        const float into = a.row_weight ? a.row_weight[a.gather[m]] : 1.0f;
 #pragma unroll
         for (int j = 0; j < 4; ++j) {
             const int n = n0 + tx + 16 * j;
             if (n >= a.N) continue;
-            float v = acc[i][j];
-            if (GLU) v = glu_pair(v, acc2[i][j], a.act, a.limit);
+            float v = acc[i][j] * into;
+            if (GLU) v = glu_pair(v, acc2[i][j] * into, a.act, a.limit);
             else if (a.act == ACT_RELU2) v = fmaxf(v, 0.0f), v *= v;
             out[(size_t)m * a.out_ld + n] = from_f32<OT>(v * scale);
         }
@@ -300,14 +303,15 @@ __global__ void __launch_bounds__(256) tile_gemm_mma_kernel(const TileGemmArgs a
             if (m >= row_end) continue;
             float scale = 1.0f;
             if (a.gate) scale = 1.0f / (1.0f + expf(-to_f32(((const __nv_bfloat16*)a.gate)[(size_t)m * a.gate_ld + batch])));
+            const float into = a.row_weight ? a.row_weight[a.gather[m]] : 1.0f;
 #pragma unroll
             for (int nj = 0; nj < 4; ++nj) {
 #pragma unroll
                 for (int e = 0; e < 2; ++e) {
                     const int n = n0 + wn * 32 + nj * 8 + t4 * 2 + e;
                     if (n >= a.N) continue;
-                    float v = acc[mi][nj][hrow * 2 + e];
-                    if (GLU) v = glu_pair(v, acc2[mi][nj][hrow * 2 + e], a.act, a.limit);
+                    float v = acc[mi][nj][hrow * 2 + e] * into;
+                    if (GLU) v = glu_pair(v, acc2[mi][nj][hrow * 2 + e] * into, a.act, a.limit);
                     else if (a.act == ACT_RELU2) v = fmaxf(v, 0.0f), v *= v;
                     out[(size_t)m * a.out_ld + n] = from_f32<OT>(v * scale);
                 }
@@ -511,12 +515,12 @@ __global__ void moe_place_kernel(const int* __restrict__ ids, const int* __restr
 }
 
 // out[t] = extra[t] (* sigmoid(extra_gate[t])) + sum_j weights[t, j] * y[place[t * top + j]], the choices in
-// their order; a choice whose id is `experts` or more is an identity expert: it adds weights[t, j] * x[t].
+// their order (with weigh_input the weight has gone into the expert's input and counts no more here); a choice whose id is `experts` or more is an identity expert: it adds weights[t, j] * x[t].
 template <typename AT>
 __global__ void moe_combine_kernel(const float* __restrict__ y, const int* __restrict__ place, const float* __restrict__ weights,
                                    const int* __restrict__ ids, const AT* __restrict__ x, const AT* __restrict__ extra,
                                    const float* __restrict__ extra_gate, long long extra_gate_ld, AT* __restrict__ out, int tokens,
-                                   int hidden, int top, int experts) {
+                                   int hidden, int top, int experts, int weigh_input) {
     pdl_begin();
     const long long i = (long long)blockIdx.x * blockDim.x + threadIdx.x;
     if (i >= (long long)tokens * hidden) return;
@@ -524,8 +528,9 @@ __global__ void moe_combine_kernel(const float* __restrict__ y, const int* __res
     float acc = 0.0f;
     for (int j = 0; j < top; ++j) {
         const size_t at = (size_t)t * top + j;
-        const float v = ids[at] >= experts ? to_f32(x[i]) : y[(size_t)place[at] * hidden + c];
-        acc = fmaf(weights[at], v, acc);
+        const bool identity = ids[at] >= experts;
+        const float v = identity ? to_f32(x[i]) : y[(size_t)place[at] * hidden + c];
+        acc = fmaf(weigh_input && !identity ? 1.0f : weights[at], v, acc);  // (an identity expert is linear: the weight counts on either side)
     }
     if (extra) {
         float e = to_f32(extra[i]);
@@ -544,7 +549,8 @@ __global__ void moe_combine_kernel(const float* __restrict__ y, const int* __res
 SHISO_API int shiso_routed_experts(const void* x, int act_dtype, const int* ids, const float* weights, const void* gate_up,
                                    const void* down, int w_dtype, const void* extra, const float* extra_gate,
                                    long long extra_gate_ld, void* out, int* ints, void* mid, float* y, int tokens, int hidden, int ff,
-                                   int experts, int identity, int top, int act, float limit, cudaStream_t stream) {
+                                   int experts, int identity, int top, int act, float limit, int weigh_input,
+                                   cudaStream_t stream) {
     if (tokens <= 0) return SHISO_OK;
     const int outputs = experts + identity;
     if (experts <= 0 || identity < 0 || outputs > MOE_MAX_EXPERTS || top <= 0 || hidden <= 0 || ff <= 0 || act < GLU_SILU ||
@@ -562,21 +568,21 @@ SHISO_API int shiso_routed_experts(const void* x, int act_dtype, const int* ids,
     int status = launch_status();
     if (status) return status;
     const int halves = act == ACT_RELU2 ? 1 : 2;  // an ungated expert has one matrix before its activation
-    TileGemmArgs up = {x, hidden, 0, source, top, gate_up, (long long)halves * ff * hidden, mid, ff, 0, counts, nullptr, 0, total, ff, hidden, experts, act, limit};
+    TileGemmArgs up = {x, hidden, 0, source, top, gate_up, (long long)halves * ff * hidden, mid, ff, 0, counts, nullptr, 0, total, ff, hidden, experts, act, limit, weigh_input ? weights : nullptr};
     status = halves == 2 ? launch_tile_gemm<true>(up, act_dtype, w_dtype, act_dtype, total, experts, 1, stream)
                          : launch_tile_gemm<false>(up, act_dtype, w_dtype, act_dtype, total, experts, 1, stream);
     if (status) return status;
-    TileGemmArgs dn = {mid, ff, 0, nullptr, 1, down, (long long)hidden * ff, y, hidden, 0, counts, nullptr, 0, total, hidden, ff, experts, 0, 0.0f};
+    TileGemmArgs dn = {mid, ff, 0, nullptr, 1, down, (long long)hidden * ff, y, hidden, 0, counts, nullptr, 0, total, hidden, ff, experts, 0, 0.0f, nullptr};
     status = launch_tile_gemm<false>(dn, act_dtype, w_dtype, SHISO_F32, total, experts, 1, stream);
     if (status) return status;
     const unsigned blocks = ceil_div_u((long long)tokens * hidden, 256);
     if (act_dtype == SHISO_F32)
         launch_kernel(moe_combine_kernel<float>, blocks, 256, 0, stream, (const float*)y, (const int*)place, weights, ids,
-                      (const float*)x, (const float*)extra, extra_gate, extra_gate_ld, (float*)out, tokens, hidden, top, experts);
+                      (const float*)x, (const float*)extra, extra_gate, extra_gate_ld, (float*)out, tokens, hidden, top, experts, weigh_input);
     else if (act_dtype == SHISO_BF16)
         launch_kernel(moe_combine_kernel<__nv_bfloat16>, blocks, 256, 0, stream, (const float*)y, (const int*)place, weights, ids,
                       (const __nv_bfloat16*)x, (const __nv_bfloat16*)extra, extra_gate, extra_gate_ld, (__nv_bfloat16*)out, tokens,
-                      hidden, top, experts);
+                      hidden, top, experts, weigh_input);
     else
         return SHISO_ERR_DTYPE;
     return launch_status();

@@ -26,6 +26,9 @@
 // how the sequence was cut into steps, not on the pages.  Scores, weights, statistics and
 // output sums are float.
 //
+// Neighbouring key heads may share a value head (fewer value heads than key heads), and the output
+// may be float whatever the row type (for a caller that goes on computing with it).
+//
 // Cache rows: row(p) = table[p / page_size] * page_size + p % page_size, as everywhere.
 #include "common.cuh"
 
@@ -44,7 +47,7 @@ __global__ void __launch_bounds__(MA_WARPS * 32)
 head_prepare_store_kernel(AT* __restrict__ proj, long long ld, int q_col, int k_col, int v_col, const float* __restrict__ q_w,
                           const float* __restrict__ k_w, const float* __restrict__ inv_freq, const int* __restrict__ positions,
                           const int* __restrict__ seq_of_token, const int* __restrict__ table, int table_width,
-                          AT* __restrict__ k_cache, AT* __restrict__ v_cache, int heads, int kv_heads, int dim, int vdim,
+                          AT* __restrict__ k_cache, AT* __restrict__ v_cache, int heads, int kv_heads, int v_heads, int dim, int vdim,
                           int rotary_dim, int page_size, float eps, float magnitude, int norm_mode, int store) {
     __shared__ float buf[MA_WARPS][MA_MAX_DIM];
     pdl_begin();
@@ -122,8 +125,9 @@ head_prepare_store_kernel(AT* __restrict__ proj, long long ld, int q_col, int k_
         const int c = lane + 32 * e;
         if (c < dim) kd[c] = from_f32<AT>(x[e]);
     }
+    if (head >= v_heads) return;
     const AT* vs = proj + (size_t)t * ld + v_col + (size_t)head * vdim;
-    AT* vd = v_cache + (row * kv_heads + head) * vdim;
+    AT* vd = v_cache + (row * v_heads + head) * vdim;
     for (int c = lane; c < vdim; c += 32) vd[c] = vs[c];
 }
 
@@ -140,7 +144,7 @@ head_prepare_store_vec_kernel(__nv_bfloat16* __restrict__ proj, long long ld, in
                               const float* __restrict__ q_w, const float* __restrict__ k_w, const float* __restrict__ inv_freq,
                               const int* __restrict__ positions, const int* __restrict__ seq_of_token, const int* __restrict__ table,
                               int table_width, __nv_bfloat16* __restrict__ k_cache, __nv_bfloat16* __restrict__ v_cache, int heads,
-                              int kv_heads, int dim, int vdim, int rotary_dim, int page_size, float eps, float magnitude,
+                              int kv_heads, int v_heads, int dim, int vdim, int rotary_dim, int page_size, float eps, float magnitude,
                               int norm_mode, int store, int group) {
     __shared__ float cs[MA_MAX_DIM / 2], sn[MA_MAX_DIM / 2];
     pdl_begin();
@@ -222,9 +226,9 @@ head_prepare_store_vec_kernel(__nv_bfloat16* __restrict__ proj, long long ld, in
         *reinterpret_cast<uint4*>(k_cache + (cache_row * kv_heads + head) * dim + c0) = packed;
     }
     if (store && have_row) {  // the values: 16-byte pieces, copied as they are
-        const int pieces = kv_heads * vdim / 8;
+        const int pieces = v_heads * vdim / 8;
         const uint4* vs = reinterpret_cast<const uint4*>(proj + (size_t)t * ld + v_col);
-        uint4* vd = reinterpret_cast<uint4*>(v_cache + cache_row * kv_heads * vdim);
+        uint4* vd = reinterpret_cast<uint4*>(v_cache + cache_row * v_heads * vdim);
         for (int i = blockIdx.y * MA_VEC_THREADS + threadIdx.x; i < pieces; i += MA_VEC_THREADS * gridDim.y) vd[i] = vs[i];
     }
 }
@@ -274,7 +278,8 @@ struct MaskedArgs {
     const float* key_bias;  // [heads], sigmoid weighting only; may be null
     const float* sink;      // [heads], softmax only; may be null: exp(sink) joins a head's sum, with no key and no value
     long long q_ld, out_ld, gate_ld;
-    int table_width, heads, kv_heads, dim, vdim, page_size, mask_kind, size, keep_first;
+    int table_width, heads, kv_heads, v_heads, dim, vdim, page_size, mask_kind, size, keep_first;
+    int out_float;   // out is float whatever the row type
     int gate_wide;   // the gate has a column per output entry (heads * vdim) instead of one per head
     int splits;      // CTAs that share a (row, head)'s runs of keys; more than one: partial results go to `scratch`
     float* scratch;  // [rows * heads * splits][vdim + 2]: sums, running maximum, sum of weights
@@ -332,7 +337,7 @@ __device__ __forceinline__ void ma_fold(const MaskedArgs& a, const AT* __restric
     // the run's weights and rows go through the warp's shared memory: every lane reads them all
     __syncwarp();
     run_weight[lane] = weight;
-    run_row[lane] = row >= 0 ? ((long long)row * a.kv_heads + kv_head) * a.vdim : -1;
+    run_row[lane] = row >= 0 ? ((long long)row * a.v_heads + kv_head / (a.kv_heads / a.v_heads)) * a.vdim : -1;
     __syncwarp();
     // (no branch between two loads - a key the run does not have reads row 0 with weight zero -
     // so that the value rows of eight keys are asked for together)
@@ -359,9 +364,22 @@ __device__ __forceinline__ void ma_fold(const MaskedArgs& a, const AT* __restric
     }
 }
 
+// Where a (row, head)'s outputs go, in the row type or in float.
+template <typename AT> struct MaskedOut {
+    AT* narrow;
+    float* wide;
+    __device__ __forceinline__ MaskedOut(void* out, const MaskedArgs& a, int t, int head)
+        : narrow((AT*)out + (size_t)t * a.out_ld + (size_t)head * a.vdim),
+          wide(a.out_float ? (float*)out + (size_t)t * a.out_ld + (size_t)head * a.vdim : nullptr) {}
+    __device__ __forceinline__ void put(int c, float v) const {
+        if (wide) wide[c] = v;
+        else narrow[c] = from_f32<AT>(v);
+    }
+};
+
 template <typename AT, bool SIGMOID>
 __global__ void __launch_bounds__(MA_WARPS * 32)
-masked_attention_kernel(const AT* __restrict__ q, const AT* __restrict__ k_cache, const AT* __restrict__ v_cache, AT* out,
+masked_attention_kernel(const AT* __restrict__ q, const AT* __restrict__ k_cache, const AT* __restrict__ v_cache, void* out,
                         const AT* __restrict__ gate, MaskedArgs a) {
     __shared__ float sq[MA_MAX_DIM];
     __shared__ float run_weight[MA_WARPS][32];
@@ -429,7 +447,7 @@ masked_attention_kernel(const AT* __restrict__ q, const AT* __restrict__ k_cache
         }
         return;
     }
-    AT* dst = out + (size_t)t * a.out_ld + (size_t)head * a.vdim;
+    const MaskedOut<AT> dst(out, a, t, head);
     float gated = 1.0f;
     if (gate && !a.gate_wide) gated = 1.0f / (1.0f + expf(-to_f32(gate[(size_t)t * a.gate_ld + head])));
     const AT* wide = gate && a.gate_wide ? gate + (size_t)t * a.gate_ld + (size_t)head * a.vdim : nullptr;
@@ -438,7 +456,7 @@ masked_attention_kernel(const AT* __restrict__ q, const AT* __restrict__ k_cache
             float sum = 0.0f;
 #pragma unroll
             for (int w = 0; w < MA_WARPS; ++w) sum += part_acc[w][c];
-            dst[c] = from_f32<AT>(sum * (wide ? 1.0f / (1.0f + expf(-to_f32(wide[c]))) : gated));
+            dst.put(c, sum * (wide ? 1.0f / (1.0f + expf(-to_f32(wide[c]))) : gated));
         }
         return;
     }
@@ -446,7 +464,7 @@ masked_attention_kernel(const AT* __restrict__ q, const AT* __restrict__ k_cache
 #pragma unroll
     for (int w = 0; w < MA_WARPS; ++w) top = fmaxf(top, part_max[w]);
     if (top == -INFINITY) {
-        for (int c = threadIdx.x; c < a.vdim; c += blockDim.x) dst[c] = from_f32<AT>(0.0f);
+        for (int c = threadIdx.x; c < a.vdim; c += blockDim.x) dst.put(c, 0.0f);
         return;
     }
     float factor[MA_WARPS];
@@ -461,18 +479,18 @@ masked_attention_kernel(const AT* __restrict__ q, const AT* __restrict__ k_cache
         float sum = 0.0f;
 #pragma unroll
         for (int w = 0; w < MA_WARPS; ++w) sum += part_acc[w][c] * factor[w];
-        dst[c] = from_f32<AT>(sum / total * (wide ? 1.0f / (1.0f + expf(-to_f32(wide[c]))) : gated));
+        dst.put(c, sum / total * (wide ? 1.0f / (1.0f + expf(-to_f32(wide[c]))) : gated));
     }
 }
 
 // Adds up the shares of a (row, head) in split order; softmax shares are brought to one maximum first.
 template <typename AT, bool SIGMOID>
 __global__ void __launch_bounds__(128)
-masked_attention_merge_kernel(AT* out, const AT* __restrict__ gate, MaskedArgs a) {
+masked_attention_merge_kernel(void* out, const AT* __restrict__ gate, MaskedArgs a) {
     pdl_begin();
     const int t = blockIdx.x / a.heads, head = blockIdx.x % a.heads;
     const float* parts = a.scratch + (size_t)blockIdx.x * a.splits * (a.vdim + 2);
-    AT* dst = out + (size_t)t * a.out_ld + (size_t)head * a.vdim;
+    const MaskedOut<AT> dst(out, a, t, head);
     float gated = 1.0f;
     if (gate && !a.gate_wide) gated = 1.0f / (1.0f + expf(-to_f32(gate[(size_t)t * a.gate_ld + head])));
     const AT* wide = gate && a.gate_wide ? gate + (size_t)t * a.gate_ld + (size_t)head * a.vdim : nullptr;
@@ -480,7 +498,7 @@ masked_attention_merge_kernel(AT* out, const AT* __restrict__ gate, MaskedArgs a
     if (!SIGMOID) {
         for (int s = 0; s < a.splits; ++s) top = fmaxf(top, parts[(size_t)s * (a.vdim + 2) + a.vdim]);
         if (top == -INFINITY) {
-            for (int c = threadIdx.x; c < a.vdim; c += blockDim.x) dst[c] = from_f32<AT>(0.0f);
+            for (int c = threadIdx.x; c < a.vdim; c += blockDim.x) dst.put(c, 0.0f);
             return;
         }
         for (int s = 0; s < a.splits; ++s) {
@@ -496,15 +514,15 @@ masked_attention_merge_kernel(AT* out, const AT* __restrict__ gate, MaskedArgs a
             const float f = SIGMOID ? 1.0f : (part[a.vdim] == -INFINITY ? 0.0f : expf(part[a.vdim] - top));
             sum += part[c] * f;
         }
-        dst[c] = from_f32<AT>((SIGMOID ? sum : sum / total) * (wide ? 1.0f / (1.0f + expf(-to_f32(wide[c]))) : gated));
+        dst.put(c, (SIGMOID ? sum : sum / total) * (wide ? 1.0f / (1.0f + expf(-to_f32(wide[c]))) : gated));
     }
 }
 
 template <typename AT>
 int launch_prepare(void* proj, long long ld, int q_col, int k_col, int v_col, const float* q_w, const float* k_w, const float* inv_freq,
                    const int* positions, const int* seq_of_token, const int* table, int table_width, void* k_cache, void* v_cache,
-                   int tokens, int heads, int kv_heads, int dim, int vdim, int rotary_dim, int page_size, float eps, float magnitude,
-                   int norm_mode, int store, cudaStream_t stream) {
+                   int tokens, int heads, int kv_heads, int v_heads, int dim, int vdim, int rotary_dim, int page_size, float eps,
+                   float magnitude, int norm_mode, int store, cudaStream_t stream) {
     if constexpr (sizeof(AT) == 2) {
         const bool wide = dim % 8 == 0 && vdim % 8 == 0 && rotary_dim % 16 == 0 && ld % 8 == 0 && q_col % 8 == 0 && k_col % 8 == 0 &&
                           v_col % 8 == 0 && !(((uintptr_t)proj | (uintptr_t)k_cache | (uintptr_t)v_cache) & 15);
@@ -517,13 +535,13 @@ int launch_prepare(void* proj, long long ld, int q_col, int k_col, int v_col, co
             const dim3 vgrid(tokens, passes);
             launch_kernel(head_prepare_store_vec_kernel, vgrid, MA_VEC_THREADS, 0, stream, (__nv_bfloat16*)proj, ld, q_col, k_col, v_col, q_w,
                           k_w, inv_freq, positions, seq_of_token, table, table_width, (__nv_bfloat16*)k_cache, (__nv_bfloat16*)v_cache, heads,
-                          kv_heads, dim, vdim, rotary_dim, page_size, eps, magnitude, norm_mode, store, group);
+                          kv_heads, v_heads, dim, vdim, rotary_dim, page_size, eps, magnitude, norm_mode, store, group);
             return launch_status();
         }
     }
     const dim3 grid(tokens, ceil_div_u(heads + (store ? kv_heads : 0), MA_WARPS));
     launch_kernel(head_prepare_store_kernel<AT>, grid, MA_WARPS * 32, 0, stream, (AT*)proj, ld, q_col, k_col, v_col, q_w, k_w, inv_freq,
-                  positions, seq_of_token, table, table_width, (AT*)k_cache, (AT*)v_cache, heads, kv_heads, dim, vdim, rotary_dim,
+                  positions, seq_of_token, table, table_width, (AT*)k_cache, (AT*)v_cache, heads, kv_heads, v_heads, dim, vdim, rotary_dim,
                   page_size, eps, magnitude, norm_mode, store);
     return launch_status();
 }
@@ -534,17 +552,17 @@ int launch_attention(const void* q, const void* k_cache, const void* v_cache, vo
     const unsigned items = (unsigned)tokens * a.heads, blocks = items * a.splits;
     if (sigmoid)
         launch_kernel(masked_attention_kernel<AT, true>, blocks, MA_WARPS * 32, 0, stream, (const AT*)q, (const AT*)k_cache,
-                      (const AT*)v_cache, (AT*)out, (const AT*)gate, a);
+                      (const AT*)v_cache, out, (const AT*)gate, a);
     else
         launch_kernel(masked_attention_kernel<AT, false>, blocks, MA_WARPS * 32, 0, stream, (const AT*)q, (const AT*)k_cache,
-                      (const AT*)v_cache, (AT*)out, (const AT*)gate, a);
+                      (const AT*)v_cache, out, (const AT*)gate, a);
     if (a.splits > 1) {
         const int first = launch_status();
         if (first != SHISO_OK) return first;
         if (sigmoid)
-            launch_kernel(masked_attention_merge_kernel<AT, true>, items, 128, 0, stream, (AT*)out, (const AT*)gate, a);
+            launch_kernel(masked_attention_merge_kernel<AT, true>, items, 128, 0, stream, out, (const AT*)gate, a);
         else
-            launch_kernel(masked_attention_merge_kernel<AT, false>, items, 128, 0, stream, (AT*)out, (const AT*)gate, a);
+            launch_kernel(masked_attention_merge_kernel<AT, false>, items, 128, 0, stream, out, (const AT*)gate, a);
     }
     return launch_status();
 }
@@ -554,20 +572,20 @@ int launch_attention(const void* q, const void* k_cache, const void* v_cache, vo
 SHISO_API int shiso_head_prepare_store(void* proj, long long ld, int act_dtype, int q_col, int k_col, int v_col, const float* q_w,
                                        const float* k_w, const float* inv_freq, const int* positions, const int* seq_of_token,
                                        const int* table, int table_width, void* k_cache, void* v_cache, int tokens, int heads,
-                                       int kv_heads, int dim, int vdim, int rotary_dim, int page_size, float eps, float magnitude,
-                                       int norm_mode, int store, cudaStream_t stream) {
+                                       int kv_heads, int v_heads, int dim, int vdim, int rotary_dim, int page_size, float eps,
+                                       float magnitude, int norm_mode, int store, cudaStream_t stream) {
     if (tokens <= 0) return SHISO_OK;
     if (dim <= 0 || dim > MA_MAX_DIM || vdim <= 0 || heads <= 0 || kv_heads < 0 || rotary_dim < 0 || rotary_dim > dim || rotary_dim % 2 ||
-        norm_mode < MA_NORM_NONE || norm_mode > MA_NORM_AFTER)
+        norm_mode < MA_NORM_NONE || norm_mode > MA_NORM_AFTER || (store && (v_heads <= 0 || v_heads > kv_heads)))
         return SHISO_ERR_SHAPE;
     if (rotary_dim > 0 && !inv_freq) return SHISO_ERR_SHAPE;
     if (act_dtype == SHISO_F32)
         return launch_prepare<float>(proj, ld, q_col, k_col, v_col, q_w, k_w, inv_freq, positions, seq_of_token, table, table_width, k_cache,
-                                     v_cache, tokens, heads, kv_heads, dim, vdim, rotary_dim, page_size, eps, magnitude, norm_mode, store,
+                                     v_cache, tokens, heads, kv_heads, v_heads, dim, vdim, rotary_dim, page_size, eps, magnitude, norm_mode, store,
                                      stream);
     if (act_dtype == SHISO_BF16)
         return launch_prepare<__nv_bfloat16>(proj, ld, q_col, k_col, v_col, q_w, k_w, inv_freq, positions, seq_of_token, table, table_width,
-                                             k_cache, v_cache, tokens, heads, kv_heads, dim, vdim, rotary_dim, page_size, eps, magnitude,
+                                             k_cache, v_cache, tokens, heads, kv_heads, v_heads, dim, vdim, rotary_dim, page_size, eps, magnitude,
                                              norm_mode, store, stream);
     return SHISO_ERR_DTYPE;
 }
@@ -575,12 +593,13 @@ SHISO_API int shiso_head_prepare_store(void* proj, long long ld, int act_dtype, 
 SHISO_API int shiso_masked_attention(const void* q, long long q_ld, int act_dtype, const void* k_cache, const void* v_cache,
                                      const int* table, int table_width, const int* positions, const int* seq_of_token, void* out,
                                      long long out_ld, const void* gate, long long gate_ld, const float* key_bias, int tokens,
-                                     int heads, int kv_heads, int dim, int vdim, int page_size, float scale, float softcap,
+                                     int heads, int kv_heads, int v_heads, int dim, int vdim, int page_size, float scale, float softcap,
                                      int mask_kind, int size, int keep_first, int sigmoid, int splits, float* scratch,
-                                     int gate_wide, const float* sink, cudaStream_t stream) {
+                                     int gate_wide, const float* sink, int out_float, cudaStream_t stream) {
     if (tokens <= 0) return SHISO_OK;
     if (splits < 1 || (splits > 1 && !scratch)) return SHISO_ERR_SHAPE;
-    if (dim <= 0 || dim > MA_MAX_DIM || vdim <= 0 || vdim > MA_MAX_DIM || kv_heads <= 0 || heads % kv_heads || size < 1 || keep_first < 0 ||
+    if (dim <= 0 || dim > MA_MAX_DIM || vdim <= 0 || vdim > MA_MAX_DIM || kv_heads <= 0 || heads % kv_heads || v_heads <= 0 || kv_heads % v_heads ||
+        size < 1 || keep_first < 0 ||
         (mask_kind != MA_MASK_WINDOW && mask_kind != MA_MASK_CHUNK))
         return SHISO_ERR_SHAPE;
     if ((long long)tokens * heads * splits > 0x7fffffffLL) return SHISO_ERR_SHAPE;
@@ -597,6 +616,8 @@ SHISO_API int shiso_masked_attention(const void* q, long long q_ld, int act_dtyp
     a.table_width = table_width;
     a.heads = heads;
     a.kv_heads = kv_heads;
+    a.v_heads = v_heads;
+    a.out_float = out_float;
     a.dim = dim;
     a.vdim = vdim;
     a.page_size = page_size;

@@ -15,7 +15,7 @@
 // memory for every 16 channels instead of being kept in registers.  The value size is a template
 // parameter (multiples of 16 up to 128), because the output accumulators live in registers.
 // Keys outside every row's range are zero-filled, never read: a window group's table has holes
-// there.  A masked key scores minus infinity under the softmax and weighs zero under the sigmoid.
+// there.  Neighbouring key heads may share a value head, and the output may be float.  A masked key scores minus infinity under the softmax and weighs zero under the sigmoid.
 #include "mma_tiles.cuh"
 
 namespace {
@@ -33,17 +33,18 @@ enum { MT_MASK_WINDOW = 0, MT_MASK_CHUNK = 1 };
 struct TileArgs {
     const __nv_bfloat16* q;        // [T, ...] rows q_ld apart, head h at column h * dim
     const __nv_bfloat16* k_cache;  // [pages, page, kv_heads, dim]
-    const __nv_bfloat16* v_cache;  // [pages, page, kv_heads, vdim]
+    const __nv_bfloat16* v_cache;  // [pages, page, v_heads, vdim]
     const __nv_bfloat16* gate;     // [T, ...] rows gate_ld apart, head h at column h; or null
     const float* key_bias;         // [heads] or null
     const float* sink;             // [heads] or null (softmax): exp(sink) joins a head's sum, with no key and no value
     const int* block_table;        // [S, width]
     const int* q_start;            // [S + 1]
     const int* start_pos;          // [S]
-    __nv_bfloat16* out;            // [T, ...] rows out_ld apart, head h at column h * vdim
+    void* out;                     // [T, ...] rows out_ld apart, head h at column h * vdim; bfloat16, or float with out_float
     long long q_ld, out_ld, gate_ld;
     int gate_wide;                 // the gate has a column per output entry (head h's at h * DV) instead of one per head
-    int width, num_seqs, heads, kv_heads, dim, page_size, mask_kind, size, keep_first;
+    int out_float;
+    int width, num_seqs, heads, kv_heads, v_heads, dim, page_size, mask_kind, size, keep_first;
     float scale, softcap;
 };
 
@@ -95,6 +96,7 @@ masked_tiles_kernel(TileArgs a) {
     const int last_pos = first_pos + rows - 1;
     const int head = blockIdx.x;
     const int kv_head = head / (a.heads / a.kv_heads);
+    const int v_head = kv_head / (a.kv_heads / a.v_heads);
     const int* table = a.block_table + (size_t)seq * a.width;
     const int keep = a.mask_kind == MT_MASK_WINDOW ? a.keep_first : 0;
     const int key_lo = max(0, low_edge(a, first_pos));  // low edges do not fall as positions rise
@@ -143,7 +145,7 @@ masked_tiles_kernel(TileArgs a) {
             if (valid) page = table[key / a.page_size];
             valid = page >= 0;
             const size_t row = valid ? (size_t)page * a.page_size + key % a.page_size : 0;
-            cp_async16(vd + r * V_ROW + ch * 16, a.v_cache + (row * a.kv_heads + kv_head) * DV + ch * 8, valid);
+            cp_async16(vd + r * V_ROW + ch * 16, a.v_cache + (row * a.v_heads + v_head) * DV + ch * 8, valid);
         }
     };
     load_kv(tile_of(0), 0);
@@ -308,7 +310,9 @@ masked_tiles_kernel(TileArgs a) {
             float f = factor[r];
             if (a.gate && !a.gate_wide) f *= 1.0f / (1.0f + expf(-__bfloat162float(a.gate[(size_t)(first_token + row) * a.gate_ld + head])));
             const __nv_bfloat16* wide = a.gate && a.gate_wide ? a.gate + (size_t)(first_token + row) * a.gate_ld + (size_t)head * DV : nullptr;
-            __nv_bfloat16* dst = a.out + (size_t)(first_token + row) * a.out_ld + (size_t)head * DV;
+            const size_t at = (size_t)(first_token + row) * a.out_ld + (size_t)head * DV;
+            __nv_bfloat16* dst = (__nv_bfloat16*)a.out + at;
+            float* dst_float = a.out_float ? (float*)a.out + at : nullptr;
 #pragma unroll
             for (int i = 0; i < DTILES; ++i) {
                 float f0 = f, f1 = f;
@@ -316,7 +320,10 @@ masked_tiles_kernel(TileArgs a) {
                     f0 *= 1.0f / (1.0f + expf(-__bfloat162float(wide[i * 8 + t4 * 2])));
                     f1 *= 1.0f / (1.0f + expf(-__bfloat162float(wide[i * 8 + t4 * 2 + 1])));
                 }
-                *reinterpret_cast<uint32_t*>(dst + i * 8 + t4 * 2) = pack_bf16(o_acc[i][r * 2] * f0, o_acc[i][r * 2 + 1] * f1);
+                if (dst_float)
+                    *reinterpret_cast<float2*>(dst_float + i * 8 + t4 * 2) = make_float2(o_acc[i][r * 2] * f0, o_acc[i][r * 2 + 1] * f1);
+                else
+                    *reinterpret_cast<uint32_t*>(dst + i * 8 + t4 * 2) = pack_bf16(o_acc[i][r * 2] * f0, o_acc[i][r * 2 + 1] * f1);
             }
         }
     }
@@ -353,11 +360,11 @@ SHISO_API int shiso_masked_attention_tiles_supported(int dim, int vdim) {
 SHISO_API int shiso_masked_attention_tiles(const void* q, long long q_ld, const void* k_cache, const void* v_cache, const int* table,
                                            int table_width, const int* q_start, const int* start_pos, void* out, long long out_ld,
                                            const void* gate, long long gate_ld, const float* key_bias, int num_seqs, int max_tiles,
-                                           int heads, int kv_heads, int dim, int vdim, int page_size, float scale, float softcap,
-                                           int mask_kind, int size, int keep_first, int sigmoid, int gate_wide, const float* sink,
-                                           cudaStream_t stream) {
+                                           int heads, int kv_heads, int v_heads, int dim, int vdim, int page_size, float scale,
+                                           float softcap, int mask_kind, int size, int keep_first, int sigmoid, int gate_wide,
+                                           const float* sink, int out_float, cudaStream_t stream) {
     if (num_seqs <= 0 || max_tiles <= 0) return SHISO_OK;
-    if (kv_heads <= 0 || heads % kv_heads || size < 1 || keep_first < 0 || (mask_kind != MT_MASK_WINDOW && mask_kind != MT_MASK_CHUNK))
+    if (kv_heads <= 0 || heads % kv_heads || v_heads <= 0 || kv_heads % v_heads || size < 1 || keep_first < 0 || (mask_kind != MT_MASK_WINDOW && mask_kind != MT_MASK_CHUNK))
         return SHISO_ERR_SHAPE;
     if (!shiso_masked_attention_tiles_supported(dim, vdim) || max_tiles > 65535) return SHISO_ERR_UNSUPPORTED;
     if ((out_ld % 2) || (((uintptr_t)out | (uintptr_t)k_cache | (uintptr_t)v_cache) & 15)) return SHISO_ERR_ALIGN;
@@ -371,7 +378,9 @@ SHISO_API int shiso_masked_attention_tiles(const void* q, long long q_ld, const 
     a.block_table = table;
     a.q_start = q_start;
     a.start_pos = start_pos;
-    a.out = (__nv_bfloat16*)out;
+    a.out = out;
+    a.out_float = out_float;
+    a.v_heads = v_heads;
     a.q_ld = q_ld;
     a.out_ld = out_ld;
     a.gate_ld = gate_ld;

@@ -3,7 +3,8 @@
 //   norm_into   residual[t] += y[t] * rsqrt(mean(y[t]^2) + eps) * w   (float, in place), and, when
 //               asked, the new residual row in the activation type: what the next sublayer reads.
 //   normed_pair residual[t] += scale * (norm(left[t]) + norm(right[t])), and the norm of the new row: what
-//               closes a mixer of two branches and opens the sublayer behind it.
+//               closes a mixer of two branches and opens the sublayer behind it; without `right` one
+//               branch alone.
 //   polynorm    out[t] = a * N(z[t]) + b * N(z[t]^2) + c * N(z[t]^3) + e, powers taken element by
 //               element, N(u) = u * rsqrt(mean(u^2) + eps) over the row.
 //
@@ -194,7 +195,8 @@ template <int N> __device__ __forceinline__ void pair_store(__nv_bfloat16* p, co
     else p[0] = __float2bfloat16_rn(v[0]);
 }
 
-template <typename AT, int N>
+// PAIR false: there is no second branch (right, wb unused).
+template <typename AT, int N, bool PAIR>
 __global__ void normed_pair_kernel(const NormedPairArgs a, const AT* __restrict__ left, const AT* __restrict__ right, AT* __restrict__ out) {
     __shared__ float scratch[33];
     extern __shared__ __align__(16) float row_cache[];
@@ -207,22 +209,31 @@ __global__ void normed_pair_kernel(const NormedPairArgs a, const AT* __restrict_
     for (int i = first; i < a.hidden; i += stride) {
         float x[N], y[N];
         pair_load<N>(l + i, x);
-        pair_load<N>(r + i, y);
+        if constexpr (PAIR) pair_load<N>(r + i, y);
 #pragma unroll
-        for (int e = 0; e < N; ++e) sl += x[e] * x[e], sr += y[e] * y[e];
+        for (int e = 0; e < N; ++e) {
+            sl += x[e] * x[e];
+            if constexpr (PAIR) sr += y[e] * y[e];
+        }
     }
     const float il = rsqrtf(block_sum(sl, scratch) / (float)a.hidden + a.pair_eps);
-    const float ir = rsqrtf(block_sum(sr, scratch) / (float)a.hidden + a.pair_eps);
+    const float ir = PAIR ? rsqrtf(block_sum(sr, scratch) / (float)a.hidden + a.pair_eps) : 0.0f;
     float* res = a.residual ? a.residual + (size_t)src * a.hidden : nullptr;
     float ss = 0.0f;
     for (int i = first; i < a.hidden; i += stride) {
         float x[N], y[N], wl[N], wr[N];
         pair_load<N>(l + i, x);
-        pair_load<N>(r + i, y);
         pair_load<N>(a.wa + i, wl);
-        pair_load<N>(a.wb + i, wr);
+        if constexpr (PAIR) {
+            pair_load<N>(r + i, y);
+            pair_load<N>(a.wb + i, wr);
+        }
 #pragma unroll
-        for (int e = 0; e < N; ++e) x[e] = a.scale * (x[e] * il * wl[e] + y[e] * ir * wr[e]);
+        for (int e = 0; e < N; ++e) {
+            x[e] = x[e] * il * wl[e];
+            if constexpr (PAIR) x[e] += y[e] * ir * wr[e];
+            x[e] *= a.scale;
+        }
         if (!res) {
             pair_store<N>(a.sum + (size_t)blockIdx.x * a.hidden + i, x);
             continue;
@@ -248,7 +259,8 @@ __global__ void normed_pair_kernel(const NormedPairArgs a, const AT* __restrict_
 template <typename AT>
 int launch_normed_pair(const NormedPairArgs& a, const void* left, const void* right, void* out, int out_rows, bool wide, cudaStream_t stream) {
     const size_t smem = a.residual ? (size_t)a.hidden * sizeof(float) : 0;
-    auto kernel = wide ? normed_pair_kernel<AT, 8> : normed_pair_kernel<AT, 1>;
+    auto kernel = wide ? (right ? normed_pair_kernel<AT, 8, true> : normed_pair_kernel<AT, 8, false>)
+                       : (right ? normed_pair_kernel<AT, 1, true> : normed_pair_kernel<AT, 1, false>);
     if (smem > 48 * 1024) cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
     launch_kernel(kernel, out_rows, wide ? vec_block_for(a.hidden) : block_for(a.hidden), smem, stream, a, (const AT*)left, (const AT*)right,
                   (AT*)out);
@@ -291,13 +303,14 @@ SHISO_API int shiso_polynorm(const void* z, long long z_ld, int act_dtype, const
     return launch_status();
 }
 
-// left, right [T, hidden] in the activation type; weights float [hidden].  out_rows: T, or the length of `rows`.
+// left, right [T, hidden] in the activation type (right and wb may be null together: one branch); weights float [hidden].  out_rows: T, or the length of `rows`.
 SHISO_API int shiso_normed_pair(const void* left, const void* right, int act_dtype, const float* wa, const float* wb, float scale,
                                 float pair_eps, float* residual, const int* rows, const float* w, float eps, void* out, float* sum,
                                 int out_rows, int hidden, cudaStream_t stream) {
     if (out_rows <= 0) return SHISO_OK;
     if (hidden <= 0 || hidden > 50 * 1024) return SHISO_ERR_SHAPE;
     if (residual ? (!w || !out) : !sum) return SHISO_ERR_UNSUPPORTED;
+    if ((right != nullptr) != (wb != nullptr)) return SHISO_ERR_UNSUPPORTED;
     const NormedPairArgs a = {residual, rows, wa, wb, w, sum, hidden, scale, pair_eps, eps};
     const bool wide = hidden % 8 == 0 && aligned16(left, right, residual, out) && aligned16(wa, wb, w, sum);
     if (act_dtype == SHISO_F32) return launch_normed_pair<float>(a, left, right, out, out_rows, wide, stream);

@@ -2,10 +2,12 @@
 //
 //     S_t = a_t S_{t-1} + b_t k_t v_t^T,        o_t = S_t^T q_t + skip_h v_t,
 //
-// S[dim, vdim] per head, float, carried per request in its state slot.  Two ways to give a and b:
+// S[dim, vdim] per head, float, carried per request in its state slot.  Three ways to give a and b:
 // a fixed decay per head (loss_h = 1 - decay_h; S - loss S is formed, so that a decay near one
 // loses nothing to its own rounding; b = 1), or a step size per token and head, dt, with
-// b = softplus(dt + dt_bias_h) and a = exp(-exp(a_log_h) b).  q and k may be shared by the heads of
+// b = softplus(dt + dt_bias_h) and a = exp(-exp(a_log_h) b); or both factors as they are, a pair per token
+// and head.  With the last, a normaliser n <- a n + b k may run along as one more value column that is
+// always 1 (its state and its outputs are kept apart).  q and k may be shared by the heads of
 // a group (head h reads group h / (heads / groups)); silu may be applied to q, k and v on load.
 //
 // One CTA walks the rows of one (head, sequence, range of value columns) in order.  A warp holds 8
@@ -32,6 +34,10 @@ struct StateRecurrenceArgs {
     const int *q_start, *state_slots;
     float* out;
     int heads, groups, dim, vdim, cols, silu;
+    const float *keep, *add;  // [T, heads] each, or null: a and b themselves
+    float* normaliser;        // [slots][heads][dim], norm_stride apart, or null
+    long long norm_stride;
+    float* norm_out;          // [T, heads]: n . q
     int bulk;  // rows may be fetched 16 bytes at a time (widths, strides and addresses allow it)
 };
 
@@ -56,7 +62,7 @@ __global__ void __launch_bounds__(256 + SR_PRODUCERS) state_recurrence_kernel(co
     const bool producer = (int)threadIdx.x >= workers;
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
     const int part = lane & 7, local = warp * 8 + (lane >> 3) * 2, col = col0 + local;  // columns col and col + 1
-    const bool live = !producer && col < a.vdim, live1 = !producer && col + 1 < a.vdim;
+    const bool live = !producer && col < a.vdim + (a.normaliser ? 1 : 0), live1 = !producer && col + 1 < a.vdim + (a.normaliser ? 1 : 0);
     const int dim = a.dim, vdim = a.vdim, g = h / (a.heads / a.groups);
     constexpr int DP = 8 * RPT;             // key rows with padding (zeros: their state stays zero)
     extern __shared__ __align__(16) float sm[];
@@ -69,17 +75,20 @@ __global__ void __launch_bounds__(256 + SR_PRODUCERS) state_recurrence_kernel(co
     const int first = a.q_start[s], n = a.q_start[s + 1] - first;
     if (n <= 0) return;
     float* slot = a.state + (size_t)a.state_slots[s] * a.slot_stride + (size_t)h * dim * vdim;
+    float* nslot = a.normaliser ? a.normaliser + (size_t)a.state_slots[s] * a.norm_stride + (size_t)h * dim : nullptr;
+    auto at = [&](int row, int c) { return c < vdim ? slot + (size_t)row * vdim + c : nslot + row; };
     float S[RPT], S1[RPT];
 #pragma unroll
     for (int r = 0; r < RPT; ++r) {
         const int row = (r >> 2) * 32 + part * 4 + (r & 3);
-        S[r] = (live && row < dim) ? slot[(size_t)row * vdim + col] : 0.0f;
-        S1[r] = (live1 && row < dim) ? slot[(size_t)row * vdim + col + 1] : 0.0f;
+        S[r] = (live && row < dim) ? *at(row, col) : 0.0f;
+        S1[r] = (live1 && row < dim) ? *at(row, col + 1) : 0.0f;
     }
     const AT* qp = (const AT*)a.q + (size_t)g * dim;
     const AT* kp = (const AT*)a.k + (size_t)g * dim;
     const AT* vp = (const AT*)a.v + (size_t)h * vdim + col0;
     const AT* dtp = a.dt ? (const AT*)a.dt + h : nullptr;
+    const bool factors = dtp || a.keep;  // a pair of factors per token and head
     float* op = a.out + (size_t)h * vdim + col;
 
     // Rows base .. base + count - 1 into a stage, by `threads` threads of which this is number `me`.
@@ -122,16 +131,22 @@ __global__ void __launch_bounds__(256 + SR_PRODUCERS) state_recurrence_kernel(co
             for (int u = 0; u < 4; ++u) {
                 const int i = i0 + u * threads, t = i / a.cols, c = i - t * a.cols;
                 ok[u] = i < SR_TOKENS * a.cols && t < count && col0 + c < vdim;
-                vv[u] = to_f32(vp[(ok[u] ? row0 + t : row0) * a.v_ld + (ok[u] ? c : 0)]);
+                vv[u] = to_f32(vp[(ok[u] ? row0 + t : row0) * a.v_ld + (ok[u] ? c : min(0, vdim - 1 - col0))]);  // (the normaliser may have the CTA to itself)
             }
 #pragma unroll
             for (int u = 0; u < 4; ++u) {
                 const int i = i0 + u * threads;
                 if (i >= SR_TOKENS * a.cols) continue;
                 if (a.silu) vv[u] = sr_silu<AT>(vv[u]);
-                sv[i] = ok[u] ? vv[u] : 0.0f;
+                const int t = i / a.cols, c = i - t * a.cols;
+                sv[i] = ok[u] ? vv[u] : (nslot && col0 + c == vdim && t < count ? 1.0f : 0.0f);
             }
         }
+        if (a.keep)
+            for (int t = me; t < count; t += threads) {
+                sa[t] = a.keep[(row0 + t) * a.heads + h];
+                sb[t] = a.add[(row0 + t) * a.heads + h];
+            }
         if (dtp) {
             for (int t = me; t < count; t += threads) {
                 const float z = to_f32(dtp[(row0 + t) * a.dt_ld]) + dt_bias;
@@ -195,7 +210,12 @@ __global__ void __launch_bounds__(256 + SR_PRODUCERS) state_recurrence_kernel(co
         for (int i = me; i < SR_TOKENS * a.cols; i += threads) {
             float vv = to_f32(rv[i]);  // zeros where the copy was left out
             if (a.silu) vv = sr_silu<AT>(vv);
-            sv[i] = vv;
+            const int t = i / a.cols, c = i - t * a.cols;
+            sv[i] = nslot && col0 + c == vdim && t < count ? 1.0f : vv;
+        }
+        if (a.keep && me < count) {
+            sa[me] = a.keep[((size_t)(first + base) + me) * a.heads + h];
+            sb[me] = a.add[((size_t)(first + base) + me) * a.heads + h];
         }
         if (dtp && me < count) {
             const float step = z > 20.0f ? z : log1pf(expf(z));
@@ -240,7 +260,7 @@ __global__ void __launch_bounds__(256 + SR_PRODUCERS) state_recurrence_kernel(co
                 const float2 vt = *reinterpret_cast<const float2*>(sv + t * a.cols + local);
                 float a0 = 0.0f, a1 = 0.0f, a2 = 0.0f, a3 = 0.0f;  // four chains a column instead of one of dim / 8 links
                 float b0 = 0.0f, b1 = 0.0f, b2 = 0.0f, b3 = 0.0f;
-                if (dtp) {
+                if (factors) {
                     const float decay = sa[t], bv0 = sb[t] * vt.x, bv1 = sb[t] * vt.y;
 #pragma unroll
                     for (int j = 0; j < RPT / 4; ++j) {
@@ -292,8 +312,8 @@ __global__ void __launch_bounds__(256 + SR_PRODUCERS) state_recurrence_kernel(co
                 }
                 if (part == 0) {
                     float* o_row = op + (row0 + t) * ((size_t)a.heads * vdim);
-                    if (live) o_row[0] = fmaf(skip, vt.x, acc);
-                    if (live1) o_row[1] = fmaf(skip, vt.y, acc1);
+                    if (live) *(col < vdim ? o_row : a.norm_out + (row0 + t) * a.heads + h) = fmaf(skip, vt.x, acc);
+                    if (live1) *(col + 1 < vdim ? o_row + 1 : a.norm_out + (row0 + t) * a.heads + h) = fmaf(skip, vt.y, acc1);
                 }
             }
         }
@@ -303,8 +323,8 @@ __global__ void __launch_bounds__(256 + SR_PRODUCERS) state_recurrence_kernel(co
 #pragma unroll
     for (int r = 0; r < RPT; ++r) {
         const int row = (r >> 2) * 32 + part * 4 + (r & 3);
-        if (live && row < dim) slot[(size_t)row * vdim + col] = S[r];
-        if (live1 && row < dim) slot[(size_t)row * vdim + col + 1] = S1[r];
+        if (live && row < dim) *at(row, col) = S[r];
+        if (live1 && row < dim) *at(row, col + 1) = S1[r];
     }
 }
 
@@ -314,14 +334,15 @@ static int launch_state_recurrence(const StateRecurrenceArgs& a, int num_seqs, i
     // warps bring and activate its head's keys and queries themselves, so narrow CTAs repeat that
     // work), or what the head has
     int cols = 64;
-    while (cols > 16 && (long long)a.heads * num_seqs * ((a.vdim + cols - 1) / cols) < sm_count) cols /= 2;
-    while (cols > 8 && cols / 2 >= a.vdim) cols /= 2;
+    const int width = a.vdim + (a.normaliser ? 1 : 0);
+    while (cols > 16 && (long long)a.heads * num_seqs * ((width + cols - 1) / cols) < sm_count) cols /= 2;
+    while (cols > 8 && cols / 2 >= width) cols /= 2;
     StateRecurrenceArgs args = a;
     args.cols = cols;
     const int epv = 16 / (int)sizeof(AT);
     args.bulk = a.dim % epv == 0 && a.vdim % epv == 0 && a.q_ld % epv == 0 && a.k_ld % epv == 0 && a.v_ld % epv == 0 &&
                 (((uintptr_t)a.q | (uintptr_t)a.k | (uintptr_t)a.v) & 15) == 0;
-    const dim3 grid(a.heads, num_seqs, (a.vdim + cols - 1) / cols), block(cols * 4 + SR_PRODUCERS);
+    const dim3 grid(a.heads, num_seqs, (width + cols - 1) / cols), block(cols * 4 + SR_PRODUCERS);
     const int rpt = (a.dim + 31) / 32 * 4;  // key rows in runs of 32: four to each of a column pair's eight lanes
 #define SR_CASE(R)                                                                                                   \
     if (rpt <= R) {                                                                                                  \
@@ -347,7 +368,24 @@ SHISO_API int shiso_state_recurrence(const void* q, const void* k, const void* v
     if ((dt != nullptr) == (head_loss != nullptr)) return SHISO_ERR_UNSUPPORTED;  // one of the two forms
     if (dt && (!dt_bias || !a_log)) return SHISO_ERR_UNSUPPORTED;
     StateRecurrenceArgs a = {q, k, v, dt, q_ld, k_ld, v_ld, dt_ld, dt_bias, a_log, skip, head_loss, state, slot_stride,
-                             q_start, state_slots, out, heads, groups, dim, vdim, 0, silu, 0};
+                             q_start, state_slots, out, heads, groups, dim, vdim, 0, silu, nullptr, nullptr, nullptr, 0, nullptr, 0};
+    if (act_dtype == SHISO_F32) return launch_state_recurrence<float>(a, num_seqs, sm_count, stream);
+    if (act_dtype == SHISO_BF16) return launch_state_recurrence<__nv_bfloat16>(a, num_seqs, sm_count, stream);
+    return SHISO_ERR_DTYPE;
+}
+
+// The same with both factors given, keep and add float [T, heads], and a normaliser [slots, heads, dim] along:
+// out float [T, heads * vdim], norm_out float [T, heads].
+SHISO_API int shiso_state_recurrence_factors(const void* q, const void* k, const void* v, long long q_ld, long long k_ld, long long v_ld,
+                                             int act_dtype, const float* keep, const float* add, float* state, long long slot_stride,
+                                             float* normaliser, long long norm_stride, const int* q_start, const int* state_slots,
+                                             float* out, float* norm_out, int tokens, int num_seqs, int heads, int dim, int vdim, int sm_count,
+                                             cudaStream_t stream) {
+    if (tokens <= 0 || num_seqs <= 0) return SHISO_OK;
+    if (heads <= 0 || dim <= 0 || dim > 256 || vdim <= 0) return SHISO_ERR_SHAPE;
+    if (!keep || !add || !normaliser || !norm_out) return SHISO_ERR_UNSUPPORTED;
+    StateRecurrenceArgs a = {q, k, v, nullptr, q_ld, k_ld, v_ld, 0, nullptr, nullptr, nullptr, nullptr, state, slot_stride,
+                             q_start, state_slots, out, heads, heads, dim, vdim, 0, 0, keep, add, normaliser, norm_stride, norm_out, 0};
     if (act_dtype == SHISO_F32) return launch_state_recurrence<float>(a, num_seqs, sm_count, stream);
     if (act_dtype == SHISO_BF16) return launch_state_recurrence<__nv_bfloat16>(a, num_seqs, sm_count, stream);
     return SHISO_ERR_DTYPE;

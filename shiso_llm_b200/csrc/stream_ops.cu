@@ -4,6 +4,9 @@
 // add_dyt_kernel:      x = residual (+ up to two block outputs), stored back; out = tanh(alpha x) * w + b.
 // stream_add_kernel:   out = residual + up to three blocks of rows (each float or bfloat16) + one vector
 //                      that is the same for every row; out may be the residual itself.
+// stream_add_rows:     residual += scale * (one or two blocks of rows), in place, and the new rows in the
+//                      activation type where a part reads the stream itself.
+// side_gate:           gelu_tanh(z[t, c]) * table[token of row t, first column + c].
 // gate_rows_kernel:    x *= sigmoid(gate), entry by entry, in place.
 // glu_act_kernel:      the gated pair of a feed-forward over rows [gate | up]: silu(g) u, the tanh form
 //                      of gelu(g) u, or min(g, L) sigmoid(1.702 min(g, L)) (clamp(u, -L, L) + 1).
@@ -178,6 +181,87 @@ SHISO_API int shiso_stream_add(const float* residual, float* out, const void* d0
         if (a.d[j] && a.dtype[j] != SHISO_F32 && a.dtype[j] != SHISO_BF16) return SHISO_ERR_DTYPE;
     launch_kernel(stream_add_kernel, ceil_div_u(a.total, 256), 256, 0, stream, a);
     return launch_status();
+}
+
+// A thread per N neighbouring columns.
+template <typename AT, int N>
+__global__ void __launch_bounds__(256)
+stream_add_rows_kernel(float* __restrict__ residual, const AT* __restrict__ d0, const AT* __restrict__ d1, float scale,
+                       AT* __restrict__ rows, long long total) {
+    pdl_begin();
+    const long long i = ((long long)blockIdx.x * blockDim.x + threadIdx.x) * N;
+    if (i >= total) return;
+    float x[N], a[N], b[N];
+    load_n<N>(d0 + i, a);
+    if (d1) load_n<N>(d1 + i, b);
+    load_n<N>(residual + i, x);
+#pragma unroll
+    for (int e = 0; e < N; ++e) x[e] = fmaf(scale, d1 ? a[e] + b[e] : a[e], x[e]);
+    store_n<N>(residual + i, x);
+    if (rows) store_n<N>(rows + i, x);
+}
+
+// residual float [T, hidden]; d0, d1 (or null) and rows (or null) [T, hidden] in the activation type.
+SHISO_API int shiso_stream_add_rows(float* residual, const void* d0, const void* d1, int act_dtype, float scale, void* rows, int tokens,
+                                    int hidden, cudaStream_t stream) {
+    if (tokens <= 0 || hidden <= 0) return SHISO_OK;
+    if (!d0) return SHISO_ERR_UNSUPPORTED;
+    const long long total = (long long)tokens * hidden;
+    const bool aligned = ((((uintptr_t)residual) | ((uintptr_t)d0) | ((uintptr_t)d1) | ((uintptr_t)rows)) & 15) == 0;
+    const int n = !aligned ? 1 : total % 8 == 0 ? 8 : total % 4 == 0 ? 4 : 1;
+    const unsigned blocks = ceil_div_u(total / n, 256);
+#define ROWS_GO(AT, N) \
+    launch_kernel(stream_add_rows_kernel<AT, N>, blocks, 256, 0, stream, residual, (const AT*)d0, (const AT*)d1, scale, (AT*)rows, total)
+    if (act_dtype == SHISO_F32) {
+        if (n == 8) ROWS_GO(float, 8);
+        else if (n == 4) ROWS_GO(float, 4);
+        else ROWS_GO(float, 1);
+    } else if (act_dtype == SHISO_BF16) {
+        if (n == 8) ROWS_GO(__nv_bfloat16, 8);
+        else if (n == 4) ROWS_GO(__nv_bfloat16, 4);
+        else ROWS_GO(__nv_bfloat16, 1);
+    } else {
+        return SHISO_ERR_DTYPE;
+    }
+#undef ROWS_GO
+    return launch_status();
+}
+
+template <typename WT, typename AT>
+__global__ void __launch_bounds__(256)
+side_gate_kernel(const float* __restrict__ z, const WT* __restrict__ table, long long table_ld, int first_column, int vocab,
+                 const int* __restrict__ ids, const int* __restrict__ feed_index, const int* __restrict__ fed_tokens, AT* __restrict__ out,
+                 int tokens, int dim) {
+    pdl_begin();
+    const long long i = (long long)blockIdx.x * blockDim.x + threadIdx.x;
+    if (i >= (long long)tokens * dim) return;
+    const int t = (int)(i / dim), c = (int)(i % dim);
+    int id = ids[t];
+    if (feed_index && feed_index[t] >= 0) id = fed_tokens[feed_index[t]];
+    const float e = id >= 0 && id < vocab ? to_f32(table[(size_t)id * table_ld + first_column + c]) : 0.0f;
+    out[i] = from_f32<AT>(glu_pair(z[i], e, GLU_GELU_TANH, 0.0f));
+}
+
+// z float [T, dim]; table [vocab, table_ld], its columns first_column .. + dim; a row's token is ids[t], or
+// fed_tokens[feed_index[t]] where feed_index (may be null) is not negative; out [T, dim].
+SHISO_API int shiso_side_gate(const float* z, const void* table, int table_dtype, long long table_ld, int first_column, int vocab,
+                              const int* ids, const int* feed_index, const int* fed_tokens, void* out, int out_dtype, int tokens, int dim,
+                              cudaStream_t stream) {
+    if (tokens <= 0 || dim <= 0) return SHISO_OK;
+    if (first_column < 0 || first_column + dim > table_ld || (feed_index && !fed_tokens)) return SHISO_ERR_SHAPE;
+    const unsigned blocks = ceil_div_u((long long)tokens * dim, 256);
+#define SIDE_GO(WT, AT)                                                                                                              \
+    {                                                                                                                                \
+        launch_kernel(side_gate_kernel<WT, AT>, blocks, 256, 0, stream, z, (const WT*)table, table_ld, first_column, vocab, ids, feed_index, \
+                      fed_tokens, (AT*)out, tokens, dim);                                                                            \
+        return launch_status();                                                                                                      \
+    }
+    if (table_dtype == SHISO_F32 && out_dtype == SHISO_F32) SIDE_GO(float, float)
+    if (table_dtype == SHISO_F32 && out_dtype == SHISO_BF16) SIDE_GO(float, __nv_bfloat16)
+    if (table_dtype == SHISO_BF16 && out_dtype == SHISO_BF16) SIDE_GO(__nv_bfloat16, __nv_bfloat16)
+    if (table_dtype == SHISO_BF16 && out_dtype == SHISO_F32) SIDE_GO(__nv_bfloat16, float)
+#undef SIDE_GO
+    return SHISO_ERR_DTYPE;
 }
 
 // --------------------------------------------------------------------------- the stream beside the first rows

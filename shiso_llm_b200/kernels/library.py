@@ -79,15 +79,15 @@ _SIGNATURES = {
     "shiso_state_recurrence": [P, P, P, P, LL, LL, LL, LL, I, P, P, P, P, P, LL, P, P, P, I, I, I, I, I, I, I, I, P],
     "shiso_head_linear": [P, LL, LL, I, P, I, P, LL, LL, I, P, LL, I, I, I, I, P],
     "shiso_moe_route": [P, LL, P, P, P, I, I, I, I, I, F, I, I, F, P],
-    "shiso_routed_experts": [P, I, P, P, P, P, I, P, P, LL, P, P, P, P, I, I, I, I, I, I, I, F, P],
+    "shiso_routed_experts": [P, I, P, P, P, P, I, P, P, LL, P, P, P, P, I, I, I, I, I, I, I, F, I, P],
     "shiso_latent_attention_smem": [I, I],
     "shiso_latent_attention": [P, I, P, P, I, P, P, P, P, I, I, I, I, I, F, I, P],
     "shiso_latent_prefill_supported": [I, I],
     "shiso_latent_prefill": [P, P, P, I, P, P, P, I, I, I, I, I, I, F, P],
-    "shiso_head_prepare_store": [P, LL, I, I, I, I, P, P, P, P, P, P, I, P, P, I, I, I, I, I, I, I, F, F, I, I, P],
-    "shiso_masked_attention": [P, LL, I, P, P, P, I, P, P, P, LL, P, LL, P, I, I, I, I, I, I, F, F, I, I, I, I, I, P, I, P, P],
+    "shiso_head_prepare_store": [P, LL, I, I, I, I, P, P, P, P, P, P, I, P, P, I, I, I, I, I, I, I, I, F, F, I, I, P],
+    "shiso_masked_attention": [P, LL, I, P, P, P, I, P, P, P, LL, P, LL, P, I, I, I, I, I, I, I, F, F, I, I, I, I, I, P, I, P, I, P],
     "shiso_masked_attention_tiles_supported": [I, I],
-    "shiso_masked_attention_tiles": [P, LL, P, P, P, I, P, P, P, LL, P, LL, P, I, I, I, I, I, I, I, F, F, I, I, I, I, I, P, P],
+    "shiso_masked_attention_tiles": [P, LL, P, P, P, I, P, P, P, LL, P, LL, P, I, I, I, I, I, I, I, I, F, F, I, I, I, I, I, P, I, P],
     "shiso_norm_into": [P, P, I, P, P, I, I, F, P],
     "shiso_polynorm": [P, LL, I, P, P, I, I, F, P],
     "shiso_gemm_stream_glu": [P, P, P, I, I, I, I, I, F, I, P],
@@ -105,6 +105,13 @@ _SIGNATURES = {
     "shiso_delta_step": [P, P, P, P, LL, I, P, P, P, P, P, LL, P, LL, P, P, P, LL, I, I, I, I, I, I, F, F, F, P],
     "shiso_delta_rule": [P, P, P, P, P, LL, LL, LL, LL, LL, I, P, P, P, LL, P, P, P, P, I, I, I, I, I, I, F, F, I, P],
     "shiso_delta_output": [P, P, LL, I, P, P, LL, I, I, I, F, P],
+    "shiso_stream_add_rows": [P, P, P, I, F, P, I, I, P],
+    "shiso_side_gate": [P, P, I, LL, I, I, P, P, P, P, I, I, I, P],
+    "shiso_state_recurrence_factors": [P, P, P, LL, LL, LL, I, P, P, P, LL, P, LL, P, P, P, P, I, I, I, I, I, I, P],
+    "shiso_memory_gates": [P, F, P, LL, P, P, P, P, P, I, I, P],
+    "shiso_memory_output": [P, P, P, P, LL, I, P, P, LL, I, I, I, F, F, F, P],
+    "shiso_memory_step": [P, P, P, P, P, P, P, LL, I, P, P, LL, P, LL, P, LL, P, P, P, LL, I, I, I, I, I, F, F, F, F, P],
+    "shiso_map_difference": [P, P, LL, I, P, LL, I, I, I, I, F, F, F, P],
 }
 
 

@@ -221,6 +221,52 @@ def stream_add(residual, deltas, vector, in_place=True):
     return out
 
 
+def stream_add_rows(residual, deltas, scale, out_dtype):
+    """``residual += scale * sum(deltas)`` for one or two block outputs of one type (float32 sums, in
+    place); returns the new rows in ``out_dtype``, which is the outputs' type - the residual itself when
+    that is float32 - or None when ``out_dtype`` is None."""
+    _check(residual, "residual", torch.float32, 2)
+    tokens, hidden = residual.shape
+    deltas = tuple(deltas)
+    if not 1 <= len(deltas) <= 2:
+        raise KernelError(f"{len(deltas)} block outputs to add; the kernel takes one or two")
+    act = deltas[0].dtype
+    for d in deltas:
+        _check(d, "rows to add", act, 2)
+        if d.shape != residual.shape:
+            raise KernelError(f"rows of {tuple(d.shape)} added to a residual of {tuple(residual.shape)}")
+    if out_dtype not in (None, act):
+        raise KernelError(f"rows of {out_dtype} from outputs of {act}")
+    rows = torch.empty_like(deltas[0]) if out_dtype is not None and act != torch.float32 else None
+    status = library().shiso_stream_add_rows(
+        _ptr(residual), _ptr(deltas[0]), _ptr(deltas[1]) if len(deltas) > 1 else 0, _code(deltas[0]), float(scale), _ptr(rows), tokens, hidden, _stream())
+    _done(status, f"stream_add_rows ({len(deltas)})", shape=(tokens, hidden))
+    if out_dtype is None:
+        return None
+    return residual if rows is None else rows
+
+
+def side_gate(z, table, first_column, ids, feed_index, fed_tokens, out_dtype):
+    """``gelu_tanh(z[t, c]) * table[id_t, first_column + c]`` for ``z`` float32 ``[T, dim]``; ids as in ``embed``."""
+    _check(z, "z", torch.float32, 2)
+    _check(table, "side table", None, 2)
+    _check(ids, "ids", torch.int32, 1)
+    tokens, dim = z.shape
+    if ids.shape[0] != tokens or not 0 <= first_column <= table.shape[1] - dim:
+        raise KernelError(f"{ids.shape[0]} ids and columns from {first_column} of {table.shape[1]} for rows of {tokens} x {dim}")
+    if (feed_index is None) != (fed_tokens is None):
+        raise KernelError("side_gate: feed_index and fed_tokens come together")
+    for name, t in (("feed_index", feed_index), ("fed_tokens", fed_tokens)):
+        if t is not None:
+            _check(t, name, torch.int32, 1)
+    out = torch.empty((tokens, dim), dtype=out_dtype, device=z.device)
+    status = library().shiso_side_gate(
+        _ptr(z), _ptr(table), _code(table), table.shape[1], int(first_column), table.shape[0], _ptr(ids), _ptr(feed_index), _ptr(fed_tokens),
+        _ptr(out), _code(out), tokens, dim, _stream())
+    _done(status, "side_gate", shape=(tokens, dim))
+    return out
+
+
 def stream_concat(residual, deltas, first, out_dtype):
     """``[residual + sum(deltas) | first]``, rows ``[T, 2 H]`` of ``out_dtype``: ``residual`` and ``first``
     float32 ``[T, H]``, up to two blocks of rows ``deltas`` (float32 or bfloat16 each)."""
@@ -1286,9 +1332,11 @@ def head_prepare_store(proj, heads, kv_heads, dim, vdim, q_w, k_w, eps, norm_ord
     rotation; weights ``q_w`` / ``k_w`` of ``[dim]`` or None for a unit norm), the half-split
     rotation of the first ``rotary_dim`` entries by ``position * inv_freq`` with cosine and sine
     times ``magnitude``.  Queries are written back where they stood; keys and the values (copied
-    as they are) go to the paged caches.  Returns the query columns."""
+    as they are) go to the paged caches.  A value cache of fewer heads than the key cache stands for key heads
+    that share their values: ``proj`` then holds that many value heads.  Returns the query columns."""
     act = proj.dtype
-    q_cols, k_cols, v_cols = heads * dim, kv_heads * dim, kv_heads * vdim
+    v_heads = v_cache.shape[2] if store else kv_heads
+    q_cols, k_cols, v_cols = heads * dim, kv_heads * dim, v_heads * vdim
     ld = _rows(proj, "projected rows", act)
     if proj.shape[1] < q_cols + k_cols + v_cols:
         raise KernelError(f"projected rows of {proj.shape[1]} do not hold {heads} + {kv_heads} heads of {dim} and {kv_heads} of {vdim}")
@@ -1307,12 +1355,12 @@ def head_prepare_store(proj, heads, kv_heads, dim, vdim, q_w, k_w, eps, norm_ord
     if store:
         _paged(k_cache, "k cache", act, page_size)
         _paged(v_cache, "v cache", act, page_size)
-        if k_cache.shape[2:] != (kv_heads, dim) or v_cache.shape[2:] != (kv_heads, vdim):
+        if k_cache.shape[2:] != (kv_heads, dim) or v_cache.shape[3] != vdim or kv_heads % v_heads:
             raise KernelError(f"caches of shape {tuple(k_cache.shape)} / {tuple(v_cache.shape)} for {kv_heads} heads of {dim} / {vdim}")
     status = library().shiso_head_prepare_store(
         proj.data_ptr(), ld, _CODES[act], 0, q_cols, q_cols + k_cols, _ptr(q_w), _ptr(k_w), _ptr(inv_freq) if rotary_dim else 0,
         _ptr(step.positions), _ptr(step.seq_of_token), _ptr(block_table), block_table.shape[1],
-        _ptr(k_cache) if store else 0, _ptr(v_cache) if store else 0, proj.shape[0], heads, kv_heads, dim, vdim, int(rotary_dim),
+        _ptr(k_cache) if store else 0, _ptr(v_cache) if store else 0, proj.shape[0], heads, kv_heads, v_heads, dim, vdim, int(rotary_dim),
         page_size, float(eps), float(magnitude), _HEAD_NORMS[norm_order], int(bool(store)), _stream(),
     )
     _done(status, "head_prepare_store", shape=(proj.shape[0], heads + kv_heads, dim))
@@ -1370,7 +1418,8 @@ def joined_norm_store(proj, heads, kv_heads, dim, vdim, q_w, k_w, eps, q_tempera
 
 
 def masked_attention(q, heads, k_cache, v_cache, block_table, page_size, scale, mask, size, keep_first, step, *, sigmoid=False,
-                     key_bias=None, softcap=None, gate=None, general=False, gate_per_element=False, sink=None, out=None):
+                     key_bias=None, softcap=None, gate=None, general=False, gate_per_element=False, sink=None, out=None,
+                     out_dtype=None):
     """Attention of every row over the keys its mask shows: ``mask`` "window" (the last ``size``
     positions and the first ``keep_first`` of the sequence) or "chunk" (the positions of the row's
     own run of ``size``, counted from 0).  Scores ``(q . k) * scale``, capped as
@@ -1379,7 +1428,8 @@ def masked_attention(q, heads, k_cache, v_cache, block_table, page_size, scale, 
     only): ``exp(sink[head])`` joins a head's denominator, with no key and no value.  ``gate[T, heads]`` (logits)
     multiplies each head's output by its sigmoid; with ``gate_per_element`` it is ``[T, heads * vdim]``
     and every output entry has a gate of its own.  ``q`` and ``gate`` may be column ranges.
-    Returns ``[T, heads * vdim]`` (``out``, where rows to write are given).  bfloat16 steps that hold prompt portions take the tiled
+    A value cache of fewer heads than the key cache: neighbouring key heads share a value head.  Returns
+    ``[T, heads * vdim]`` (``out``, where rows to write are given), in ``out_dtype`` (the row type, or float32).  bfloat16 steps that hold prompt portions take the tiled
     tensor-core kernel (key sizes in multiples of 16 up to 256, value sizes up to 128); steps of
     single tokens, float32 and other sizes take the general kernel, as does ``general=True``
     (tests compare the routes)."""
@@ -1401,11 +1451,15 @@ def masked_attention(q, heads, k_cache, v_cache, block_table, page_size, scale, 
             raise KernelError(f"{sink.shape[0]} sinks for {heads} heads under {'sigmoid weights' if sigmoid else 'a softmax'}")
     gate_ld = _rows(gate, "gate", act, heads * (vdim if gate_per_element else 1)) if gate is not None else 0
     wide = int(bool(gate is not None and gate_per_element))
-    tokens = q.shape[0]
+    tokens, v_heads = q.shape[0], v_cache.shape[2]
+    if kv_heads % v_heads or out_dtype not in (None, act, torch.float32):
+        raise KernelError(f"{v_heads} value heads for {kv_heads} key heads, output of {out_dtype}")
+    out_dtype = out_dtype or act
+    out_float = int(out_dtype == torch.float32)
     if out is None:
-        out = torch.empty((tokens, heads * vdim), dtype=act, device=q.device)
+        out = torch.empty((tokens, heads * vdim), dtype=out_dtype, device=q.device)
     else:
-        _check(out, "out", act, 2)
+        _check(out, "out", out_dtype, 2)
         if out.shape != (tokens, heads * vdim):
             raise KernelError(f"out of {tuple(out.shape)} for {tokens} rows of {heads} heads of {vdim}")
     lib = library()
@@ -1416,7 +1470,7 @@ def masked_attention(q, heads, k_cache, v_cache, block_table, page_size, scale, 
     # (A gate per output entry is applied behind them by a row kernel; a gate per head keeps the kernels that know it.)
     plain_window = (
         not general and act == torch.bfloat16 and mask == "window" and not sigmoid and not softcap and (gate is None or wide)
-        and dim == vdim and q.data_ptr() % 16 == 0 and q_ld % 8 == 0
+        and dim == vdim and v_heads == kv_heads and out_dtype == act and q.data_ptr() % 16 == 0 and q_ld % 8 == 0
     )
     if (
         plain_window and getattr(step, "all_decode", False) and heads // kv_heads <= MAX_DECODE_GROUP
@@ -1459,8 +1513,8 @@ def masked_attention(q, heads, k_cache, v_cache, block_table, page_size, scale, 
         status = lib.shiso_masked_attention_tiles(
             q.data_ptr(), q_ld, _ptr(k_cache), _ptr(v_cache), _ptr(block_table), block_table.shape[1], _ptr(step.q_start),
             _ptr(step.start_pos), _ptr(out), heads * vdim, gate.data_ptr() if gate is not None else 0, gate_ld, _ptr(key_bias),
-            step.num_seqs, tiles, heads, kv_heads, dim, vdim, page_size, float(scale), float(softcap or 0.0), _MASKS[mask], int(size),
-            int(keep_first), int(bool(sigmoid)), wide, _ptr(sink), _stream(),
+            step.num_seqs, tiles, heads, kv_heads, v_heads, dim, vdim, page_size, float(scale), float(softcap or 0.0), _MASKS[mask], int(size),
+            int(keep_first), int(bool(sigmoid)), wide, _ptr(sink), out_float, _stream(),
         )
         _done(status, f"masked_attention_tiles {what}", shape=(tokens, heads, dim))
         return out
@@ -1473,10 +1527,27 @@ def masked_attention(q, heads, k_cache, v_cache, block_table, page_size, scale, 
     status = lib.shiso_masked_attention(
         q.data_ptr(), q_ld, _CODES[act], _ptr(k_cache), _ptr(v_cache), _ptr(block_table), block_table.shape[1], _ptr(step.positions),
         _ptr(step.seq_of_token), _ptr(out), heads * vdim, gate.data_ptr() if gate is not None else 0, gate_ld, _ptr(key_bias),
-        tokens, heads, kv_heads, dim, vdim, page_size, float(scale), float(softcap or 0.0), _MASKS[mask], int(size), int(keep_first),
-        int(bool(sigmoid)), splits, _ptr(scratch), wide, _ptr(sink), _stream(),
+        tokens, heads, kv_heads, v_heads, dim, vdim, page_size, float(scale), float(softcap or 0.0), _MASKS[mask], int(size), int(keep_first),
+        int(bool(sigmoid)), splits, _ptr(scratch), wide, _ptr(sink), out_float, _stream(),
     )
     _done(status, f"masked_attention {what}", 2 if splits > 1 else 1, shape=(tokens, heads, dim))
+    return out
+
+
+def map_difference(maps, pairs, groups, second, factor, eps, gate, out):
+    """``d = a_1 - second * a_2`` of the maps' outputs ``maps`` (float32 ``[T, 2 pairs * vdim]`` in the order key
+    head, map, query head of the group), ``out = d / rms(d) * factor * sigmoid(gate)`` per head of ``vdim``
+    entries; ``gate`` and ``out`` ``[T, pairs * vdim]`` of one type, head by head (column ranges may be given)."""
+    _check(maps, "maps", torch.float32, 2)
+    tokens, width = out.shape
+    vdim = width // pairs
+    if width != pairs * vdim or maps.shape != (tokens, 2 * width) or pairs % groups or gate.shape[0] != tokens:
+        raise KernelError(f"maps {tuple(maps.shape)} and rows {tuple(out.shape)} for {pairs} heads in {groups} groups")
+    gate_ld, out_ld = _rows(gate, "gate", out.dtype, width), _rows(out, "out", None, width)
+    status = library().shiso_map_difference(
+        _ptr(maps), gate.data_ptr(), gate_ld, _code(out), out.data_ptr(), out_ld, tokens, pairs, groups, vdim, float(second), float(factor),
+        float(eps), _stream())
+    _done(status, "map_difference", shape=(tokens, pairs, vdim))
     return out
 
 
@@ -1501,12 +1572,14 @@ def norm_into(residual, y, w, eps, want_rows=True):
 
 
 def _normed_pair(left, right, wa, wb, scale, pair_eps, residual, rows, w, eps, out, total, out_rows):
-    for name, t in (("left", left), ("right", right)):
+    for name, t in (("left", left), ("right", right)) if right is not None else (("left", left),):
         _check(t, f"{name} rows", left.dtype, 2)
         if t.shape != left.shape:
             raise KernelError(f"branches of {tuple(left.shape)} and {tuple(right.shape)}")
     tokens, hidden = left.shape
-    for t in (wa, wb) if w is None else (wa, wb, w):
+    for t in (wa, wb, w):
+        if t is None:
+            continue
         _check(t, "norm weight", torch.float32, 1)
         if t.shape[0] != hidden:
             raise KernelError(f"a norm weight of {t.shape[0]} entries for rows of {hidden}")
@@ -1518,11 +1591,13 @@ def _normed_pair(left, right, wa, wb, scale, pair_eps, residual, rows, w, eps, o
         _ptr(left), _ptr(right), _code(left), _ptr(wa), _ptr(wb), float(scale), float(pair_eps), _ptr(residual), _ptr(rows), _ptr(w), float(eps),
         _ptr(out), _ptr(total), out_rows, hidden, _stream(),
     )
-    _done(status, "normed_pair" if residual is None else "add normed_pair + rmsnorm", shape=(out_rows, hidden))
+    what = "normed_pair" if right is not None else "normed_output"
+    _done(status, what if residual is None else f"add {what} + rmsnorm", shape=(out_rows, hidden))
 
 
 def normed_pair(left, right, wa, wb, scale, pair_eps):
-    """``scale * (norm(left) * wa + norm(right) * wb)`` with RMS norms over whole rows: float32 ``[T, H]``."""
+    """``scale * (norm(left) * wa + norm(right) * wb)`` with RMS norms over whole rows: float32 ``[T, H]``.
+    ``right`` and ``wb`` None: one branch alone."""
     total = torch.empty(left.shape, dtype=torch.float32, device=left.device)
     _normed_pair(left, right, wa, wb, scale, pair_eps, None, None, None, 0.0, None, total, left.shape[0])
     return total
@@ -1765,6 +1840,102 @@ def delta_output(x, gate, weight, heads, eps, out):
     return out
 
 
+# --------------------------------------------------------------------------- matrix memory with exponential gates
+
+
+def memory_gates(logits, cap, top, step):
+    """``logits[T, 2 heads]`` (float32; input gates, then forget gates) to the factors on the old state and on
+    the new write and to ``exp(-m)`` of the running maximum ``m``, float32 ``[T, heads]`` each; ``top`` (float32
+    ``[slots, heads]``) holds each request's ``m`` and is brought up to date."""
+    _check(logits, "gate logits", torch.float32, 2)
+    tokens, heads = logits.shape[0], logits.shape[1] // 2
+    stride = _slot_rows(top, "running maximum", torch.float32)
+    if logits.shape[1] != 2 * heads or top.shape[1:] != (heads,):
+        raise KernelError(f"logits {tuple(logits.shape)} and a running maximum {tuple(top.shape)} do not fit")
+    keep, add, floor = (torch.empty((tokens, heads), dtype=torch.float32, device=logits.device) for _ in range(3))
+    status = library().shiso_memory_gates(
+        _ptr(logits), float(cap), top.data_ptr(), stride, _ptr(step.q_start), _ptr(step.state_slots), _ptr(keep), _ptr(add), _ptr(floor),
+        step.num_seqs, heads, _stream())
+    _done(status, "memory_gates", shape=(tokens, heads))
+    return keep, add, floor
+
+
+def _memory_state(state, normaliser, heads, dim, vdim):
+    if state.shape[1:] != (heads, dim, vdim) or normaliser.shape[1:] != (heads, dim):
+        raise KernelError(f"a state {tuple(state.shape)} and a normaliser {tuple(normaliser.shape)} for {heads} heads of {dim} x {vdim}")
+    return _slot_rows(state, "recurrent state", torch.float32), _slot_rows(normaliser, "normaliser", torch.float32)
+
+
+def memory_recurrence(q, k, v, keep, add, state, normaliser, step, heads, dim, vdim):
+    """Per head ``S <- keep S + add k v^T``, ``n <- keep n + add k`` over each sequence's rows in order; returns
+    ``S^T q`` (float32 ``[T, heads * vdim]``) and ``n . q`` (``[T, heads]``) of every row, read behind its own write.
+    ``state`` and ``normaliser``: float32 ``[slots, heads, dim(, vdim)]``.  Inputs may be column ranges."""
+    act, tokens = q.dtype, q.shape[0]
+    q_ld, k_ld, v_ld = _rows(q, "q", act, heads * dim), _rows(k, "k", act, heads * dim), _rows(v, "v", act, heads * vdim)
+    for name, t in (("keep", keep), ("add", add)):
+        _check(t, name, torch.float32, 2)
+        if t.shape != (tokens, heads):
+            raise KernelError(f"{name} of {tuple(t.shape)} for {tokens} rows of {heads} heads")
+    stride, norm_stride = _memory_state(state, normaliser, heads, dim, vdim)
+    out = torch.empty((tokens, heads * vdim), dtype=torch.float32, device=q.device)
+    norm_out = torch.empty((tokens, heads), dtype=torch.float32, device=q.device)
+    status = library().shiso_state_recurrence_factors(
+        q.data_ptr(), k.data_ptr(), v.data_ptr(), q_ld, k_ld, v_ld, _CODES[act], _ptr(keep), _ptr(add), state.data_ptr(), stride,
+        normaliser.data_ptr(), norm_stride, _ptr(step.q_start), _ptr(step.state_slots), _ptr(out), _ptr(norm_out), tokens, step.num_seqs,
+        heads, dim, vdim, _sm_count(), _stream())
+    _done(status, "memory_recurrence", shape=(tokens, heads, dim, vdim))
+    return out, norm_out
+
+
+def memory_output(raw, norm_out, floor, gate, weight, heads, vdim, q_scale, denominator_eps, eps, out):
+    """``o = q_scale raw / (max(|q_scale n . q|, floor) + denominator_eps)`` per head, ``out = o / rms(o) * weight *
+    sigmoid(gate)``: ``raw`` float32 ``[T, heads * vdim]``, ``norm_out`` and ``floor`` ``[T, heads]``, ``weight`` float32
+    ``[heads * vdim]``, ``gate`` and ``out`` ``[T, heads * vdim]`` of one type (column ranges may be given)."""
+    tokens, width = out.shape
+    for name, t, n in (("raw", raw, heads * vdim), ("n . q", norm_out, heads), ("floor", floor, heads)):
+        _check(t, name, torch.float32, 2)
+        if t.shape != (tokens, n):
+            raise KernelError(f"{name} of {tuple(t.shape)} for {tokens} rows of {heads} heads of {vdim}")
+    _check(weight, "norm weight", torch.float32, 1)
+    if width != heads * vdim or weight.shape[0] != width or gate.shape[0] != tokens:
+        raise KernelError(f"rows of {width} and a weight of {weight.shape[0]} for {heads} heads of {vdim}")
+    gate_ld, out_ld = _rows(gate, "gate", out.dtype, width), _rows(out, "out", None, width)
+    status = library().shiso_memory_output(
+        _ptr(raw), _ptr(norm_out), _ptr(floor), gate.data_ptr(), gate_ld, _code(out), _ptr(weight), out.data_ptr(), out_ld, tokens, heads,
+        vdim, float(q_scale), float(denominator_eps), float(eps), _stream())
+    _done(status, "memory_output", shape=(tokens, heads, vdim))
+    return out
+
+
+def memory_step(x, gate_w, gate_b, proj, weight, state, normaliser, top, step, heads, dim, vdim, cap, q_scale, denominator_eps, eps, out):
+    """For a step of one row per sequence: the gates' logits ``gate_w x + gate_b`` and ``memory_gates``,
+    ``memory_recurrence`` and ``memory_output`` of ``proj[T, q | k | v | gate]`` in one launch.  Writes ``out[T, heads *
+    vdim]`` and returns it, or None (nothing done) for a step that holds longer portions or for gate
+    matrices of another type than the rows."""
+    if not getattr(step, "all_decode", False) or gate_w.dtype != x.dtype or proj.dtype != x.dtype:
+        return None
+    act, (tokens, hidden) = x.dtype, x.shape
+    _check(x, "x", None, 2)
+    _check(gate_w, "gate matrix", act, 2)
+    _check(gate_b, "gate bias", torch.float32, 1)
+    _check(weight, "norm weight", torch.float32, 1)
+    qk, v = heads * dim, heads * vdim
+    ld, out_ld = _rows(proj, "projected rows", act, 2 * (qk + v)), _rows(out, "out", act, v)
+    if gate_w.shape != (2 * heads, hidden) or gate_b.shape[0] != 2 * heads or weight.shape[0] != v or proj.shape[0] != tokens or out.shape[0] != tokens:
+        raise KernelError(f"gates {tuple(gate_w.shape)}, weight {tuple(weight.shape)} and rows {tuple(proj.shape)} do not fit")
+    if top.shape[1:] != (heads,):
+        raise KernelError(f"a running maximum of shape {tuple(top.shape)} for {heads} heads")
+    stride, norm_stride = _memory_state(state, normaliser, heads, dim, vdim)
+    top_stride = _slot_rows(top, "running maximum", torch.float32)
+    at, size = proj.data_ptr(), proj.element_size()
+    status = library().shiso_memory_step(
+        _ptr(x), _ptr(gate_w), _ptr(gate_b), at, at + size * qk, at + size * 2 * qk, at + size * (2 * qk + v), ld, _CODES[act], _ptr(weight),
+        state.data_ptr(), stride, normaliser.data_ptr(), norm_stride, top.data_ptr(), top_stride, _ptr(step.q_start), _ptr(step.state_slots),
+        out.data_ptr(), out_ld, step.num_seqs, hidden, heads, dim, vdim, float(cap), float(q_scale), float(denominator_eps), float(eps), _stream())
+    _done(status, "memory_step", shape=(tokens, heads, dim, vdim))
+    return out
+
+
 # --------------------------------------------------------------------------- latent attention
 
 
@@ -1929,13 +2100,14 @@ UNGATED_RELU2 = "relu2"
 MOE_MAX_EXPERTS = 256  # router outputs the grouping kernels keep in shared memory
 
 
-def routed_experts(x, ids, weights, gate_up, down, extra=None, act="silu", limit=0.0, extra_gate=None, identity=0):
+def routed_experts(x, ids, weights, gate_up, down, extra=None, act="silu", limit=0.0, extra_gate=None, identity=0, weigh_input=False):
     """``out[t] = extra[t] + sum_j weights[t, j] * expert_{ids[t, j]}(x[t])`` with gated experts
     ``down[e] pair(gate x, up x)`` (``act`` / ``limit``: the pairs of ``glu_act``), ``gate_up[e] =
     [gate; up]``: ``x[T, H]``, ``gate_up[E, 2F, H]``, ``down[E, H, F]``; with ``act = "relu2"`` ungated
     experts ``down[e] relu(up x)^2`` and ``gate_up[E, F, H]`` holds the up matrices.  Ids ``E .. E + identity - 1`` are
     identity experts: one adds ``weights[t, j] * x[t]``.  ``extra_gate`` (float32 ``[T, 1]``, a column
-    range may be given) multiplies ``extra[t]`` by its sigmoid.  The (row, choice) pairs are grouped
+    range may be given) multiplies ``extra[t]`` by its sigmoid.  ``weigh_input``: ``sum_j expert_{ids[t, j]}(weights[t, j]
+    * x[t])`` instead.  The (row, choice) pairs are grouped
     by expert on the device; nothing about the routing reaches the host."""
     gated = act != UNGATED_RELU2
     _check(x, "x", None, 2)
@@ -1972,7 +2144,8 @@ def routed_experts(x, ids, weights, gate_up, down, extra=None, act="silu", limit
     status = library().shiso_routed_experts(
         _ptr(x), _code(x), _ptr(ids), _ptr(weights), _ptr(gate_up), _ptr(down), _code(gate_up), _ptr(extra),
         extra_gate.data_ptr() if extra_gate is not None else 0, gate_ld, _ptr(out), _ptr(ints),
-        _ptr(mid), _ptr(y), tokens, hidden, ff, experts, int(identity), top, _GLU_ACTS[act] if gated else 3, float(limit), _stream(),
+        _ptr(mid), _ptr(y), tokens, hidden, ff, experts, int(identity), top, _GLU_ACTS[act] if gated else 3, float(limit), int(bool(weigh_input)),
+        _stream(),
     )
     _done(status, "routed_experts", 6, shape=(tokens, top, experts, ff, hidden))
     return out

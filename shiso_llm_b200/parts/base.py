@@ -15,6 +15,7 @@ Kinds of part and what each must provide:
 ``Block``            ``forward(stream, step, cache)`` - the arrangement of the above
 ``Embedding``        ``forward(step)`` -> float32 residual rows
 ``Head``             ``forward(x)`` -> float32 logits
+``SideInput``        ``forward(rows, step)`` -> something to add to the stream behind a layer
 """
 
 from __future__ import annotations
@@ -64,10 +65,15 @@ class PagedKV:
     dtype: Optional[torch.dtype] = None
     every: int = 1
     keep_first: int = 0
+    num_v_heads: Optional[int] = None  # fewer value heads than key heads: neighbouring key heads share one (None: as many)
 
     @property
     def value_dim(self) -> int:
         return self.head_dim if self.v_head_dim is None else self.v_head_dim
+
+    @property
+    def value_heads(self) -> int:
+        return self.num_kv_heads if self.num_v_heads is None else self.num_v_heads
 
 
 @dataclass(frozen=True)
@@ -186,6 +192,13 @@ class Head(Part):
         raise NotImplementedError
 
 
+class SideInput(Part):
+    def forward(self, rows: torch.Tensor, step, scale: float):
+        """``rows[T, hidden]``: the stream itself in the compute type, not normed.  Returns what waits
+        on the stream (a tensor, ``DeferredLinear`` or ``NormedOutput``), already times ``scale``."""
+        raise NotImplementedError
+
+
 class DeferredLinear:
     """A block's output projection that has not run yet: ``x @ w^T``.
 
@@ -214,6 +227,18 @@ class NormedPair:
 
     def materialize(self) -> torch.Tensor:
         return self.ops.normed_pair(self.left, self.right, self.left_w, self.right_w, self.scale, self.eps)
+
+
+class NormedOutput:
+    """A sublayer output that is not formed yet: ``scale * norm(y) * w``, the RMS norm of its rows over
+    the model width (``eps`` inside the root).  It waits on the stream as a ``NormedPair`` does, and the
+    same norms take it."""
+
+    def __init__(self, ops, y, w, scale: float, eps: float):
+        self.ops, self.y, self.w, self.scale, self.eps = ops, y, w, scale, eps
+
+    def materialize(self) -> torch.Tensor:
+        return self.ops.normed_pair(self.y, None, self.w, None, self.scale, self.eps)
 
 
 class DeferredNorm:
@@ -353,7 +378,7 @@ class Stream:
             if not getattr(norm, "takes_several", False):
                 raise RuntimeError(f"{type(norm).__name__} adds one block output at a time, {len(delta)} are waiting")
             return norm.add_apply(self.residual, tuple(d.materialize() if isinstance(d, DeferredLinear) else d for d in delta))
-        if isinstance(delta, NormedPair) and not getattr(norm, "takes_pairs", False):
+        if isinstance(delta, (NormedPair, NormedOutput)) and not getattr(norm, "takes_pairs", False):
             self.residual = norm.env.ops.stream_add(self.residual, (delta.materialize(),), None)
             return norm.apply(self.residual)
         if isinstance(delta, DeferredLinear):
@@ -365,15 +390,27 @@ class Stream:
 
     def take_pending(self, norm: Optional[Norm] = None) -> Optional[torch.Tensor]:
         """The block output still waiting to be added, as a tensor (or None); a tuple of tensors
-        where a layer left several.  A ``NormedPair`` stays one where ``norm`` says it takes those."""
+        where a layer left several.  A ``NormedPair`` or ``NormedOutput`` stays one where ``norm`` says it
+        takes those."""
         delta, self.pending = self.pending, None
-        if isinstance(delta, NormedPair):
+        if isinstance(delta, (NormedPair, NormedOutput)):
             return delta if norm is not None and getattr(norm, "takes_pairs", False) else delta.materialize()
         if isinstance(delta, tuple):
             return tuple(d.materialize() if isinstance(d, DeferredLinear) else d for d in delta)
         if isinstance(delta, DeferredLinear):
             delta = delta.materialize()
         return delta
+
+    def add_now(self, deltas, scale: float, env, want_rows: bool) -> Optional[torch.Tensor]:
+        """``residual += scale * sum(deltas)`` at once, in float32 and in place; returns the new rows in
+        the compute type of ``env`` where they are wanted (for a part that reads the stream itself)."""
+        if self.pending is not None:
+            raise RuntimeError("a block output is already waiting to be added to the residual")
+        deltas = tuple(d.materialize() if isinstance(d, DeferredLinear) else d for d in deltas)
+        self.current = env.ops.stream_add_rows(self.residual, deltas, scale, env.dtype if want_rows else None)
+        if self.observer is not None:
+            self.observer(self)
+        return self.current
 
     def add(self, delta) -> None:
         if self.pending is not None:
@@ -433,3 +470,4 @@ FEED_FORWARDS = Registry("feed-forward")
 BLOCKS = Registry("block arrangement")
 EMBEDDINGS = Registry("embedding")
 HEADS = Registry("head")
+SIDES = Registry("side input")

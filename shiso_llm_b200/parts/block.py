@@ -13,7 +13,7 @@ compute type for the next reader.
 
 from __future__ import annotations
 
-from .base import BLOCKS, FEED_FORWARDS, MIXERS, NORMS, Block
+from .base import BLOCKS, FEED_FORWARDS, MIXERS, NORMS, SIDES, Block
 
 
 @BLOCKS.register("pre_norm")
@@ -57,7 +57,12 @@ class PreNormBlock(Block):
 class ParallelPreNormBlock(Block):
     """``x' = x + mixer(h) + ff(h)`` with ``h = norm(x)``: one norm, read by both sublayers.
     Both outputs wait on the stream together; the next norm adds them in float32 while it
-    normalises.  A layer without a feed-forward leaves the mixer's output alone."""
+    normalises.  A layer without a feed-forward leaves the mixer's output alone.
+
+    ``params``: ``scale`` (default 1) multiplies whatever the layer adds.  With a ``side`` input the layer
+    goes on: ``x'' = x' + side(x')``, where ``side`` reads the stream as the sublayers have left it; the
+    sublayers' outputs are then added at once, by a kernel that also hands the new rows on in the
+    compute type, and what the side input gives waits for the next norm."""
 
     def __init__(self, spec, env, layer):
         super().__init__(spec, env)
@@ -67,9 +72,11 @@ class ParallelPreNormBlock(Block):
         self.norm = NORMS.build(layer.mixer_norm, env)
         self.mixer = MIXERS.build(layer.mixer, env)
         self.feed_forward = FEED_FORWARDS.build(layer.feed_forward, env) if layer.feed_forward is not None else None
+        self.scale = float(spec.params.get("scale", 1.0))
+        self.side = SIDES.build(layer.side, env) if layer.side is not None else None
 
     def sub_parts(self):
-        return [p for p in (self.norm, self.mixer, self.feed_forward) if p is not None]
+        return [p for p in (self.norm, self.mixer, self.feed_forward, self.side) if p is not None]
 
     def tensor_specs(self):
         specs = []
@@ -87,7 +94,12 @@ class ParallelPreNormBlock(Block):
     def forward(self, stream, step, cache):
         h = stream.normed(self.norm)
         mixed = self.mixer.forward(h, step, cache)
-        if self.feed_forward is None:
+        if self.side is not None or self.scale != 1.0:
+            outs = (mixed,) if self.feed_forward is None else (mixed, self.feed_forward.forward(h, step))
+            rows = stream.add_now(outs, self.scale, self.env, self.side is not None)
+            if self.side is not None:
+                stream.add(self.side.forward(rows, step, self.scale))
+        elif self.feed_forward is None:
             stream.add(mixed)
         else:
             stream.add((mixed, self.feed_forward.forward(h, step)))

@@ -150,6 +150,9 @@ class RoutedExperts(FeedForward):
     logits only.  ``activation = "relu2"`` makes the experts ungated, ``W_down relu(W_up x)^2``, with names
     ``up`` and ``down`` each.
 
+    ``weigh = "input"`` multiplies a chosen expert's INPUT by its weight instead of its output: the sum of
+    ``expert_e(w_e x)``, in which the weight passes the activation.
+
     The expert matrices are stacked ``[experts, 2 ff, hidden]`` (gate over up) and
     ``[experts, hidden, ff]`` when bound; a step's (token, choice) pairs are grouped by expert
     on the device and each group runs as row tiles of one launch, so nothing about the routing
@@ -178,6 +181,9 @@ class RoutedExperts(FeedForward):
         if not known or (self.activation == "swish_clamped" and self.limit <= 0.0):
             raise UnsupportedShape("expert activation", (self.activation, self.limit), f"one of {GLU_ACTIVATIONS} or {UNGATED_RELU2!r}; a clamped pair needs a positive limit")
         self.in_names = ("up",) if self.activation == UNGATED_RELU2 else ("gate", "up")
+        self.weigh = p.get("weigh", "output")
+        if self.weigh not in ("output", "input"):
+            raise UnsupportedShape("weigh", self.weigh, "expected 'output' or 'input'")
         if not 0 <= self.identity < self.experts:
             raise UnsupportedShape("identity experts", self.identity, f"fewer than the router's {self.experts} outputs")
         if self.shared_gate_name is not None and p.get("shared") is None:
@@ -260,4 +266,6 @@ class RoutedExperts(FeedForward):
             more["extra_gate"] = logits[:, self.experts : self.experts + 1]  # [T, 1] float32 logits
         if self.identity:
             more["identity"] = self.identity
+        if self.weigh == "input":
+            more["weigh_input"] = True
         return ops.routed_experts(x, ids, weights, self.gate_up, self.down, extra, **more)

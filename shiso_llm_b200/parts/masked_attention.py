@@ -11,7 +11,11 @@ projected (bias included), before any norm, so ``vdim = dim``.  Then, per query 
     norm over all query heads' entries together and one over all key heads', with weights of
     ``[heads * dim]`` and ``[kv_heads * dim]``, taken before the rotation (if any);
   * the position encoding on the first ``rotary_dim`` entries (half-split pairs; cosine and sine
-    times the encoding's ``magnitude``).
+    times the encoding's ``magnitude``).  An encoding of neighbouring pairs runs in the same kernels:
+    scores do not care in which order a head's entries stand, so the rows of ``W_q`` and ``W_k`` are put in
+    half-split order when bound (without a head norm or biases, whose entries would have to follow).
+
+``value_share = s`` gives the layer ``kv_heads / s`` value heads: ``s`` neighbouring key heads read one.
 
 ``q_temperature = {"coef": c, "every": n}`` multiplies the query at position ``p`` by
 ``1 + c * ln(floor((p + 1) / n) + 1)`` (with the joined norm).  ``score = (q . k) * scale``, then ``softcap * tanh(score / softcap)`` if a cap is given.  What
@@ -54,7 +58,7 @@ EVERYTHING = 1 << 30  # the size of a window that never ends
 class MaskedAttention(Mixer):
     """``params``: ``hidden_size``, ``num_heads``, ``num_kv_heads``, ``head_dim``, ``v_head_dim``,
     ``scale``, ``mask``, ``weights``, optionally ``softcap``, ``head_norm`` (+ ``eps``, ``q_norm``,
-    ``k_norm``), ``position``, ``key_bias``, ``sink``, ``gate`` (+ ``gate_per``), ``values``, ``q_temperature``,
+    ``k_norm``), ``position``, ``key_bias``, ``sink``, ``gate`` (+ ``gate_per``), ``values``, ``value_share``, ``q_temperature``,
     ``q_bias`` / ``k_bias`` / ``v_bias``, and the names ``q_proj``, ``k_proj``, ``v_proj``, ``out_proj``."""
 
     def __init__(self, spec, env):
@@ -97,6 +101,10 @@ class MaskedAttention(Mixer):
             raise UnsupportedShape("values", self.values, "expected 'projected' or 'keys'")
         if self.values == "keys" and self.vdim != self.dim:
             raise UnsupportedShape("v_head_dim", self.vdim, f"values that are the keys have the keys' size {self.dim}")
+        share = int(p.get("value_share", 1))
+        if share < 1 or self.kv_heads % share or (share > 1 and self.values == "keys"):
+            raise UnsupportedShape("value_share", share, f"must divide the {self.kv_heads} key heads, whose values are projected")
+        self.v_heads = self.kv_heads // share
         self.gate_per = p.get("gate_per", "head")
         if self.gate_per not in ("head", "element"):
             raise UnsupportedShape("gate_per", self.gate_per, "expected 'head' or 'element'")
@@ -108,12 +116,15 @@ class MaskedAttention(Mixer):
         joined = self.head_norm == "joined"
         if joined and float(getattr(self.position, "magnitude", 1.0)) != 1.0:
             raise UnsupportedShape("position", p["position"].kind, "the kernel of the joined norm rotates without a magnitude on cosine and sine")
+        if joined and share > 1:
+            raise UnsupportedShape("value_share", share, "the kernel of the joined norm stores as many value heads as key heads")
         if (self.values == "keys" or self.q_temperature is not None) and not joined:
             raise UnsupportedShape("head_norm", self.head_norm, "values that are the keys and a query temperature come with the joined norm's kernel")
         if joined and (p.get("q_norm") is None or p.get("k_norm") is None):
             raise UnsupportedShape("head_norm", self.head_norm, "the joined norm has a weight for the queries and one for the keys")
-        if getattr(self.position, "interleaved", False):
-            raise UnsupportedShape("position", p["position"].kind, "the kernel that prepares the heads rotates half-split pairs")
+        self.interleaved = bool(getattr(self.position, "interleaved", False))
+        if self.interleaved and (self.head_norm is not None or self.values == "keys" or p.get("q_bias") is not None or p.get("k_bias") is not None):
+            raise UnsupportedShape("position", p["position"].kind, "neighbouring pairs come without a head norm, biases or values that are the keys")
         self.names = {k: p.get(k) for k in ("q_proj", "k_proj", "v_proj", "out_proj", "q_bias", "k_bias", "v_bias", "q_norm", "k_norm",
                                              "key_bias", "sink", "gate")}
         if self.names["key_bias"] is not None and self.weights != "sigmoid":
@@ -129,7 +140,7 @@ class MaskedAttention(Mixer):
 
     @property
     def kv_cols(self):
-        return self.kv_heads * (self.dim + (self.vdim if self.values == "projected" else 0))
+        return self.kv_heads * self.dim + (self.v_heads * self.vdim if self.values == "projected" else 0)
 
     @property
     def gate_cols(self):
@@ -143,6 +154,13 @@ class MaskedAttention(Mixer):
     def out_width(self):
         return self.heads * self.vdim
 
+    def _half_split(self, matrix, heads):
+        """The rows of a projection in half-split order: each head's neighbours ``(2i, 2i + 1)`` to ``(i, i + dims/2)``."""
+        _, dims = self.position.rotary()
+        order = torch.arange(self.dim, device=matrix.device)
+        order = torch.cat([order[0:dims:2], order[1:dims:2], order[dims:]])
+        return matrix.view(heads, self.dim, -1)[:, order].reshape(matrix.shape)
+
     def sub_parts(self):
         return [self.position]
 
@@ -151,11 +169,11 @@ class MaskedAttention(Mixer):
         specs = [
             TensorSpec(n["q_proj"], (self.heads * self.dim, self.hidden)),
             TensorSpec(n["k_proj"], (self.kv_heads * self.dim, self.hidden)),
-            TensorSpec(n["out_proj"], (self.hidden, self.heads * self.vdim)),
+            TensorSpec(n["out_proj"], (self.hidden, self.out_width)),
         ]
         if self.values == "projected":
-            specs.append(TensorSpec(n["v_proj"], (self.kv_heads * self.vdim, self.hidden)))
-        for key, rows in (("q_bias", self.heads * self.dim), ("k_bias", self.kv_heads * self.dim), ("v_bias", self.kv_heads * self.vdim)):
+            specs.append(TensorSpec(n["v_proj"], (self.v_heads * self.vdim, self.hidden)))
+        for key, rows in (("q_bias", self.heads * self.dim), ("k_bias", self.kv_heads * self.dim), ("v_bias", self.v_heads * self.vdim)):
             if n[key] is not None and not (key == "v_bias" and self.values == "keys"):
                 specs.append(TensorSpec(n[key], (rows,), VECTOR, NORMAL))
         joined = self.head_norm == "joined"
@@ -174,13 +192,15 @@ class MaskedAttention(Mixer):
         n = self.names
         projected = ("q_proj", "k_proj", "v_proj") if self.values == "projected" else ("q_proj", "k_proj")
         mats = [tensors[n[k]] for k in projected]
+        if self.interleaved:
+            mats[0], mats[1] = self._half_split(mats[0], self.heads), self._half_split(mats[1], self.kv_heads)
         if n["gate"] is not None:
             mats.append(tensors[n["gate"]])
         if len({m.dtype for m in mats}) > 1:
             mats = [m.float() for m in mats]
         self.in_matrix = torch.cat(mats, dim=0).contiguous()
         if any(n[k] is not None for k in ("q_bias", "k_bias", "v_bias")):
-            rows = (self.heads * self.dim, self.kv_heads * self.dim, self.kv_heads * self.vdim)
+            rows = (self.heads * self.dim, self.kv_heads * self.dim, self.v_heads * self.vdim)
             parts = [tensors[n[k]].to(torch.float32) if n[k] is not None else torch.zeros(r, dtype=torch.float32, device=self.in_matrix.device)
                      for k, r in zip(("q_bias", "k_bias", "v_bias")[: len(projected)], rows)]
             if n["gate"] is not None:
@@ -193,31 +213,36 @@ class MaskedAttention(Mixer):
         self.sink = tensors[n["sink"]] if n["sink"] is not None else None
 
     def cache_spec(self):
-        return PagedKV(self.kv_heads, self.dim, None if self.causal else self.size, self.vdim, keep_first=self.keep_first)
+        return PagedKV(self.kv_heads, self.dim, None if self.causal else self.size, self.vdim, keep_first=self.keep_first,
+                       num_v_heads=self.v_heads if self.v_heads != self.kv_heads else None)
 
-    def _attend(self, proj, step, cache, out=None):
-        """Prepares the heads of the projected rows in place, stores keys and values, and attends;
-        ``out``: rows to write (of their own when None)."""
+    def _prepare(self, proj, step, cache):
+        """Prepares the heads of the projected rows in place and stores keys and values; returns the
+        query columns and the block table."""
         ops = self.env.ops
         inv_freq, rotary_dim = self.position.rotary()
         table = step.block_tables[cache.group]
+        if self.head_norm == "joined":
+            turn = {"inv_freq": inv_freq, "rotary_dim": rotary_dim} if rotary_dim else {}
+            return ops.joined_norm_store(
+                proj, self.heads, self.kv_heads, self.dim, self.vdim, self.q_weight, self.k_weight, self.eps, self.q_temperature,
+                self.values == "keys", step, cache.k, cache.v, table, cache.page_size, **turn,
+            ), table
+        return ops.head_prepare_store(
+            proj, self.heads, self.kv_heads, self.dim, self.vdim, self.q_weight, self.k_weight, self.eps, self.head_norm,
+            inv_freq, rotary_dim, float(getattr(self.position, "magnitude", 1.0)), step, cache.k, cache.v, table, cache.page_size,
+        ), table
+
+    def _attend(self, proj, step, cache, out=None):
+        """``_prepare``, then attention; ``out``: rows to write (of their own when None)."""
+        ops = self.env.ops
         gate = proj[:, self.q_cols + self.kv_cols :] if self.names["gate"] is not None else None
         more = {"gate_per_element": True} if gate is not None and self.gate_per == "element" else {}
         if self.sink is not None:
             more["sink"] = self.sink
         if out is not None:
             more["out"] = out
-        if self.head_norm == "joined":
-            turn = {"inv_freq": inv_freq, "rotary_dim": rotary_dim} if rotary_dim else {}
-            q = ops.joined_norm_store(
-                proj, self.heads, self.kv_heads, self.dim, self.vdim, self.q_weight, self.k_weight, self.eps, self.q_temperature,
-                self.values == "keys", step, cache.k, cache.v, table, cache.page_size, **turn,
-            )
-        else:
-            q = ops.head_prepare_store(
-                proj, self.heads, self.kv_heads, self.dim, self.vdim, self.q_weight, self.k_weight, self.eps, self.head_norm,
-                inv_freq, rotary_dim, float(getattr(self.position, "magnitude", 1.0)), step, cache.k, cache.v, table, cache.page_size,
-            )
+        q, table = self._prepare(proj, step, cache)
         return ops.masked_attention(
             q, self.heads, cache.k, cache.v, table, cache.page_size, self.scale, self.mask, self.size, self.keep_first, step,
             sigmoid=self.weights == "sigmoid", key_bias=self.key_bias, softcap=self.softcap, gate=gate, **more,
@@ -237,7 +262,7 @@ class MaskedAttention(Mixer):
         if (
             from_qkv is not None and self.mask == "window" and self.weights == "softmax" and self.softcap is None and self.sink is None
             and self.names["gate"] is None and self.head_norm == "before" and self.q_weight is not None and self.k_weight is not None
-            and self.dim == self.vdim and float(getattr(self.position, "magnitude", 1.0)) == 1.0
+            and self.dim == self.vdim and self.v_heads == self.kv_heads and float(getattr(self.position, "magnitude", 1.0)) == 1.0
         ):
             # steps of single tokens, heads of 64 rotated whole: norm, rotation, cache store and
             # attention in the one launch the framework's other attention layers take (None otherwise)

@@ -76,9 +76,13 @@ class Model:
         return [self.embedding, *self.blocks, self.final_norm, self.head]
 
     def tensor_specs(self) -> list[TensorSpec]:
-        specs = []
+        specs, shared = [], {}
         for part in self.parts():
-            specs += part.tensor_specs()
+            for spec in part.tensor_specs():
+                if shared.get(spec.name) == spec and spec.shared:
+                    continue  # a table that several parts read
+                shared[spec.name] = spec
+                specs.append(spec)
         for name, rows in self.entry_vectors.items():
             specs.append(TensorSpec(name, (rows, self.plan.hidden_size), VECTOR, NORMAL))
         for name in self.entry_mixes:

@@ -22,7 +22,7 @@ from __future__ import annotations
 import torch
 
 from ..weights.spec import NORMAL, ONES, VECTOR, TensorSpec
-from .base import NORMS, Norm, NormedPair
+from .base import NORMS, Norm, NormedOutput, NormedPair
 
 
 @NORMS.register("rmsnorm")
@@ -66,6 +66,9 @@ class RMSNorm(Norm):
         if isinstance(delta, NormedPair):
             return self.env.ops.add_normed_pair_rmsnorm(
                 residual, delta.left, delta.right, delta.left_w, delta.right_w, delta.scale, delta.eps, self.weight, self.eps, rows)
+        if isinstance(delta, NormedOutput):
+            return self.env.ops.add_normed_pair_rmsnorm(
+                residual, delta.y, None, delta.w, None, delta.scale, delta.eps, self.weight, self.eps, rows)
         return self.env.ops.add_rmsnorm(residual, delta, self.weight, self.eps, self.env.dtype, rows)
 
     def add_normed(self, residual, y, want_rows=True):

@@ -36,7 +36,8 @@ class LayerSpec:
     """One layer's parts.  ``name`` prefixes the layer's tensor names.
 
     ``block`` chooses the arrangement (how norms, mixer, feed-forward and the
-    residual stream are wired); the other specs are handed to that block.
+    residual stream are wired); the other specs are handed to that block.  ``side``: an input
+    of the layer's own beside the stream (its token once more), for blocks that take one.
     """
 
     name: str
@@ -45,6 +46,7 @@ class LayerSpec:
     mixer_norm: PartSpec
     feed_forward: Optional[PartSpec] = None
     feed_forward_norm: Optional[PartSpec] = None
+    side: Optional[PartSpec] = None
 
 
 @dataclass(frozen=True)

@@ -18,7 +18,8 @@ multiplied by ``magnitude = 0.1 * ln(factor) + 1``; kernels that rotate read it 
 ``PositionEncoding.magnitude``.
 
 Both take ``interleaved`` (default false): pair ``i`` is then the neighbours ``(2i, 2i + 1)``
-instead of ``(i, i + rotary_dim/2)``, on the same ladder.
+instead of ``(i, i + rotary_dim/2)``, on the same ladder.  ``rope_half_split`` takes ``factor``
+(default 1): every frequency is divided by it (positions stretched linearly).
 """
 
 from __future__ import annotations
@@ -41,7 +42,10 @@ class RopeHalfSplit(PositionEncoding):
         if self.rotary_dim % 2 or not 0 < self.rotary_dim <= head_dim:
             raise UnsupportedShape("rotary_dim", self.rotary_dim, f"must be even and at most the head size {head_dim}")
         i = torch.arange(self.rotary_dim // 2, dtype=torch.float64)
-        self.inv_freq = (self.theta ** (-2.0 * i / self.rotary_dim)).to(torch.float32).to(env.device)
+        factor = float(spec.params.get("factor", 1.0))
+        if factor <= 0.0:
+            raise UnsupportedShape("rotation factor", factor, "must be positive")
+        self.inv_freq = (self.theta ** (-2.0 * i / self.rotary_dim) / factor).to(torch.float32).to(env.device)
 
     def rotary(self):
         return self.inv_freq, self.rotary_dim

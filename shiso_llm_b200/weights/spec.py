@@ -30,3 +30,4 @@ class TensorSpec:
     # Random weights: NORMAL draws around ``init_mean`` with ``init_std`` (None: the caller's std).
     init_mean: float = 0.0
     init_std: float | None = None
+    shared: bool = False  # several parts may ask for it (a table they all read); it is loaded once

@@ -46,6 +46,20 @@ def stream_add(residual, deltas, vector, in_place=True):
     return total.to(residual.dtype)
 
 
+def stream_add_rows(residual, deltas, scale, out_dtype):
+    """``residual += scale * sum(deltas)`` in place; the new rows in ``out_dtype`` (None: not wanted)."""
+    residual.copy_((residual.to(F64) + scale * sum(d.to(F64) for d in deltas)).to(residual.dtype))
+    if out_dtype is None:
+        return None
+    return residual if out_dtype == torch.float32 else residual.to(out_dtype)
+
+
+def side_gate(z, table, first_column, ids, feed_index, fed_tokens, out_dtype):
+    """``gelu_tanh(z[t, c]) * table[id_t, first_column + c]``."""
+    e = table[_step_ids(ids, feed_index, fed_tokens)][:, first_column : first_column + z.shape[1]].to(F64)
+    return _glu(z.to(F64), e, "gelu_tanh", 0.0).to(out_dtype)
+
+
 def add_dyt(residual, deltas, alpha, w, b, out_dtype, rows=None):
     """``tanh(alpha * x) * w + b`` of ``x = residual + sum(deltas)``; without ``rows`` the sum is
     stored back into ``residual``."""
@@ -681,10 +695,10 @@ def moe_route(logits, top, group_count, group_keep, scale, sigmoid=False, renorm
     return ids.to(torch.int32), (w * scale).to(torch.float32)
 
 
-def routed_experts(x, ids, weights, gate_up, down, extra=None, act="silu", limit=0.0, extra_gate=None, identity=0):
+def routed_experts(x, ids, weights, gate_up, down, extra=None, act="silu", limit=0.0, extra_gate=None, identity=0, weigh_input=False):
     """``sum_j weights[t, j] * expert_{ids[t, j]}(x[t])`` (+ ``extra``, times ``sigmoid(extra_gate[t])``
     where one is given), in ``x``'s type.  An id from the number of stacked matrices on is an
-    identity expert: its output is ``x[t]``."""
+    identity expert: its output is ``x[t]``.  ``weigh_input``: ``sum_j expert_{ids[t, j]}(weights[t, j] * x[t])``."""
     T, H = x.shape
     x64 = x.to(F64)
     out = torch.zeros(T, H, dtype=F64)
@@ -700,9 +714,10 @@ def routed_experts(x, ids, weights, gate_up, down, extra=None, act="silu", limit
                 assert e < gate_up.shape[0] + identity, f"choice {e} beyond the experts and identity experts"
                 out[t] += float(weights[t, j]) * x64[t]
                 continue
-            y = gate_up[e].to(F64) @ x64[t]
+            into, behind = (float(weights[t, j]), 1.0) if weigh_input else (1.0, float(weights[t, j]))
+            y = gate_up[e].to(F64) @ x64[t] * into
             mid = torch.relu(y) ** 2 if act == "relu2" else _glu(y[:inter], y[inter:], act, limit)
-            out[t] += float(weights[t, j]) * (down[e].to(F64) @ mid)
+            out[t] += behind * (down[e].to(F64) @ mid)
     return out.to(x.dtype)
 
 
@@ -731,11 +746,12 @@ def head_prepare_store(proj, heads, kv_heads, dim, vdim, q_w, k_w, eps, norm_ord
     q = prepare(x[:, :q_cols].reshape(T, heads, dim), q_w)
     proj[:, :q_cols] = q.reshape(T, q_cols).to(proj.dtype)
     if store:
+        v_heads = v_cache.shape[2]  # fewer than key heads where neighbours share one
         k = prepare(x[:, q_cols : q_cols + k_cols].reshape(T, kv_heads, dim), k_w)
-        v = proj[:, q_cols + k_cols : q_cols + k_cols + kv_heads * vdim].reshape(T, kv_heads, vdim)
+        v = proj[:, q_cols + k_cols : q_cols + k_cols + v_heads * vdim].reshape(T, v_heads, vdim)
         rows = _cache_rows(block_table, step.seq_of_token, step.positions, page_size)
         k_cache.view(-1, kv_heads, dim)[rows] = k.to(k_cache.dtype)
-        v_cache.view(-1, kv_heads, vdim)[rows] = v.to(v_cache.dtype)
+        v_cache.view(-1, v_heads, vdim)[rows] = v.to(v_cache.dtype)
     return proj[:, :q_cols]
 
 
@@ -773,11 +789,12 @@ def joined_norm_store(proj, heads, kv_heads, dim, vdim, q_w, k_w, eps, q_tempera
 
 
 def masked_attention(q, heads, k_cache, v_cache, block_table, page_size, scale, mask, size, keep_first, step, *, sigmoid=False,
-                     key_bias=None, softcap=None, gate=None, general=False, gate_per_element=False, sink=None, out=None):
+                     key_bias=None, softcap=None, gate=None, general=False, gate_per_element=False, sink=None, out=None, out_dtype=None):
     T = q.shape[0]
     kv_heads, dim, vdim = k_cache.shape[2], k_cache.shape[3], v_cache.shape[3]
     q64 = q.to(F64).reshape(T, heads, dim)
-    kf, vf = k_cache.view(-1, kv_heads, dim), v_cache.view(-1, kv_heads, vdim)
+    kf, vf = k_cache.view(-1, kv_heads, dim), v_cache.view(-1, v_cache.shape[2], vdim)
+    share = kv_heads // v_cache.shape[2]
     given, out = out, torch.zeros(T, heads, vdim, dtype=F64)
     seq, pos = step.seq_of_token.tolist(), step.positions.tolist()
     for t in range(T):
@@ -803,12 +820,12 @@ def masked_attention(q, heads, k_cache, v_cache, block_table, page_size, scale, 
                 w = torch.softmax(torch.cat([s, sink[h].to(F64).reshape(1)]), dim=0)[:-1]
             else:
                 w = torch.softmax(s, dim=0)
-            out[t, h] = w @ v[:, g, :]
+            out[t, h] = w @ v[:, g // share, :]
             if gate is not None and gate_per_element:
                 out[t, h] *= torch.sigmoid(gate[t, h * vdim : (h + 1) * vdim].to(F64))
             elif gate is not None:
                 out[t, h] *= torch.sigmoid(gate[t, h].to(F64))
-    out = out.reshape(T, heads * vdim).to(q.dtype)
+    out = out.reshape(T, heads * vdim).to(out_dtype or q.dtype)
     return out if given is None else given.copy_(out)
 
 
@@ -827,6 +844,8 @@ def _unit_rms(x, eps):
 
 
 def normed_pair(left, right, wa, wb, scale, pair_eps):
+    if right is None:
+        return (scale * _unit_rms(left, pair_eps) * wa.to(F64)).to(torch.float32)
     return (scale * (_unit_rms(left, pair_eps) * wa.to(F64) + _unit_rms(right, pair_eps) * wb.to(F64))).to(torch.float32)
 
 
@@ -837,6 +856,60 @@ def add_normed_pair_rmsnorm(residual, left, right, wa, wb, scale, pair_eps, w, e
         return rmsnorm(residual, w, eps, left.dtype)
     idx = rows.long()
     return rmsnorm(residual[idx] + delta[idx], w, eps, left.dtype)
+
+
+def map_difference(maps, pairs, groups, second, factor, eps, gate, out):
+    """``maps[T, (group, map, head of the group) x vdim]``: ``d = first - second * other`` per head, over its
+    root mean square, times ``factor`` and ``sigmoid(gate)``; ``out[T, pairs * vdim]`` head by head."""
+    T = maps.shape[0]
+    m = maps.to(F64).reshape(T, groups, 2, pairs // groups, -1)
+    d = _unit_rms(m[:, :, 0] - second * m[:, :, 1], eps).reshape(T, -1) * factor
+    return out.copy_((d * _sigmoid(gate.to(F64))).to(out.dtype))
+
+
+def memory_gates(logits, cap, top, step):
+    """``logits[T, 2 heads]`` (input gates, forget gates): the factors on the old state and on the new
+    write, and ``exp(-m)`` of the running maximum ``m`` (``top[slots, heads]``, brought up to date)."""
+    T, heads = logits.shape[0], logits.shape[1] // 2
+    z = cap * torch.tanh(logits.to(F64) / cap)
+    i, f = z[:, :heads], torch.nn.functional.logsigmoid(z[:, heads:])
+    keep, add, floor = (torch.zeros(T, heads, dtype=F64) for _ in range(3))
+    q_start, slots = step.q_start.tolist(), step.state_slots.tolist()
+    for s in range(step.num_seqs):
+        m = top[slots[s]].to(F64)
+        for t in range(q_start[s], q_start[s + 1]):
+            new = torch.maximum(f[t] + m, i[t])
+            keep[t], add[t], floor[t] = torch.exp(f[t] + m - new), torch.exp(i[t] - new), torch.exp(-new)
+            m = new
+        if q_start[s + 1] > q_start[s]:
+            top[slots[s]] = m.to(top.dtype)
+    return keep.float(), add.float(), floor.float()
+
+
+def memory_recurrence(q, k, v, keep, add, state, normaliser, step, heads, dim, vdim):
+    """Per head ``S <- keep S + add k [v | 1]^T``, ``o = S^T q``; the last column is the normaliser's.
+    Returns float32 ``[T, heads * vdim]`` and ``[T, heads]``."""
+    T = q.shape[0]
+    q64, k64 = (x.to(F64).reshape(T, heads, dim) for x in (q, k))
+    v64 = torch.cat([v.to(F64).reshape(T, heads, vdim), torch.ones(T, heads, 1, dtype=F64)], dim=-1)
+    o = torch.zeros(T, heads, vdim + 1, dtype=F64)
+    q_start, slots = step.q_start.tolist(), step.state_slots.tolist()
+    for s in range(step.num_seqs):
+        if q_start[s + 1] == q_start[s]:
+            continue
+        S = torch.cat([state[slots[s]].to(F64), normaliser[slots[s]].to(F64)[..., None]], dim=-1)
+        for t in range(q_start[s], q_start[s + 1]):
+            S = keep[t].to(F64)[:, None, None] * S + add[t].to(F64)[:, None, None] * k64[t][:, :, None] * v64[t][:, None, :]
+            o[t] = torch.einsum("hi,hij->hj", q64[t], S)
+        state[slots[s]], normaliser[slots[s]] = S[..., :vdim].to(state.dtype), S[..., vdim].to(normaliser.dtype)
+    return o[..., :vdim].reshape(T, -1).to(torch.float32), o[..., vdim].to(torch.float32).contiguous()
+
+
+def memory_output(raw, norm_out, floor, gate, weight, heads, vdim, q_scale, denominator_eps, eps, out):
+    T = raw.shape[0]
+    r = raw.to(F64).reshape(T, heads, vdim) * q_scale
+    o = r / (torch.maximum((norm_out.to(F64) * q_scale).abs(), floor.to(F64)) + denominator_eps)[..., None]
+    return out.copy_((_unit_rms(o, eps).reshape(T, -1) * weight.to(F64) * _sigmoid(gate.to(F64))).to(out.dtype))
 
 
 def stream_concat(residual, deltas, first, out_dtype):
