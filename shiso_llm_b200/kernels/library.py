@@ -111,6 +111,10 @@ _SIGNATURES = {
     "shiso_memory_gates": [P, F, P, LL, P, P, P, P, P, I, I, P],
     "shiso_memory_output": [P, P, P, P, LL, I, P, P, LL, I, I, I, F, F, F, P],
     "shiso_memory_step": [P, P, P, P, P, P, P, LL, I, P, P, LL, P, LL, P, LL, P, P, P, LL, I, I, I, I, I, F, F, F, F, P],
+    "shiso_differential_prefill_supported": [I, I, I],
+    "shiso_differential_prefill": [P, LL, P, P, P, I, P, P, P, LL, P, LL, I, I, I, I, I, I, I, I, LL, F, I, F, F, F, P],
+    "shiso_differential_decode_supported": [I, I, I, I, I],
+    "shiso_differential_decode": [P, LL, P, P, P, I, P, P, P, LL, P, LL, I, I, I, I, I, I, LL, F, I, I, F, F, F, P],
     "shiso_map_difference": [P, P, LL, I, P, LL, I, I, I, I, F, F, F, P],
 }
 

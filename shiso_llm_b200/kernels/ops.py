@@ -1551,6 +1551,60 @@ def map_difference(maps, pairs, groups, second, factor, eps, gate, out):
     return out
 
 
+DIFFERENTIAL_MAX_PARTS = 8  # CTAs (a portable cluster) that share a decoded row's keys
+
+
+def differential_attention(q, pairs, groups, k_cache, v_cache, block_table, page_size, scale, size, keep_first, step, second, factor, eps,
+                           gate, out):
+    """``masked_attention`` of both maps (a window of ``size``) and ``map_difference`` in one launch: long prompt
+    portions by the tensor-memory kernel, steps of single tokens by the TMA kernel.  ``q`` is ``[T, 2 pairs * dim]``
+    in the order key head, map, query head of the group; ``k_cache`` ``[pages, page_size, 2 groups, dim]``, ``v_cache``
+    ``[pages, page_size, groups, vdim]``.  Writes ``out[T, pairs * vdim]`` and returns it, or None (nothing done)
+    where sizes, types or the step are not the kernels'."""
+    lib = library()
+    dim, vdim = k_cache.shape[3], v_cache.shape[3]
+    tokens = q.shape[0]
+    if q.dtype != torch.bfloat16 or keep_first or not scale > 0.0 or k_cache.shape[2] != 2 * groups or v_cache.shape[2] != groups:
+        return None
+    decode = bool(getattr(step, "all_decode", False))
+    if decode:
+        if not lib.shiso_differential_decode_supported(pairs, groups, dim, vdim, page_size):
+            return None
+    elif (
+        tokens < TC_ATTENTION_MIN_TOKENS or getattr(step, "max_q_len", tokens) < TC_ATTENTION_MIN_PORTION
+        or not lib.shiso_differential_prefill_supported(dim, vdim, page_size)
+    ):
+        return None
+    q_ld = _rows(q, "q", torch.bfloat16, 2 * pairs * dim)
+    gate_ld, out_ld = _rows(gate, "gate", torch.bfloat16, pairs * vdim), _rows(out, "out", torch.bfloat16, pairs * vdim)
+    if q.data_ptr() % 16 or (not decode and (q_ld % 8 or gate_ld % 8 or out_ld % 8 or gate.data_ptr() % 16 or out.data_ptr() % 16)):
+        return None
+    _paged(k_cache, "k cache", torch.bfloat16, page_size)
+    _paged(v_cache, "v cache", torch.bfloat16, page_size)
+    _check(block_table, "block table", torch.int32, 2)
+    window = 0 if size >= NO_WINDOW else int(size)
+    if decode:
+        capacity = min(block_table.shape[1] * page_size, size + 2 * 64)
+        splits = max(1, min(DIFFERENTIAL_MAX_PARTS, _sm_count() // (tokens * groups), -(-capacity // 128)))
+        status = lib.shiso_differential_decode(
+            q.data_ptr(), q_ld, _ptr(k_cache), _ptr(v_cache), _ptr(block_table), block_table.shape[1], _ptr(step.positions),
+            _ptr(step.seq_of_token), gate.data_ptr(), gate_ld, out.data_ptr(), out_ld, tokens, pairs, groups, dim, vdim, page_size,
+            k_cache.shape[0], float(scale), window, splits, float(second), float(factor), float(eps), _stream())
+        _done(status, "differential_attention (decode)", shape=(tokens, pairs, dim))
+        return out
+    starts = getattr(step, "h_q_start", None)
+    if starts:
+        tiles = sum(-(-(b - a) // 128) for a, b in zip(starts[:-1], starts[1:]))
+    else:
+        tiles = tokens // 128 + step.num_seqs
+    status = lib.shiso_differential_prefill(
+        q.data_ptr(), q_ld, _ptr(k_cache), _ptr(v_cache), _ptr(block_table), block_table.shape[1], _ptr(step.q_start), _ptr(step.start_pos),
+        gate.data_ptr(), gate_ld, out.data_ptr(), out_ld, tokens, step.num_seqs, tiles, pairs, groups, dim, vdim, page_size, k_cache.shape[0],
+        float(scale), window, float(second), float(factor), float(eps), _stream())
+    _done(status, "differential_attention (tcgen05)", shape=(tokens, pairs, dim))
+    return out
+
+
 # --------------------------------------------------------------------------- norms on a sublayer's output, polynomial activation
 
 

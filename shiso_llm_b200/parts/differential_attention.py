@@ -14,7 +14,8 @@ To the attention kernels the maps are heads: the mixer is ``masked_attention`` (
 encodings, cache) over ``2 heads`` query and ``2 kv_heads`` key heads of which neighbours share a value
 head.  A map's query heads of one key head have to be neighbours for that, so the rows of ``W_q`` are
 put in the order (key head, map, query head of the group) when bound.  The maps' outputs stay float32
-until the difference is taken, normed and gated by one row kernel.
+until the difference is taken, normed and gated by one row kernel - or, in bfloat16 at the sizes of
+``ops.differential_attention``, all of it is one launch, for long prompt portions and for single tokens.
 """
 
 from __future__ import annotations
@@ -82,10 +83,12 @@ class DifferentialAttention(MaskedAttention):
         ops = self.env.ops
         gate = proj[:, self.q_cols + self.kv_cols :]
         q, table = self._prepare(proj, step, cache)
-        sizes = (self.pairs, self.groups, cache.k, cache.v, table, cache.page_size, self.scale, self.size, self.keep_first, step)
         in_one = getattr(ops, "differential_attention", None)
-        if self.mask == "window" and in_one is not None and in_one(q, *sizes, self.second, 1.0 - self.diff, self.eps, gate, out) is not None:
-            return
+        if in_one is not None and self.mask == "window" and self.softcap is None and in_one(
+            q, self.pairs, self.groups, cache.k, cache.v, table, cache.page_size, self.scale, self.size, self.keep_first, step, self.second,
+            1.0 - self.diff, self.eps, gate, out,
+        ) is not None:
+            return  # both maps and their difference in one launch
         maps = ops.masked_attention(q, self.heads, cache.k, cache.v, table, cache.page_size, self.scale, self.mask, self.size,
                                     self.keep_first, step, softcap=self.softcap, out_dtype=torch.float32)
         ops.map_difference(maps, self.pairs, self.groups, self.second, 1.0 - self.diff, self.eps, gate, out)
