@@ -14,7 +14,8 @@
 //   memory_step_kernel    steps of single rows: everything behind the projections in one launch, the two
 //                         gate logits included.
 //
-// The rows between the two are walked by the kernel for scalar-decay recurrences (state_recurrence.cu).
+// The rows between the two are taken 64 at a time on the tensor cores (matrix_memory_chunks.cu, which wants
+// the logarithms of the two factors) or walked by the kernel for scalar-decay recurrences (state_recurrence.cu).
 #include "common.cuh"
 
 namespace {
@@ -38,7 +39,7 @@ struct GatesArgs {
     long long top_stride;
     const int *q_start, *state_slots;
     float *keep, *add, *floor;  // [T, heads]
-    int heads;
+    int heads, logs;  // logs: the two factors' logarithms
     float cap;
 };
 
@@ -81,8 +82,8 @@ __global__ void __launch_bounds__(MG_THREADS) memory_gates_kernel(const GatesArg
         if (lane == 0) last = before;
         if (t < n) {
             const size_t at = (size_t)(first + t) * a.heads + h;
-            a.keep[at] = expf(f + last - now);
-            a.add[at] = expf(i - now);
+            a.keep[at] = a.logs ? f + (last - now) : expf(f + (last - now));
+            a.add[at] = a.logs ? i - now : expf(i - now);
             a.floor[at] = expf(-now);
         }
         m = all;
@@ -300,10 +301,10 @@ int launch_memory_step(const StepArgs& a, int num_seqs, cudaStream_t stream) {
 }  // namespace
 
 SHISO_API int shiso_memory_gates(const float* logits, float cap, float* top, long long top_stride, const int* q_start, const int* state_slots,
-                                 float* keep, float* add, float* floor, int num_seqs, int heads, cudaStream_t stream) {
+                                 float* keep, float* add, float* floor, int num_seqs, int heads, int logs, cudaStream_t stream) {
     if (num_seqs <= 0) return SHISO_OK;
     if (heads <= 0 || num_seqs > 65535 || cap <= 0.0f) return SHISO_ERR_SHAPE;
-    const GatesArgs a = {logits, top, top_stride, q_start, state_slots, keep, add, floor, heads, cap};
+    const GatesArgs a = {logits, top, top_stride, q_start, state_slots, keep, add, floor, heads, logs, cap};
     launch_kernel(memory_gates_kernel, dim3(heads, num_seqs), MG_THREADS, 0, stream, a);
     return launch_status();
 }

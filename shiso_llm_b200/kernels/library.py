@@ -108,7 +108,9 @@ _SIGNATURES = {
     "shiso_stream_add_rows": [P, P, P, I, F, P, I, I, P],
     "shiso_side_gate": [P, P, I, LL, I, I, P, P, P, P, I, I, I, P],
     "shiso_state_recurrence_factors": [P, P, P, LL, LL, LL, I, P, P, P, LL, P, LL, P, P, P, P, I, I, I, I, I, I, P],
-    "shiso_memory_gates": [P, F, P, LL, P, P, P, P, P, I, I, P],
+    "shiso_memory_gates": [P, F, P, LL, P, P, P, P, P, I, I, I, P],
+    "shiso_memory_chunks_supported": [I, I],
+    "shiso_memory_chunks": [P, P, P, LL, LL, LL, P, P, P, LL, P, LL, P, P, P, P, I, I, I, I, P],
     "shiso_memory_output": [P, P, P, P, LL, I, P, P, LL, I, I, I, F, F, F, P],
     "shiso_memory_step": [P, P, P, P, P, P, P, LL, I, P, P, LL, P, LL, P, LL, P, P, P, LL, I, I, I, I, I, F, F, F, F, P],
     "shiso_differential_prefill_supported": [I, I, I],

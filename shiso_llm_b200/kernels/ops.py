@@ -1897,10 +1897,19 @@ def delta_output(x, gate, weight, heads, eps, out):
 # --------------------------------------------------------------------------- matrix memory with exponential gates
 
 
-def memory_gates(logits, cap, top, step):
+def memory_chunks_supported(proj, dim, vdim) -> bool:
+    """Whether prompt portions of these rows (bfloat16 columns ``[q | k | v | ..]``) run in chunks on the tensor
+    cores; the factors are then handed on as logarithms."""
+    return (
+        proj.dtype == torch.bfloat16 and proj.stride(0) % 8 == 0 and proj.data_ptr() % 16 == 0
+        and bool(library().shiso_memory_chunks_supported(int(dim), int(vdim)))
+    )
+
+
+def memory_gates(logits, cap, top, step, logs=False):
     """``logits[T, 2 heads]`` (float32; input gates, then forget gates) to the factors on the old state and on
     the new write and to ``exp(-m)`` of the running maximum ``m``, float32 ``[T, heads]`` each; ``top`` (float32
-    ``[slots, heads]``) holds each request's ``m`` and is brought up to date."""
+    ``[slots, heads]``) holds each request's ``m`` and is brought up to date.  ``logs``: the factors' logarithms."""
     _check(logits, "gate logits", torch.float32, 2)
     tokens, heads = logits.shape[0], logits.shape[1] // 2
     stride = _slot_rows(top, "running maximum", torch.float32)
@@ -1909,7 +1918,7 @@ def memory_gates(logits, cap, top, step):
     keep, add, floor = (torch.empty((tokens, heads), dtype=torch.float32, device=logits.device) for _ in range(3))
     status = library().shiso_memory_gates(
         _ptr(logits), float(cap), top.data_ptr(), stride, _ptr(step.q_start), _ptr(step.state_slots), _ptr(keep), _ptr(add), _ptr(floor),
-        step.num_seqs, heads, _stream())
+        step.num_seqs, heads, int(bool(logs)), _stream())
     _done(status, "memory_gates", shape=(tokens, heads))
     return keep, add, floor
 
@@ -1920,10 +1929,11 @@ def _memory_state(state, normaliser, heads, dim, vdim):
     return _slot_rows(state, "recurrent state", torch.float32), _slot_rows(normaliser, "normaliser", torch.float32)
 
 
-def memory_recurrence(q, k, v, keep, add, state, normaliser, step, heads, dim, vdim):
+def memory_recurrence(q, k, v, keep, add, state, normaliser, step, heads, dim, vdim, logs=False):
     """Per head ``S <- keep S + add k v^T``, ``n <- keep n + add k`` over each sequence's rows in order; returns
     ``S^T q`` (float32 ``[T, heads * vdim]``) and ``n . q`` (``[T, heads]``) of every row, read behind its own write.
-    ``state`` and ``normaliser``: float32 ``[slots, heads, dim(, vdim)]``.  Inputs may be column ranges."""
+    ``state`` and ``normaliser``: float32 ``[slots, heads, dim(, vdim)]``.  Inputs may be column ranges.  ``logs``: the
+    factors come as logarithms, for the kernel that takes 64 rows at a time (``memory_chunks_supported``)."""
     act, tokens = q.dtype, q.shape[0]
     q_ld, k_ld, v_ld = _rows(q, "q", act, heads * dim), _rows(k, "k", act, heads * dim), _rows(v, "v", act, heads * vdim)
     for name, t in (("keep", keep), ("add", add)):
@@ -1933,6 +1943,12 @@ def memory_recurrence(q, k, v, keep, add, state, normaliser, step, heads, dim, v
     stride, norm_stride = _memory_state(state, normaliser, heads, dim, vdim)
     out = torch.empty((tokens, heads * vdim), dtype=torch.float32, device=q.device)
     norm_out = torch.empty((tokens, heads), dtype=torch.float32, device=q.device)
+    if logs:
+        status = library().shiso_memory_chunks(
+            q.data_ptr(), k.data_ptr(), v.data_ptr(), q_ld, k_ld, v_ld, _ptr(keep), _ptr(add), state.data_ptr(), stride, normaliser.data_ptr(),
+            norm_stride, _ptr(step.q_start), _ptr(step.state_slots), _ptr(out), _ptr(norm_out), step.num_seqs, heads, dim, vdim, _stream())
+        _done(status, "memory_recurrence (chunks)", shape=(tokens, heads, dim, vdim))
+        return out, norm_out
     status = library().shiso_state_recurrence_factors(
         q.data_ptr(), k.data_ptr(), v.data_ptr(), q_ld, k_ld, v_ld, _CODES[act], _ptr(keep), _ptr(add), state.data_ptr(), stride,
         normaliser.data_ptr(), norm_stride, _ptr(step.q_start), _ptr(step.state_slots), _ptr(out), _ptr(norm_out), tokens, step.num_seqs,

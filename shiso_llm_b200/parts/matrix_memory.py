@@ -95,9 +95,11 @@ class MatrixMemory(Mixer):
             self.denominator_eps, self.eps, out,
         ) is None:
             logits = ops.linear(x, self.gate_matrix, torch.float32, self.gate_bias)
-            keep, add, floor = ops.memory_gates(logits, self.cap, top, step)
+            fits = getattr(ops, "memory_chunks_supported", None)
+            chunks = {"logs": True} if fits is not None and fits(proj, self.dim, self.vdim) else {}
+            keep, add, floor = ops.memory_gates(logits, self.cap, top, step, **chunks)
             raw, read = ops.memory_recurrence(
-                proj[:, :qk], proj[:, qk : 2 * qk], proj[:, 2 * qk : 2 * qk + v], keep, add, state, normaliser, step, *sizes)
+                proj[:, :qk], proj[:, qk : 2 * qk], proj[:, 2 * qk : 2 * qk + v], keep, add, state, normaliser, step, *sizes, **chunks)
             ops.memory_output(raw, read, floor, proj[:, 2 * qk + v :], self.norm_weight, self.heads, self.vdim, self.dim**-0.5,
                               self.denominator_eps, self.eps, out)
         return DeferredLinear(ops, out, self.out_matrix, self.env.dtype)
