@@ -74,6 +74,8 @@ class ParallelPreNormBlock(Block):
         self.feed_forward = FEED_FORWARDS.build(layer.feed_forward, env) if layer.feed_forward is not None else None
         self.scale = float(spec.params.get("scale", 1.0))
         self.side = SIDES.build(layer.side, env) if layer.side is not None else None
+        # (two outputs at once wait only for norms that add several)
+        self.adds_now = self.side is not None or self.scale != 1.0 or not getattr(self.norm, "takes_several", False)
 
     def sub_parts(self):
         return [p for p in (self.norm, self.mixer, self.feed_forward, self.side) if p is not None]
@@ -94,7 +96,7 @@ class ParallelPreNormBlock(Block):
     def forward(self, stream, step, cache):
         h = stream.normed(self.norm)
         mixed = self.mixer.forward(h, step, cache)
-        if self.side is not None or self.scale != 1.0:
+        if self.adds_now:
             outs = (mixed,) if self.feed_forward is None else (mixed, self.feed_forward.forward(h, step))
             rows = stream.add_now(outs, self.scale, self.env, self.side is not None)
             if self.side is not None:
