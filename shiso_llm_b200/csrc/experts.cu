@@ -410,7 +410,8 @@ __global__ void moe_route_kernel(const float* __restrict__ logits, long long ld,
     for (int e = lane; e < experts; e += 32) {
         const float v = sc[e] * inv;
         sc[e] = v;
-        ch[e] = correction ? v + correction[e] : v;
+        // (sigmoids without a correction are ranked by their logits: the same order, also where scores round to one)
+        ch[e] = correction ? v + correction[e] : sigmoid ? z[e] : v;
     }
     __syncwarp();
     const int per = experts / group_count;
