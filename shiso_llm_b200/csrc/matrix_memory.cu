@@ -31,7 +31,7 @@ template <typename AT> __device__ __forceinline__ float gate_of(float z) {
 
 // --------------------------------------------------------------------------- the gates
 
-constexpr int MG_THREADS = 256, MG_WARPS = MG_THREADS / 32;
+constexpr int MG_THREADS = 512, MG_WARPS = MG_THREADS / 32;
 
 struct GatesArgs {
     const float* logits;  // [T, 2 heads]: input gates, then forget gates
@@ -39,11 +39,11 @@ struct GatesArgs {
     long long top_stride;
     const int *q_start, *state_slots;
     float *keep, *add, *floor;  // [T, heads]
-    int heads, logs;  // logs: the two factors' logarithms
+    int heads, logs;  // logs: the two factors' base-2 logarithms
     float cap;
 };
 
-// One CTA per (head, sequence); 256 rows at a time.
+// One CTA per (head, sequence); 512 rows at a time, the next ones' logits on their way meanwhile.
 __global__ void __launch_bounds__(MG_THREADS) memory_gates_kernel(const GatesArgs a) {
     __shared__ float sF[MG_WARPS], sI[MG_WARPS];
     pdl_begin();
@@ -52,14 +52,23 @@ __global__ void __launch_bounds__(MG_THREADS) memory_gates_kernel(const GatesArg
     if (n <= 0) return;
     float* top = a.top + (size_t)a.state_slots[s] * a.top_stride + h;
     float m = *top;  // before this round's first row
+    const float* z = a.logits + (size_t)first * 2 * a.heads + h;
+    float zi = 0.0f, zf = 0.0f;
+    auto fetch = [&](int t) {
+        if (t < n) {
+            zi = z[(size_t)t * 2 * a.heads];
+            zf = z[(size_t)t * 2 * a.heads + a.heads];
+        }
+    };
+    fetch(threadIdx.x);
     for (int base = 0; base < n; base += MG_THREADS) {
         const int t = base + threadIdx.x;
         float f = 0.0f, i = -INFINITY;  // rows beyond the portion change nothing
         if (t < n) {
-            const float* z = a.logits + (size_t)(first + t) * 2 * a.heads;
-            i = capped(z[h], a.cap);
-            f = log_sigmoid(capped(z[a.heads + h], a.cap));
+            i = capped(zi, a.cap);
+            f = log_sigmoid(capped(zf, a.cap));
         }
+        fetch(t + MG_THREADS);
         float F = f, I = i;  // the composition of this warp's rows up to this one
 #pragma unroll
         for (int o = 1; o < 32; o <<= 1) {
@@ -82,8 +91,9 @@ __global__ void __launch_bounds__(MG_THREADS) memory_gates_kernel(const GatesArg
         if (lane == 0) last = before;
         if (t < n) {
             const size_t at = (size_t)(first + t) * a.heads + h;
-            a.keep[at] = a.logs ? f + (last - now) : expf(f + (last - now));
-            a.add[at] = a.logs ? i - now : expf(i - now);
+            constexpr float LOG2E = 1.4426950408889634f;
+            a.keep[at] = a.logs ? (f + (last - now)) * LOG2E : expf(f + (last - now));
+            a.add[at] = a.logs ? (i - now) * LOG2E : expf(i - now);
             a.floor[at] = expf(-now);
         }
         m = all;

@@ -1,10 +1,10 @@
 // The matrix memory's recurrence for prompt portions in chunks of 64 rows on the tensor cores (bfloat16 rows).
 //
-// With S the state before a chunk, l_t <= 0 the logarithm of row t's factor on the old state, b_t <= 0 that of
-// its factor on the new write and L_i = l_1 + .. + l_i,
+// With S the state before a chunk, l_t <= 0 the base-2 logarithm of row t's factor on the old state, b_t <= 0
+// that of its factor on the new write and L_i = l_1 + .. + l_i,
 //
-//     S^T q read at row i = e^(L_i) S^T q_i + sum_(j<=i) e^(L_i - L_j + b_j) (q_i . k_j) v_j
-//     S behind the chunk  = e^(L_64) S + sum_j e^(L_64 - L_j + b_j) k_j v_j^T,
+//     S^T q read at row i = 2^(L_i) S^T q_i + sum_(j<=i) 2^(L_i - L_j + b_j) (q_i . k_j) v_j
+//     S behind the chunk  = 2^(L_64) S + sum_j 2^(L_64 - L_j + b_j) k_j v_j^T,
 //
 // every exponent at most zero.  The normaliser is one more value column that is always 1.
 //
@@ -38,7 +38,7 @@ constexpr int V_ROW = VC * 2 + 16;  // bytes of a padded row of values, weighted
 struct ChunkArgs {
     const __nv_bfloat16 *q, *k, *v;
     long long q_ld, k_ld, v_ld;
-    const float *log_keep, *log_add;  // [T, heads]
+    const float *log_keep, *log_add;  // [T, heads], base 2
     float *state, *normaliser;
     long long state_stride, norm_stride;
     const int *q_start, *state_slots;
@@ -59,11 +59,20 @@ __device__ __forceinline__ void split2(float x, float y, uint32_t& hi, uint32_t&
 
 __device__ __forceinline__ void ldmatrix_a_trans(uint32_t addr, uint32_t (&r)[4]) { ldmatrix_x4_trans(addr, r[0], r[1], r[2], r[3]); }
 
+// 2^x of a weight (x <= 0): two units in the last place, below 2^-126 zero.
+__device__ __forceinline__ float ex2(float x) {
+    float y;
+    asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+    return y;
+}
+
+// DIM: the key size, or 0 where it is a run-time number.
+template <int DIM>
 __global__ void __launch_bounds__(MC_THREADS, 2) memory_chunks_kernel(const ChunkArgs a) {
     const int h = blockIdx.x, s = blockIdx.y, col0 = blockIdx.z * VC;
     const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
     const int wr = warp & 3, wc = warp >> 2, g = lane >> 2, t4 = lane & 3;
-    const int dim = a.dim, vdim = a.vdim, ksteps = dim / 16;
+    const int dim = DIM ? DIM : a.dim, vdim = a.vdim, ksteps = dim / 16;
     const int k_row = dim * 2 + 16, pieces = dim / 8;
     extern __shared__ __align__(16) uint8_t sm[];
     const int tile = CH * k_row;
@@ -90,19 +99,28 @@ __global__ void __launch_bounds__(MC_THREADS, 2) memory_chunks_kernel(const Chun
         if (col0 + c >= vdim)
             *reinterpret_cast<uint4*>(sm + stage * stage_bytes + 2 * tile + r * V_ROW + c * 2) = make_uint4(col0 + c == vdim ? 0x3f80u : 0u, 0u, 0u, 0u);
     }
+    const int shift = pieces > 8 ? 4 : pieces > 4 ? 3 : pieces > 2 ? 2 : 1;  // 2^shift threads a row of queries and keys
+    const int piece = tid & ((1 << shift) - 1), row_of = tid >> shift, rows_a_pass = MC_THREADS >> shift;
     auto load = [&](int chunk, int stage) {
         uint8_t* base = sm + stage * stage_bytes;
         const int row0 = chunk * CH, count = min(CH, n - row0);
-        for (int i = tid; i < CH * pieces; i += MC_THREADS) {
-            const int r = i / pieces, c = i % pieces;
-            const bool ok = r < count;
-            const size_t row = (size_t)(row0 + (ok ? r : 0));
-            cp_async16(base + r * k_row + c * 16, qp + row * a.q_ld + c * 8, ok);
-            cp_async16(base + tile + r * k_row + c * 16, kp + row * a.k_ld + c * 8, ok);
+        if (piece < pieces) {
+            uint8_t* to = base + row_of * k_row + piece * 16;
+            const __nv_bfloat16* from_q = qp + (size_t)(row0 + row_of) * a.q_ld + piece * 8;
+            const __nv_bfloat16* from_k = kp + (size_t)(row0 + row_of) * a.k_ld + piece * 8;
+#pragma unroll
+            for (int r = row_of; r < CH; r += rows_a_pass) {
+                const bool ok = r < count;
+                cp_async16(to, ok ? from_q : qp, ok);
+                cp_async16(to + tile, ok ? from_k : kp, ok);
+                to += rows_a_pass * k_row;
+                from_q += rows_a_pass * a.q_ld;
+                from_k += rows_a_pass * a.k_ld;
+            }
         }
-        for (int i = tid; i < CH * (VC / 8); i += MC_THREADS) {
-            const int r = i / (VC / 8), c = i % (VC / 8) * 8;
-            if (col0 + c >= vdim) continue;
+        static_assert(VC == 16 && MC_THREADS >= 2 * CH, "two threads a row of values");
+        if (tid < 2 * CH && col0 + (tid & 1) * 8 < vdim) {
+            const int r = tid >> 1, c = (tid & 1) * 8;
             const bool ok = r < count;
             cp_async16(base + 2 * tile + r * V_ROW + c * 2, vp + (size_t)(row0 + (ok ? r : 0)) * a.v_ld + col0 + c, ok);
         }
@@ -148,8 +166,9 @@ __global__ void __launch_bounds__(MC_THREADS, 2) memory_chunks_kernel(const Chun
         }
     publish();
 
-    const int half_steps = (ksteps + 1) / 2;
-    const int d_first = wc ? half_steps : 0, d_last = wc ? ksteps : half_steps;  // this warp's share of the channels of S^T q
+    const int half_steps = (ksteps + 1) / 2;  // wc shares out the channels of S^T q: each its own first
+    const int kk_first = wc ? half_steps : 0;
+    const int reads_steps = wc ? ksteps - half_steps : half_steps;
     for (int chunk = 0; chunk < chunks; ++chunk) {
         asm volatile("cp.async.wait_group 0;" ::: "memory");
         __syncthreads();  // the chunk has landed, the state is published, nobody reads the other stage any more
@@ -181,9 +200,11 @@ __global__ void __launch_bounds__(MC_THREADS, 2) memory_chunks_kernel(const Chun
         const uint32_t k_base = smem_addr(ks + (wc * 32 + (lane & 7) + (lane >> 4) * 8) * k_row + ((lane >> 3) & 1) * 16);
         const uint32_t s_off = ((lane & 7) + ((lane >> 3) & 1) * 8) * V_ROW + (lane >> 4) * 16;
 #pragma unroll 4
-        for (int kk = 0; kk < ksteps; ++kk) {
-            const bool reads = kk >= d_first && kk < d_last;
-            if (!sees && !reads) continue;
+        for (int step = 0; step < ksteps; ++step) {
+            const bool reads = step < reads_steps;
+            if (!sees && !reads) break;
+            int kk = kk_first + step;
+            if (kk >= ksteps) kk -= ksteps;
             uint32_t qf[4];
             ldmatrix_x4(q_base + kk * 32, qf[0], qf[1], qf[2], qf[3]);
             if (sees) {
@@ -208,7 +229,7 @@ __global__ void __launch_bounds__(MC_THREADS, 2) memory_chunks_kernel(const Chun
                 }
             }
         }
-        const float decay[2] = {expf(row_l[0]), expf(row_l[1])};
+        const float decay[2] = {ex2(row_l[0]), ex2(row_l[1])};
 #pragma unroll
         for (int j = 0; j < VC / 8; ++j)
 #pragma unroll
@@ -226,7 +247,7 @@ __global__ void __launch_bounds__(MC_THREADS, 2) memory_chunks_kernel(const Chun
 #pragma unroll
                     for (int e = 0; e < 4; ++e) {
                         const int row = wr * 16 + g + (e >> 1) * 8;
-                        m[e] = c + (e & 1) <= row ? dot[j][e] * expf(row_l[e >> 1] + ((e & 1) ? b1 : b0)) : 0.0f;
+                        m[e] = c + (e & 1) <= row ? dot[j][e] * ex2(row_l[e >> 1] + ((e & 1) ? b1 : b0)) : 0.0f;
                     }
                     split2(m[0], m[1], hi[half * 2], lo[half * 2]);
                     split2(m[2], m[3], hi[half * 2 + 1], lo[half * 2 + 1]);
@@ -250,14 +271,16 @@ __global__ void __launch_bounds__(MC_THREADS, 2) memory_chunks_kernel(const Chun
                     *reinterpret_cast<float2*>(share + (wr * 16 + g + half * 8) * (VC + 2) + j * 8 + t4 * 2) = make_float2(acc[j][half * 2], acc[j][half * 2 + 1]);
         }
         // ---- the values, weighted for the state behind the chunk
-        for (int i = tid; i < CH * (VC / 2); i += MC_THREADS) {
-            const int r = i / (VC / 2), c = i % (VC / 2) * 2;
-            const uint32_t raw = *reinterpret_cast<const uint32_t*>(vs + r * V_ROW + c * 2);
-            const float w = expf(last + gates[CH + r]);
-            uint32_t hi, lo;
-            split2(w * __uint_as_float(raw << 16), w * __uint_as_float(raw & 0xffff0000u), hi, lo);
-            *reinterpret_cast<uint32_t*>(w_hi + r * V_ROW + c * 2) = hi;
-            *reinterpret_cast<uint32_t*>(w_lo + r * V_ROW + c * 2) = lo;
+        {
+            static_assert(MC_THREADS == 4 * CH, "four threads a row of four columns each");
+            const int r = tid >> 2, at = r * V_ROW + (tid & 3) * 8;
+            const uint2 raw = *reinterpret_cast<const uint2*>(vs + at);
+            const float w = ex2(last + gates[CH + r]);
+            uint2 hi, lo;
+            split2(w * __uint_as_float(raw.x << 16), w * __uint_as_float(raw.x & 0xffff0000u), hi.x, lo.x);
+            split2(w * __uint_as_float(raw.y << 16), w * __uint_as_float(raw.y & 0xffff0000u), hi.y, lo.y);
+            *reinterpret_cast<uint2*>(w_hi + at) = hi;
+            *reinterpret_cast<uint2*>(w_lo + at) = lo;
         }
         __syncthreads();  // shares and weighted values are written, the published state has been read
         if (wc == 0) {
@@ -276,7 +299,7 @@ __global__ void __launch_bounds__(MC_THREADS, 2) memory_chunks_kernel(const Chun
         }
         // ---- the state
         if (holds) {
-            const float keep = expf(last);
+            const float keep = ex2(last);
 #pragma unroll
             for (int j = 0; j < VC / 8; ++j)
 #pragma unroll
@@ -330,17 +353,16 @@ SHISO_API int shiso_memory_chunks(const void* q, const void* k, const void* v, l
     if ((((uintptr_t)q | (uintptr_t)k | (uintptr_t)v) & 15) || q_ld % 8 || k_ld % 8 || v_ld % 8 || ((uintptr_t)out & 7)) return SHISO_ERR_ALIGN;
     const int k_row = dim * 2 + 16;
     const size_t smem = (size_t)2 * (2 * CH * k_row + CH * V_ROW + 2 * CH * 4) + 2 * dim * V_ROW + 2 * CH * V_ROW + CH * (VC + 2) * 4 + 8 * 2 * CH * 4;
-    static bool configured = false;
-    if (!configured) {
-        cudaError_t e = cudaFuncSetAttribute(memory_chunks_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, 112 * 1024);
+    auto kernel = dim == 128 ? memory_chunks_kernel<128> : dim == 64 ? memory_chunks_kernel<64> : memory_chunks_kernel<0>;
+    if (smem > 48 * 1024) {
+        cudaError_t e = cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, 112 * 1024);
         if (e != cudaSuccess) return (int)e;
-        configured = true;
     }
     if (smem > 112 * 1024) return SHISO_ERR_SHAPE;
     const ChunkArgs a = {(const __nv_bfloat16*)q, (const __nv_bfloat16*)k, (const __nv_bfloat16*)v, q_ld, k_ld, v_ld, log_keep, log_add, state,
                          normaliser, state_stride, norm_stride, q_start, state_slots, out, norm_out, heads, dim, vdim};
     // (without the dependent-launch attribute: CTAs that become resident under the tail of the kernel
     // before them pile up on the SMs that have room first, and a CTA here runs as long as the portion)
-    memory_chunks_kernel<<<dim3(heads, num_seqs, (vdim + 1 + VC - 1) / VC), MC_THREADS, smem, stream>>>(a);
+    kernel<<<dim3(heads, num_seqs, (vdim + 1 + VC - 1) / VC), MC_THREADS, smem, stream>>>(a);
     return launch_status();
 }

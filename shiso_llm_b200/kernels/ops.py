@@ -1909,7 +1909,8 @@ def memory_chunks_supported(proj, dim, vdim) -> bool:
 def memory_gates(logits, cap, top, step, logs=False):
     """``logits[T, 2 heads]`` (float32; input gates, then forget gates) to the factors on the old state and on
     the new write and to ``exp(-m)`` of the running maximum ``m``, float32 ``[T, heads]`` each; ``top`` (float32
-    ``[slots, heads]``) holds each request's ``m`` and is brought up to date.  ``logs``: the factors' logarithms."""
+    ``[slots, heads]``) holds each request's ``m`` and is brought up to date.  ``logs``: the factors' base-2
+    logarithms."""
     _check(logits, "gate logits", torch.float32, 2)
     tokens, heads = logits.shape[0], logits.shape[1] // 2
     stride = _slot_rows(top, "running maximum", torch.float32)
